@@ -13,14 +13,15 @@ the same number of tokens.  A mixer that keeps several things per request (keys 
 of blocks of keys, a recurrent state) declares a tuple of needs and gets a tuple of views in the same
 order.  A group with a window gives a page back as soon as every position in it
 lies before the window of the request's next token; its block-table entry becomes -1 and the
-attention kernels never look there.  A group whose keys are visible inside a chunk of positions only
+attention kernels never look there.  A window may leave the sequence's first positions visible for good (`keep_first`):
+their pages are not given back before the request ends.  A group whose keys are visible inside a chunk of positions only
 does the same with the pages that lie wholly before the chunk of the request's next token.
 
 A request moves through reserve(n) -> (the step runs) -> commit(n).  `reserve` takes the pages the
 next n tokens need in every group, or nothing at all."""
 from __future__ import annotations
 
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 from typing import Dict, Hashable, List, Optional, Tuple
 
 import torch
@@ -39,6 +40,8 @@ class KVNeed:
     # n > 1: the entry holds one row per block of n positions (a summary of the block, written when the block's
     # last position arrives), so a request of t tokens holds t // n rows; such an entry never gives pages back
     stride: int = 1
+    # with a window: the sequence's first n positions stay visible to every later token, so their pages are kept
+    keep_first: int = 0
 
     @property
     def v_dim(self) -> int:
@@ -48,6 +51,12 @@ class KVNeed:
     def bounded(self) -> bool:
         """True when keys far enough back are never read again, so that their pages can go back to the pool."""
         return self.window is not None or self.chunk is not None
+
+    def reaching(self, other: "KVNeed") -> "KVNeed":
+        """This need with its keys held as long as `other`, who reads the same cache, can see them too."""
+        window = None if self.window is None or other.window is None else max(self.window, other.window)
+        return replace(self, window=window, chunk=self.chunk if self.chunk == other.chunk else None,
+                       keep_first=0 if window is None else max(self.keep_first, other.keep_first))
 
 
 @dataclass(frozen=True)
@@ -112,6 +121,11 @@ class KVGroup:
         if self.need.chunk is not None:
             lowest_visible = max(lowest_visible, (next_pos // self.need.chunk) * self.need.chunk)
         return lowest_visible // self.page_size
+
+    @property
+    def kept_pages(self) -> int:
+        """How many pages at the front of a request hold positions that stay visible whatever the window."""
+        return -(-self.need.keep_first // self.page_size)
 
 
 class StateSlots:
@@ -182,6 +196,8 @@ class CacheManager:
         for need in needs:
             for one in flat(need):
                 if isinstance(one, KVNeed):
+                    if one.keep_first < 0 or (one.keep_first and one.window is None):
+                        raise ValueError("a cache entry keeps its first positions only where a window would drop them")
                     if one.stride < 1 or (one.stride > 1 and one.bounded):
                         raise ValueError("a strided cache entry holds every block: it has neither window nor chunk")
                     counts[one] = counts.get(one, 0) + 1
@@ -270,10 +286,10 @@ class CacheManager:
                 continue
             table = g.tables[rid]
             first = min(g.first_needed_page(self.kv_len[rid]), len(table))
-            gone = [p for p in table[:first] if p >= 0]
+            gone = [p for p in table[g.kept_pages:first] if p >= 0]
             if gone:
                 g.pool.free(gone, rid)
-                for i in range(first):
+                for i in range(g.kept_pages, first):
                     table[i] = -1
 
     def free_request(self, rid: Hashable) -> None:

@@ -7,7 +7,8 @@ from .dunelix import DunelixConfig
 from .zozenex import ZozenexConfig
 from .fiponex import FiponexConfig
 from .gevovik import GevovikConfig
+from .vigodra import VigodraConfig
 
-__all__ = ["ConfigError", "LlamaConfig", "DunelixConfig", "ZozenexConfig", "FiponexConfig", "GevovikConfig", "LayerCall", "LayerSpec", "ModelSpec", "PartSpec",
+__all__ = ["ConfigError", "LlamaConfig", "DunelixConfig", "ZozenexConfig", "FiponexConfig", "GevovikConfig", "VigodraConfig", "LayerCall", "LayerSpec", "ModelSpec", "PartSpec",
            "config_class_for", "config_from_dict", "load_config", "register_architecture",
            "registered_architectures"]

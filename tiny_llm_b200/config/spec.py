@@ -38,6 +38,8 @@ class LayerSpec:
     more: Tuple[Tuple[str, str, PartSpec, str], ...] = ()
     # what a branch's output is multiplied by before it joins the stream: x += residual_scale * mixer(norm1(x))
     residual_scale: float = 1.0
+    # what the stream is multiplied by where a block norms the sum: x = norm(stream_scale * x + mixer(x))
+    stream_scale: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -78,3 +80,6 @@ class ModelSpec:
     on_logits_name: str = "model.on_logits"
     # the embedding rows are multiplied by this (in 32-bit, as they are gathered into the stream)
     embedding_scale: float = 1.0
+    # name (behind a layer's prefix) of the weights of a depth average: with X_0 the embedding output and X_(i+1) the
+    # result of layer i, what goes on after layer i is sum_(j <= i + 1) weights[j] X_j (i + 2 numbers per layer)
+    depth_average: Optional[str] = None

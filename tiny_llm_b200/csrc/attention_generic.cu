@@ -10,7 +10,8 @@
 //
 // The keys a query at position p sees are j in [lo, p] with lo = max(0, p - window + 1) when there is a
 // window and lo >= (p / chunk) * chunk when keys are visible inside a chunk of positions only (chunks
-// are counted from position 0 of the sequence).  They are walked in
+// are counted from position 0 of the sequence), and, with a window, also the sequence's first `keep` positions.  A score
+// may get a learned bias by head and distance, rel[h][min(p - j, length - 1)] (added behind the scale).  They are walked in
 // tiles of 32 that start at multiples of 32 of the absolute position.  Tile number i (= j / 32) belongs
 // to lane i mod 8 of eight running softmaxes (m, l, o) in 32-bit, each of which takes its tiles in
 // ascending order; at the end the eight are merged in the order 0..7.  So the order of every sum is a
@@ -38,6 +39,9 @@ constexpr int MAX_HD = 256;
 // Where the rows of the cache lie and which keys are visible; `nq` and `nk` count (head, map) rows.
 struct Geometry {
   int nq, nk, maps, kd, vd, page_size, window, chunk;
+  int keep;                 // keys j < keep are visible to every later token, whatever the window
+  const float* rel;         // [query heads, rel_len]: what is added to a score at distance p - j (the last value beyond), or null
+  int rel_len;
   int kvec;   // key rows are read with 16-byte loads (their size and strides allow it); else value by value, same order
   long long k_page_stride, k_head_stride, v_page_stride, v_head_stride;
 };
@@ -65,6 +69,19 @@ __device__ __forceinline__ void load16(const __nv_bfloat16* p, float* dst) {
   }
 }
 
+__device__ __forceinline__ float biased(const Geometry& g, float s, int head, int distance) {
+  return g.rel == nullptr ? s : __fadd_rn(s, g.rel[(size_t)head * g.rel_len + min(distance, g.rel_len - 1)]);
+}
+// The tile after the one at j0 of the same way: tiles that lie wholly between the kept keys and the window are passed over.
+__device__ __forceinline__ int next_tile(const Geometry& g, int j0, int step, int first_in_window) {
+  const int n = j0 + step;
+  return n >= g.keep ? max(n, first_in_window) : n;
+}
+// The same for the launches that walk whole groups of tiles together.
+__device__ __forceinline__ bool tile_seen(const Geometry& g, int j0, int lo, int p) {
+  return j0 <= p && (j0 + 31 >= lo || j0 < g.keep);
+}
+
 constexpr int WAYS = 8;   // running softmaxes per (token, head); a constant of the arithmetic, not a tuning knob
 
 template <int OD>   // OD * 32 >= head size: the output values of a lane
@@ -77,10 +94,10 @@ struct Softmax {
 template <typename T, int OD>
 __device__ __forceinline__ void attend_tile(Softmax<OD>& st, int j0, int lo, int p, const float* q_row, const T* kcache,
                                             const T* vcache, const int* table, int max_blocks, int kh, int vh,
-                                            const Geometry& g, int lane) {
+                                            int head, const Geometry& g, int lane) {
   const int hd = g.kd, vd = g.vd, page_size = g.page_size;
   const int j = j0 + lane;
-  bool valid = j >= lo && j <= p && j / page_size < max_blocks;
+  bool valid = (j >= lo || j < g.keep) && j <= p && j / page_size < max_blocks;
   const int page = valid ? table[j / page_size] : -1;
   valid = valid && page >= 0;   // a table entry that names no page is never followed
   long long row_off = 0;
@@ -100,7 +117,7 @@ __device__ __forceinline__ void attend_tile(Softmax<OD>& st, int j0, int lo, int
     } else {
       for (int d = 0; d < hd; ++d) acc = fmaf(q_row[d], to_f32(krow[d]), acc);
     }
-    s = acc;
+    s = biased(g, acc, head, p - j);
   }
   const float m_new = fmaxf(st.m, warp_max(s));
   const float m_ref = m_new == -CUDART_INF_F ? 0.f : m_new;   // a tile without a visible key changes nothing
@@ -111,7 +128,7 @@ __device__ __forceinline__ void attend_tile(Softmax<OD>& st, int j0, int lo, int
 #pragma unroll
   for (int i = 0; i < OD; ++i) st.o[i] = __fmul_rn(st.o[i], corr);
   const int last = min(31, p - j0);
-  const int first = max(0, lo - j0);
+  const int first = j0 < g.keep ? 0 : max(0, lo - j0);
   for (int kk = first; kk <= last; ++kk) {
     const float pk = __shfl_sync(0xffffffffu, pr, kk);
     if (pk == 0.f) continue;   // uniform across the warp: nothing to add, and the row may name no page
@@ -162,11 +179,11 @@ constexpr int GH = 4;
 template <typename T, int OD>
 __device__ __forceinline__ void attend_tile_grouped(Softmax<OD> (&st)[GH], int nh, int j0, int lo, int p,
                                                     const float (*q_rows)[OD * 32], const T* kcache, const T* vcache,
-                                                    const int* table, int max_blocks, int kh, int vh,
+                                                    const int* table, int max_blocks, int kh, int vh, int head0,
                                                     const Geometry& g, int lane) {
   const int hd = g.kd, vd = g.vd, page_size = g.page_size;
   const int j = j0 + lane;
-  bool valid = j >= lo && j <= p && j / page_size < max_blocks;
+  bool valid = (j >= lo || j < g.keep) && j <= p && j / page_size < max_blocks;
   const int page = valid ? table[j / page_size] : -1;
   valid = valid && page >= 0;
   long long row_off = 0;
@@ -197,7 +214,7 @@ __device__ __forceinline__ void attend_tile_grouped(Softmax<OD> (&st)[GH], int n
       }
     }
 #pragma unroll
-    for (int i = 0; i < GH; ++i) s[i] = acc[i];
+    for (int i = 0; i < GH; ++i) s[i] = i < nh ? biased(g, acc[i], head0 + i, p - j) : acc[i];
   }
   float pr[GH];
 #pragma unroll
@@ -215,7 +232,7 @@ __device__ __forceinline__ void attend_tile_grouped(Softmax<OD> (&st)[GH], int n
     }
   }
   const int last = min(31, p - j0);
-  const int first = max(0, lo - j0);
+  const int first = j0 < g.keep ? 0 : max(0, lo - j0);
   for (int kk = first; kk <= last; ++kk) {
     float pk[GH];
     bool any = false;
@@ -280,7 +297,7 @@ paged_attention_grouped_kernel(const T* __restrict__ q, int q_row_stride, const 
     for (int d = lane; d < hd; d += 32) q_s[warp][i][d] = 0.f;
   __syncwarp();
 
-  const int first_group = (lo / (32 * WAYS)) * (32 * WAYS);
+  const int first_group = (lo / (32 * WAYS)) * (32 * WAYS), start = g.keep > 0 ? 0 : first_group;
   for (int w = 0; w < WAYS; ++w) {
     Softmax<OD> st[GH];
 #pragma unroll
@@ -289,9 +306,9 @@ paged_attention_grouped_kernel(const T* __restrict__ q, int q_row_stride, const 
 #pragma unroll
       for (int x = 0; x < OD; ++x) st[i].o[x] = 0.f;
     }
-    for (int j0 = first_group + w * 32; j0 <= p; j0 += 32 * WAYS)
-      if (j0 + 31 >= lo)
-        attend_tile_grouped<T, OD>(st, nh, j0, lo, p, q_s[warp], kcache, vcache, table, max_blocks, kh, vh, g, lane);
+    for (int j0 = start + w * 32; j0 <= p; j0 = next_tile(g, j0, 32 * WAYS, first_group + w * 32))
+      if (tile_seen(g, j0, lo, p))
+        attend_tile_grouped<T, OD>(st, nh, j0, lo, p, q_s[warp], kcache, vcache, table, max_blocks, kh, vh, kvh * group + h0, g, lane);
 #pragma unroll
     for (int i = 0; i < GH; ++i) {
       if (lane == 0) { way_s[warp][w][i][OD * 32] = st[i].m; way_s[warp][w][i][OD * 32 + 1] = st[i].l; }
@@ -350,15 +367,16 @@ paged_attention_generic_kernel(const T* __restrict__ q, int q_row_stride, const 
   }
 
   const int first_group = (lo / (32 * WAYS)) * (32 * WAYS);   // tile numbers are absolute: way = (j0 / 32) % WAYS
+  const int start = g.keep > 0 ? 0 : first_group;
   float o[OD], l, mx;
   if (SPLIT) {
     Softmax<OD> st;
     st.m = -CUDART_INF_F; st.l = 0.f;
 #pragma unroll
     for (int i = 0; i < OD; ++i) st.o[i] = 0.f;
-    for (int j0 = first_group + warp * 32; j0 <= p; j0 += 32 * WAYS)
-      if (j0 + 31 >= lo)
-        attend_tile(st, j0, lo, p, q_row, kcache, vcache, table, max_blocks, kh, vh, g, lane);
+    for (int j0 = start + warp * 32; j0 <= p; j0 = next_tile(g, j0, 32 * WAYS, first_group + warp * 32))
+      if (tile_seen(g, j0, lo, p))
+        attend_tile(st, j0, lo, p, q_row, kcache, vcache, table, max_blocks, kh, vh, h / maps, g, lane);
     if (lane == 0) { merge_s[warp][OD * 32] = st.m; merge_s[warp][OD * 32 + 1] = st.l; }
 #pragma unroll
     for (int i = 0; i < OD; ++i)
@@ -375,12 +393,12 @@ paged_attention_generic_kernel(const T* __restrict__ q, int q_row_stride, const 
 #pragma unroll
       for (int i = 0; i < OD; ++i) st[w].o[i] = 0.f;
     }
-    for (int g0 = first_group; g0 <= p; g0 += 32 * WAYS) {
+    for (int g0 = start; g0 <= p; g0 = next_tile(g, g0, 32 * WAYS, first_group)) {
 #pragma unroll
       for (int w = 0; w < WAYS; ++w) {
         const int j0 = g0 + w * 32;
-        if (j0 <= p && j0 + 31 >= lo)
-          attend_tile(st[w], j0, lo, p, q_row, kcache, vcache, table, max_blocks, kh, vh, g, lane);
+        if (tile_seen(g, j0, lo, p))
+          attend_tile(st[w], j0, lo, p, q_row, kcache, vcache, table, max_blocks, kh, vh, h / maps, g, lane);
       }
     }
     merge_ways<OD>([&](int w) { return st[w].m; }, [&](int w) { return st[w].l; }, [&](int w, int i) { return st[w].o[i]; }, o, l, mx);
@@ -427,23 +445,27 @@ using namespace tllm;
 // `nkv` key/value heads; the key cache holds nkv * maps rows per slot, the value cache nkv.  `chunk` > 0: keys are
 // visible inside the query's chunk of positions only.  out_f32 != 0: the output rows are float32 whatever the cache's type.
 // `sink` (float32, one per query head, or null): exp(sink) joins every softmax's denominator of that head.
+// `keep`: the first positions that a window leaves visible; `rel` (float32 [nq, rel_len] or null): a bias per head and
+// distance.
 extern "C" int tllm_paged_attention_maps(const void* q, int q_row_stride, const void* kcache, const void* vcache,
                                          const int* block_table, int max_blocks, const int* token_request,
                                          const int* positions, void* out, int n_tokens, int nq, int nkv, int maps, int kd,
                                          int vd, int page_size, long long k_page_stride, long long k_head_stride,
                                          long long v_page_stride, long long v_head_stride, float scale, int window,
                                          int chunk, int dtype, int out_f32, int split_override, const float* sink,
-                                         void* stream) {
+                                         int keep, const float* rel, int rel_len, void* stream) {
   TLLM_REQUIRE(n_tokens > 0 && nq > 0 && nkv > 0 && nq % nkv == 0 && maps > 0,
                "attention: %d tokens, %d heads, %d key/value heads (heads must be a multiple of key/value heads)", n_tokens, nq, nkv);
   TLLM_REQUIRE(kd >= 1 && kd <= MAX_HD && vd >= 1 && vd <= MAX_HD,
                "attention: key size %d / value size %d is not built (both up to %d)", kd, vd, MAX_HD);
   TLLM_REQUIRE(page_size > 0 && max_blocks > 0 && window >= 0 && chunk >= 0, "attention: page size %d, %d blocks, window %d, chunk %d", page_size, max_blocks, window, chunk);
+  TLLM_REQUIRE(keep >= 0 && (rel == nullptr || rel_len >= 1), "attention: %d kept keys, %d distances of a bias", keep, rel_len);
   const int elem = dtype == TLLM_F32 ? 4 : 2;
   TLLM_REQUIRE(dtype == TLLM_F32 || dtype == TLLM_BF16, "attention: unknown dtype code %d", dtype);
   Geometry g;
   g.kvec = (kd * elem) % 16 == 0 && ((size_t)kcache % 16) == 0 && (k_page_stride * elem) % 16 == 0 && (k_head_stride * elem) % 16 == 0;
   g.nq = nq * maps; g.nk = nkv * maps; g.maps = maps; g.kd = kd; g.vd = vd; g.page_size = page_size; g.window = window;
+  g.keep = window > 0 ? keep : 0; g.rel = rel; g.rel_len = rel_len;
   g.chunk = chunk; g.k_page_stride = k_page_stride; g.k_head_stride = k_head_stride; g.v_page_stride = v_page_stride;
   g.v_head_stride = v_head_stride;
   const long long tasks = (long long)n_tokens * g.nq;
@@ -484,5 +506,5 @@ extern "C" int tllm_paged_attention_generic(const void* q, int q_row_stride, con
                "attention: cache rows must be 16-byte aligned");
   return tllm_paged_attention_maps(q, q_row_stride, kcache, vcache, block_table, max_blocks, token_request, positions, out,
                                    n_tokens, nq, nkv, 1, hd, hd, page_size, page_stride, head_stride, page_stride, head_stride,
-                                   scale, window, 0, dtype, 0, split_override, nullptr, stream);
+                                   scale, window, 0, dtype, 0, split_override, nullptr, 0, nullptr, 0, stream);
 }

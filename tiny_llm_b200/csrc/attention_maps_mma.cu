@@ -17,7 +17,12 @@
 // With a sink (a learned score per head) the softmax's denominator also holds exp(sink); it has no value row.
 //
 // Visibility: key j is visible to the row of a token at position p iff j <= p, j > p - window when there is a
-// window, and j >= (p / chunk) * chunk when keys are visible inside a chunk of positions only.
+// window, and j >= (p / chunk) * chunk when keys are visible inside a chunk of positions only.  With a window the
+// sequence's first `keep` positions stay visible as well: a row tile then walks the tiles that hold them and, behind
+// those, the tiles of the window.
+//
+// A score may get a learned bias by head and distance (`rel`, one row per head, in units of log2 e; distances past the
+// row's end take its last value).  A warp whose rows all lie at least that far from a tile adds one number per row.
 #include "attention_tiles.cuh"
 
 #ifndef TLLM_VALUE_DIM
@@ -50,6 +55,9 @@ struct MapsParams {
   // leaves its rows' unnormalised sums, maximum and denominator in part[run][row][VD + 2]; a second kernel joins them.
   int splits, total_rows;
   float* part;
+  int keep;                      // keys j < keep are visible to every later token, whatever the window
+  const float* rel;              // [nq, rel_len] bias times log2(e), or null
+  int rel_len;
 };
 
 __device__ __forceinline__ int lowest_key(const MapsParams& p, int pos) {
@@ -68,7 +76,7 @@ __device__ __forceinline__ void load_tile(__nv_bfloat16* k_dst, __nv_bfloat16* v
   const bool is_v = warp >= 2;                 // warp-uniform
   const int row = (warp & 1) * 32 + lane;      // the key or value row of this lane
   const int j = j0 + row;
-  bool ok = j >= j_begin && j <= j_end;
+  bool ok = (j >= j_begin || j < p.keep) && j <= j_end;
   const int page = ok ? pages(j / p.page_size) : -1;
   ok = ok && page >= 0;
   const __nv_bfloat16* src = is_v ? p.vcache : p.kcache;
@@ -98,7 +106,7 @@ __device__ __forceinline__ void load_tile(__nv_bfloat16* k_dst, __nv_bfloat16* v
   }
 }
 
-template <int STAGES>
+template <int STAGES, bool REL>
 __global__ void __launch_bounds__(128, (VD <= 128 ? 3 : 1))
 attention_maps_kernel(const MapsParams p) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
@@ -131,13 +139,19 @@ attention_maps_kernel(const MapsParams p) {
   const int tok_hi = min(q_len - 1, (row0 + BM - 1) / group);
   const int key_hi = start + tok_hi;
   const int key_lo = lowest_key(p, start + tok_lo);    // lowest_key grows with the position
-  int t_begin = key_lo / BN, t_end = key_hi / BN + 1;   // t_end exclusive
+  // The walk: tiles 0 .. kept - 1 (those of the kept first keys that lie ahead of the window's), then the window's from
+  // w_begin; place i of it is the tile i < kept ? i : w_begin + i - kept.
+  const int w_begin = key_lo / BN;
+  const int kept = min(w_begin, (p.keep + BN - 1) / BN), skipped = w_begin - kept;
+  int t_begin = 0, t_end = key_hi / BN + 1 - skipped;   // places of the walk, t_end exclusive
   if (p.splits > 1) {   // this CTA's run of the tiles (possibly empty: its rows then say so with a maximum of -inf)
     const int per = (t_end - t_begin + p.splits - 1) / p.splits;
     t_begin = min(t_end, t_begin + (int)blockIdx.y * per);
     t_end = min(t_end, t_begin + per);
   }
-  const PageLookup pages = stage_pages(table, page_slots, t_begin * BN, t_end * BN, p.page_size, p.max_blocks, threadIdx.x, 128);
+  const auto tile_at = [&](int i) { return i < kept ? i : i + skipped; };
+  const PageLookup pages = stage_pages(table, page_slots, tile_at(max(t_begin, kept)) * BN, tile_at(max(t_end, kept)) * BN, p.page_size,
+                                       p.max_blocks, threadIdx.x, 128);   // (the kept keys' pages are looked up in place)
   __syncthreads();
 
   // ---- Q tile: row r -> token r / group, query row ((kvh * group + r % group) * maps + map)
@@ -154,7 +168,7 @@ attention_maps_kernel(const MapsParams p) {
 #pragma unroll
   for (int st = 0; st < STAGES - 1; ++st) {
     if (t_begin + st < t_end)
-      load_tile(k_s + st * BN * LDK, v_s + st * BN * LDV, pages, (t_begin + st) * BN, key_lo, key_hi, kh, kvh, p, threadIdx.x);
+      load_tile(k_s + st * BN * LDK, v_s + st * BN * LDV, pages, tile_at(t_begin + st) * BN, key_lo, key_hi, kh, kvh, p, threadIdx.x);
     cp_async_commit();
   }
 
@@ -170,6 +184,15 @@ attention_maps_kernel(const MapsParams p) {
   const int warp_pos_max = start + min(rows_total - 1, wrow + 15) / group;
   const int warp_lo_max = lowest_key(p, warp_pos_max);
   const int warp_lo_min = lowest_key(p, warp_pos_min);
+  const float* rel_a = nullptr;
+  const float* rel_b = nullptr;
+  float far_a = 0.f, far_b = 0.f;
+  if (REL) {
+    rel_a = p.rel + (size_t)(kvh * group + r_a % group) * p.rel_len;
+    rel_b = p.rel + (size_t)(kvh * group + r_b % group) * p.rel_len;
+    far_a = __ldg(rel_a + p.rel_len - 1);
+    far_b = __ldg(rel_b + p.rel_len - 1);
+  }
 
   float m_a = -CUDART_INF_F, m_b = -CUDART_INF_F, l_a = 0.f, l_b = 0.f;
   float o[VD / 8][4];
@@ -186,13 +209,13 @@ attention_maps_kernel(const MapsParams p) {
       const int nxt = tix + STAGES - 1;
       if (nxt < t_end) {
         const int ns = (nxt - t_begin) % STAGES;
-        load_tile(k_s + ns * BN * LDK, v_s + ns * BN * LDV, pages, nxt * BN, key_lo, key_hi, kh, kvh, p, threadIdx.x);
+        load_tile(k_s + ns * BN * LDK, v_s + ns * BN * LDV, pages, tile_at(nxt) * BN, key_lo, key_hi, kh, kvh, p, threadIdx.x);
       }
       cp_async_commit();
     }
-    const int j_base = tix * BN;
+    const int j_base = tile_at(tix) * BN;
     // a tile none of the warp's rows can see (behind their chunk or window, or ahead of them) is not computed
-    if (!warp_live || j_base > warp_pos_max || j_base + BN - 1 < warp_lo_min) continue;
+    if (!warp_live || j_base > warp_pos_max || (j_base + BN - 1 < warp_lo_min && j_base >= p.keep)) continue;
 
     // ---- S = Q K^T for this warp's 16 rows x 64 keys
     float s[BN / 8][4];
@@ -212,15 +235,37 @@ attention_maps_kernel(const MapsParams p) {
     }
 
     // ---- mask, running softmax in 32-bit; a tile that every row of the warp sees whole skips the mask
-    const float c = p.scale_log2;
-    if (!(j_base + BN - 1 <= warp_pos_min && j_base >= warp_lo_max)) {
+    const float c = REL ? 1.f : p.scale_log2;   // with a bias the scores are brought to powers of two here
+    if (REL) {
+      if (warp_pos_min - (j_base + BN - 1) >= p.rel_len - 1) {
+#pragma unroll
+        for (int i = 0; i < BN / 8; ++i) {
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            s[i][e] = fmaf(s[i][e], p.scale_log2, far_a);
+            s[i][2 + e] = fmaf(s[i][2 + e], p.scale_log2, far_b);
+          }
+        }
+      } else {
+        const int last = p.rel_len - 1, d_a = pos_a - j_base - t4 * 2, d_b = pos_b - j_base - t4 * 2;
+#pragma unroll
+        for (int i = 0; i < BN / 8; ++i) {
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {   // (distances of places behind the row's position are masked below)
+            s[i][e] = fmaf(s[i][e], p.scale_log2, __ldg(rel_a + max(0, min(d_a - i * 8 - e, last))));
+            s[i][2 + e] = fmaf(s[i][2 + e], p.scale_log2, __ldg(rel_b + max(0, min(d_b - i * 8 - e, last))));
+          }
+        }
+      }
+    }
+    if (!(j_base + BN - 1 <= warp_pos_min && (j_base >= warp_lo_max || j_base + BN <= p.keep))) {
 #pragma unroll
       for (int i = 0; i < BN / 8; ++i) {
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int j = j_base + i * 8 + t4 * 2 + e;
-          if (!(live_a && j <= pos_a && j >= lo_a)) s[i][e] = -CUDART_INF_F;
-          if (!(live_b && j <= pos_b && j >= lo_b)) s[i][2 + e] = -CUDART_INF_F;
+          if (!(live_a && j <= pos_a && (j >= lo_a || j < p.keep))) s[i][e] = -CUDART_INF_F;
+          if (!(live_b && j <= pos_b && (j >= lo_b || j < p.keep))) s[i][2 + e] = -CUDART_INF_F;
         }
       }
     }
@@ -351,7 +396,8 @@ extern "C" int tllm_attention_maps_mma(const void* q, int q_row_stride, const vo
                                        float* out, int n_tokens, int n_requests, int max_q_len, int nq, int nkv, int maps,
                                        int kd, int vd, int page_size, long long k_page_stride, long long k_head_stride,
                                        long long v_page_stride, long long v_head_stride, float scale, int window, int chunk,
-                                       const float* sink, int splits, float* part, void* stream) {
+                                       const float* sink, int splits, float* part, int keep, const float* rel, int rel_len,
+                                       void* stream) {
   TLLM_REQUIRE(splits >= 1 && splits <= 65535 && (splits == 1 || (part != nullptr && max_q_len * (nq / nkv) <= BM)),
                "attention_maps_mma: %d runs of key tiles need a buffer and rows that fit one tile", splits);
   TLLM_REQUIRE(kd == KD && vd == VD, "attention_maps_mma: built for key size %d and value size %d, called with %d and %d", KD, VD, kd, vd);
@@ -362,8 +408,10 @@ extern "C" int tllm_attention_maps_mma(const void* q, int q_row_stride, const vo
   TLLM_REQUIRE(((uintptr_t)q % 16) == 0 && (q_row_stride % 8) == 0 && ((uintptr_t)kcache % 16) == 0 && ((uintptr_t)vcache % 16) == 0 &&
                (k_page_stride % 8) == 0 && (k_head_stride % 8) == 0 && (v_page_stride % 8) == 0 && (v_head_stride % 8) == 0 &&
                ((uintptr_t)out % 8) == 0, "attention_maps_mma: rows must be 16-byte aligned");
+  TLLM_REQUIRE(keep >= 0 && (rel == nullptr || rel_len >= 1), "attention_maps_mma: %d kept keys, %d distances of a bias", keep, rel_len);
   const int group = nq / nkv;
   MapsParams p;
+  p.keep = window > 0 ? keep : 0; p.rel = rel; p.rel_len = rel_len;
   p.q = (const __nv_bfloat16*)q; p.kcache = (const __nv_bfloat16*)kcache; p.vcache = (const __nv_bfloat16*)vcache;
   p.block_table = block_table; p.cu_q = cu_q; p.q_start = q_start; p.out = out; p.sink = sink;
   p.k_page_stride = k_page_stride; p.k_head_stride = k_head_stride; p.v_page_stride = v_page_stride; p.v_head_stride = v_head_stride;
@@ -378,11 +426,14 @@ extern "C" int tllm_attention_maps_mma(const void* q, int q_row_stride, const vo
   const int smem = (BM * LDK + ST * BN * (LDK + LDV)) * 2 + TABLE_SLOTS * 4;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attention_maps_kernel<ST>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(attention_maps_kernel<ST, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(attention_maps_kernel<ST, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) TLLM_FAIL(TLLM_ERR_CUDA, "attention_maps_mma: cannot reserve %d bytes of shared memory: %s", smem, cudaGetErrorString(e));
     configured = true;
   }
-  TLLM_LAUNCH("attention_maps_mma", attention_maps_kernel<ST>, dim3((unsigned)gx, (unsigned)splits), 128, smem, (cudaStream_t)stream, p);
+  const dim3 grid((unsigned)gx, (unsigned)splits);
+  if (rel != nullptr) TLLM_LAUNCH("attention_maps_mma", (attention_maps_kernel<ST, true>), grid, 128, smem, (cudaStream_t)stream, p);
+  else TLLM_LAUNCH("attention_maps_mma", (attention_maps_kernel<ST, false>), grid, 128, smem, (cudaStream_t)stream, p);
   if (splits > 1)
     TLLM_LAUNCH("attention_maps_merge", attention_maps_merge_kernel, dim3((unsigned)((p.total_rows + 3) / 4)), 128, 0,
                 (cudaStream_t)stream, (const float*)part, out, sink, p.total_rows, splits, nq * maps, maps);

@@ -12,9 +12,15 @@
 // latent_kv_write: rows are [nq query heads of (nd plain | rd rotated) values | rank latent values | rd rotated key
 //   values | ...].  The latent is normed (weight of rank values) and written both as the first `rank` values of the
 //   token's key row and as its value row; the key's rotated part and every query head's rotated part are turned in
-//   pairs (2i, 2i + 1), i < rot_dims / 2, by p * freq[i]; the key part goes behind the latent in the key row, the
-//   query parts to q_out[t, head, rank : rank + rd].  (The plain query parts reach q_out through a product with the
+//   pairs (2i, 2i + 1) or halves (i, i + rot_dims / 2), i < rot_dims / 2, by p * freq[i]; the key part goes behind the
+//   latent in the key row, the query parts to q_out[t, head, rank : rank + rd].  (The plain query parts reach q_out through a product with the
 //   keys' up-projection, which is not this kernel's.)
+// conv_norm_kv_write: rows are [nq query heads | nkv key heads] of kd values, then nkv value heads of vd values, all of
+//   them channels of a short causal filter over time: y_t[c] = sum_j taps[c, j] x_(t - n_taps + 1 + j)[c] with x the
+//   projection plus its bias, zero before the sequence's start; the last n_taps - 1 inputs of every channel are the
+//   request's state.  The filtered queries TOGETHER (all heads of the token) are divided by sqrt(mean(y^2) + eps) and
+//   multiplied by a weight per channel, and so are the keys.  Queries go to a buffer of their own (other tokens' filters
+//   still read the projection), keys and values to their pages.
 // sigmoid_gate: out[t, h, :] = x[t, h, :] * sigmoid(gate), the gate one value per element or one per head.
 #include "common.cuh"
 
@@ -127,6 +133,7 @@ struct LatentArgs {
   long long k_page_stride, v_page_stride;
   int n_tokens;
   float rot_mag;             // cos and sin are multiplied by this
+  int rot_pairs;             // pairs (2i, 2i + 1), or halves (i, i + rot_dims / 2)
 };
 
 // With kcache == null the rows hold queries only: their rotated parts are turned and nothing is written to a cache
@@ -175,8 +182,26 @@ __global__ void __launch_bounds__(128) latent_kv_write_kernel(LatentArgs a) {
       }
     }
   }
-  // rotated parts: unit 0 is the key's, unit 1 + h query head h's; pairs (2i, 2i + 1)
-  const int half = (a.rd + 1) / 2, half_rot = a.rot_dims / 2;
+  // rotated parts: unit 0 is the key's, unit 1 + h query head h's
+  const int half_rot = a.rot_dims / 2;
+  if (!a.rot_pairs) {   // a unit's items: half_rot halves (i, i + half_rot), then the values that do not turn
+    const int items = a.rd - half_rot;
+    for (int idx = threadIdx.x; idx < (a.nq + 1) * items; idx += blockDim.x) {
+      const int u = idx / items, i = idx % items;
+      if (u == 0 && slot < 0) continue;
+      const T* src = u == 0 ? lat + a.rank : row + (size_t)(u - 1) * qd + a.nd;
+      T* dst = u == 0 ? krow + a.rank : (T*)a.q_out + ((size_t)t * a.nq + (u - 1)) * kd + a.rank;
+      if (i < half_rot) {
+        const float x = to_f32(src[i]), y = to_f32(src[i + half_rot]), c = cs[i], s = sn[i];
+        dst[i] = from_f32<T>(fmaf(x, c, -__fmul_rn(y, s)));
+        dst[i + half_rot] = from_f32<T>(fmaf(y, c, __fmul_rn(x, s)));
+      } else {
+        dst[i + half_rot] = src[i + half_rot];
+      }
+    }
+    return;
+  }
+  const int half = (a.rd + 1) / 2;
   for (int idx = threadIdx.x; idx < (a.nq + 1) * half; idx += blockDim.x) {
     const int u = idx / half, i = idx % half;
     if (u == 0 && slot < 0) continue;
@@ -193,6 +218,176 @@ __global__ void __launch_bounds__(128) latent_kv_write_kernel(LatentArgs a) {
     dst[0] = from_f32<T>(ox);
     if (pair) dst[1] = from_f32<T>(oy);
   }
+}
+
+struct ConvArgs {
+  const void* proj;             // [T, ld], channels [queries | keys | values] first
+  int ld, nq, nkv, kd, vd;
+  const float* bias;            // [channels] or null
+  const float* taps;            // [channels, n_taps]; null: no filter (n_taps = 1)
+  int n_taps;
+  float* kept;                  // [slots, n_taps - 1, channels]: inputs of the tokens before this step, oldest first
+  const int *slots, *cu_q, *token_request;
+  const float *wq, *wk;         // norm weights [nq * kd], [nkv * kd] or null
+  float eps;
+  void* q_out;                  // [T, nq * kd]
+  void *kcache, *vcache;
+  const int* slot_mapping;
+  int page_size;
+  long long k_page_stride, k_head_stride, v_page_stride, v_head_stride;
+  int n_tokens;
+  int update;                   // every request brings one token: its kept inputs move up here
+};
+
+template <typename T, int V> struct Piece { T v[V]; };   // V neighbouring channels; 8 of them are 16-byte aligned
+template <> struct __align__(16) Piece<float, 8> { float v[8]; };
+template <> struct __align__(16) Piece<__nv_bfloat16, 8> { __nv_bfloat16 v[8]; };
+
+// A CTA takes TOK consecutive tokens of the step with all their channels, V channels per thread and turn; the filtered
+// queries and keys wait in shared memory for their sums of squares.  NT: the number of taps (0: any).  Which thread meets
+// which channel depends on the sizes alone, so a token's sums have the same order in every batch.
+template <typename T, int V, int TOK, int NT>
+__global__ void conv_norm_kv_write_kernel(ConvArgs a) {
+  extern __shared__ float ys[];        // [TOK, (nq + nkv) * kd]
+  __shared__ float part[2 * TOK][33];
+  pdl_trigger();
+  const int nqc = a.nq * a.kd, nkc = a.nkv * a.kd, nvc = a.nkv * a.vd, channels = nqc + nkc + nvc, nqk = nqc + nkc;
+  const int taps_n = NT ? NT : a.n_taps;
+  const int t0 = blockIdx.x * TOK;
+  pdl_wait();
+  const T* proj = (const T*)a.proj;
+  float ssq[TOK], ssk[TOK];
+#pragma unroll
+  for (int i = 0; i < TOK; ++i) ssq[i] = ssk[i] = 0.f;
+  int first[TOK];
+  float* kept[TOK];
+  long long slot[TOK];
+#pragma unroll
+  for (int i = 0; i < TOK; ++i) {
+    const int t = min(t0 + i, a.n_tokens - 1);
+    const int req = a.token_request[t];
+    first[i] = a.cu_q[req];
+    kept[i] = taps_n > 1 ? a.kept + (size_t)a.slots[req] * (taps_n - 1) * channels : nullptr;
+    slot[i] = a.slot_mapping[t];
+  }
+  for (int c = threadIdx.x * V; c < channels; c += blockDim.x * V) {
+    float w[NT ? NT * V : 1];
+    if (NT) {
+#pragma unroll
+      for (int j = 0; j < NT * V; ++j) w[j] = a.taps[(size_t)c * NT + j];
+    }
+    float bias[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) bias[e] = a.bias ? a.bias[c + e] : 0.f;
+#pragma unroll
+    for (int i = 0; i < TOK; ++i) {
+      const int t = t0 + i;
+      if (t >= a.n_tokens) continue;
+      float y[V], x[V];
+#pragma unroll
+      for (int e = 0; e < V; ++e) y[e] = 0.f;
+#pragma unroll
+      for (int j = 0; j < taps_n; ++j) {
+        const int n = t - first[i] - (taps_n - 1) + j;   // index among the request's tokens of this step; < 0: kept ones
+        if (n >= 0) {
+          const Piece<T, V> p = *reinterpret_cast<const Piece<T, V>*>(proj + (size_t)(first[i] + n) * a.ld + c);
+#pragma unroll
+          for (int e = 0; e < V; ++e) x[e] = to_f32(p.v[e]) + bias[e];
+        } else {
+          const Piece<float, V> p = *reinterpret_cast<const Piece<float, V>*>(kept[i] + (size_t)(taps_n - 1 + n) * channels + c);
+#pragma unroll
+          for (int e = 0; e < V; ++e) x[e] = p.v[e];
+          // the entry just read is the only reader's: what it holds next is the entry behind it
+          if (a.update && j > 0) *reinterpret_cast<Piece<float, V>*>(kept[i] + (size_t)(j - 1) * channels + c) = p;
+        }
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          const float f = NT ? w[e * (NT ? NT : 1) + (NT ? j : 0)] : (a.taps ? a.taps[(size_t)(c + e) * taps_n + j] : 1.f);
+          y[e] = fmaf(f, x[e], y[e]);
+        }
+      }
+      if (a.update && taps_n > 1) {   // x is the token's own input now
+        Piece<float, V> p;
+#pragma unroll
+        for (int e = 0; e < V; ++e) p.v[e] = x[e];
+        *reinterpret_cast<Piece<float, V>*>(kept[i] + (size_t)(taps_n - 2) * channels + c) = p;
+      }
+      if (c >= nqk) {   // values have no norm
+        if (slot[i] < 0) continue;
+        const int h = (c - nqk) / a.vd, d = (c - nqk) % a.vd;
+        Piece<T, V> p;
+#pragma unroll
+        for (int e = 0; e < V; ++e) p.v[e] = from_f32<T>(y[e]);
+        *reinterpret_cast<Piece<T, V>*>((T*)a.vcache + slot[i] / a.page_size * a.v_page_stride + (long long)h * a.v_head_stride +
+                                        slot[i] % a.page_size * a.vd + d) = p;
+        continue;
+      }
+      float ss = 0.f;
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        ys[(size_t)i * nqk + c + e] = y[e];
+        ss = fmaf(y[e], y[e], ss);
+      }
+      if (c < nqc) ssq[i] += ss; else ssk[i] += ss;
+    }
+  }
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+#pragma unroll
+  for (int i = 0; i < TOK; ++i) {
+    const float q = warp_sum(ssq[i]), k = warp_sum(ssk[i]);
+    if (lane == 0) { part[2 * i][warp] = q; part[2 * i + 1][warp] = k; }
+  }
+  __syncthreads();
+  for (int s = warp; s < 2 * TOK; s += warps) {
+    const float v = warp_sum(lane < warps ? part[s][lane] : 0.f);
+    if (lane == 0) part[s][32] = 1.f / sqrtf(v / (float)((s & 1) ? nkc : nqc) + a.eps);
+  }
+  __syncthreads();
+  for (int c = threadIdx.x * V; c < nqk; c += blockDim.x * V) {
+    const bool is_q = c < nqc;
+    const float* wn = is_q ? a.wq : a.wk;
+    float w[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) w[e] = wn ? wn[(is_q ? c : c - nqc) + e] : 1.f;
+    const int h = (c - nqc) / a.kd, d = (c - nqc) % a.kd;
+#pragma unroll
+    for (int i = 0; i < TOK; ++i) {
+      const int t = t0 + i;
+      if (t >= a.n_tokens || (!is_q && slot[i] < 0)) continue;
+      const float f = wn ? part[2 * i + (is_q ? 0 : 1)][32] : 1.f;
+      Piece<T, V> p;
+#pragma unroll
+      for (int e = 0; e < V; ++e) p.v[e] = from_f32<T>(__fmul_rn(__fmul_rn(ys[(size_t)i * nqk + c + e], f), w[e]));
+      T* dst = is_q ? (T*)a.q_out + (size_t)t * nqc + c
+                    : (T*)a.kcache + slot[i] / a.page_size * a.k_page_stride + (long long)h * a.k_head_stride +
+                          slot[i] % a.page_size * a.kd + d;
+      *reinterpret_cast<Piece<T, V>*>(dst) = p;
+    }
+  }
+}
+
+template <typename T, int V, int TOK, int NT>
+static int launch_conv(const ConvArgs& a, cudaStream_t s) {
+  const int channels = (a.nq + a.nkv) * a.kd + a.nkv * a.vd, pieces = channels / V;
+  const int threads = pieces >= 512 ? 512 : (pieces + 31) / 32 * 32;
+  const size_t smem = (size_t)TOK * (a.nq + a.nkv) * a.kd * 4;
+  static size_t configured = 48 * 1024;
+  if (smem + 2 * TOK * 33 * 4 > configured) {
+    cudaError_t e = cudaFuncSetAttribute(conv_norm_kv_write_kernel<T, V, TOK, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) TLLM_FAIL(TLLM_ERR_CUDA, "conv_norm_kv_write: cannot reserve %d bytes of shared memory: %s", (int)smem, cudaGetErrorString(e));
+    configured = smem + 2 * TOK * 33 * 4;
+  }
+  TLLM_LAUNCH("conv_norm_kv_write", (conv_norm_kv_write_kernel<T, V, TOK, NT>), (unsigned)((a.n_tokens + TOK - 1) / TOK), threads, smem, s, a);
+  return TLLM_OK;
+}
+
+template <typename T>
+static int launch_conv_sizes(const ConvArgs& a, bool vec, cudaStream_t s) {
+  constexpr int TOK = 4;
+  const bool many = !a.update && a.n_tokens >= 148 * TOK && (size_t)TOK * (a.nq + a.nkv) * a.kd * 4 <= 160 * 1024;
+  if (!vec) return launch_conv<T, 1, 1, 0>(a, s);
+  if (a.taps && a.n_taps == 4) return many ? launch_conv<T, 8, TOK, 4>(a, s) : launch_conv<T, 8, 1, 4>(a, s);
+  return many ? launch_conv<T, 8, TOK, 0>(a, s) : launch_conv<T, 8, 1, 0>(a, s);
 }
 
 // x float32 [T, heads * vd]; gate rows of ldg values in the engine's dtype, heads * vd of them (per_head = 0) or
@@ -246,7 +441,7 @@ extern "C" int tllm_latent_kv_write(const void* proj, int ld, int nq, int nd, in
                                     const float* w_latent, const float* freq, float eps, const int* positions, void* q_out,
                                     void* kcache, void* vcache, const int* slot_mapping, int page_size,
                                     long long k_page_stride, long long v_page_stride, int n_tokens, float rot_mag,
-                                    int dtype, void* stream) {
+                                    int rot_pairs, int dtype, void* stream) {
   TLLM_REQUIRE(n_tokens > 0 && nq > 0 && nd >= 0 && rd >= 0 && rank > 0 && rank <= MAX_ROW,
                "latent_kv_write: %d tokens, %d heads, sizes %d + %d, latent %d (at most %d)", n_tokens, nq, nd, rd, rank, MAX_ROW);
   TLLM_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= rd && rot_dims <= 512 && (rot_dims == 0 || freq),
@@ -256,12 +451,41 @@ extern "C" int tllm_latent_kv_write(const void* proj, int ld, int nq, int nd, in
   a.proj = proj; a.ld = ld; a.nq = nq; a.nd = nd; a.rd = rd; a.rank = rank; a.rot_dims = rot_dims; a.w_latent = w_latent;
   a.freq = freq; a.eps = eps; a.positions = positions; a.q_out = q_out; a.kcache = kcache; a.vcache = vcache;
   a.slot_mapping = slot_mapping; a.page_size = page_size; a.k_page_stride = k_page_stride; a.v_page_stride = v_page_stride;
-  a.n_tokens = n_tokens; a.rot_mag = rot_mag;
+  a.n_tokens = n_tokens; a.rot_mag = rot_mag; a.rot_pairs = rot_pairs;
   cudaStream_t s = (cudaStream_t)stream;
   if (dtype == TLLM_F32) TLLM_LAUNCH("latent_kv_write", latent_kv_write_kernel<float>, n_tokens, 128, 0, s, a);
   else if (dtype == TLLM_BF16) TLLM_LAUNCH("latent_kv_write", latent_kv_write_kernel<__nv_bfloat16>, n_tokens, 128, 0, s, a);
   else TLLM_FAIL(TLLM_ERR_ARG, "latent_kv_write: unknown dtype code %d", dtype);
   return TLLM_OK;
+}
+
+extern "C" int tllm_conv_norm_kv_write(const void* proj, int ld, int nq, int nkv, int kd, int vd, const float* bias,
+                                       const float* taps, int n_taps, float* kept, const int* slots, const int* cu_q,
+                                       const int* token_request, const float* wq, const float* wk, float eps, void* q_out,
+                                       void* kcache, void* vcache, const int* slot_mapping, int page_size,
+                                       long long k_page_stride, long long k_head_stride, long long v_page_stride,
+                                       long long v_head_stride, int n_tokens, int update, int dtype, void* stream) {
+  TLLM_REQUIRE(n_tokens > 0 && nq > 0 && nkv > 0 && kd > 0 && vd > 0 && ((long long)(nq + nkv) * kd) * 4 <= 220 * 1024,
+               "conv_norm_kv_write: %d tokens, %d / %d heads, key size %d, value size %d (queries and keys of a token: at most %d values)",
+               n_tokens, nq, nkv, kd, vd, 220 * 256);
+  TLLM_REQUIRE(n_taps >= 1 && (n_taps == 1 || (taps && kept && slots)) && proj && q_out && kcache && vcache && slot_mapping && cu_q &&
+               token_request && page_size > 0 && (wq == nullptr) == (wk == nullptr),
+               "conv_norm_kv_write: %d taps; a filter needs weights, kept inputs and slots; norm weights for both or neither", n_taps);
+  ConvArgs a;
+  a.proj = proj; a.ld = ld; a.nq = nq; a.nkv = nkv; a.kd = kd; a.vd = vd; a.bias = bias; a.taps = taps; a.n_taps = n_taps;
+  a.kept = kept; a.slots = slots; a.cu_q = cu_q; a.token_request = token_request; a.wq = wq; a.wk = wk; a.eps = eps;
+  a.q_out = q_out; a.kcache = kcache; a.vcache = vcache; a.slot_mapping = slot_mapping; a.page_size = page_size;
+  a.k_page_stride = k_page_stride; a.k_head_stride = k_head_stride; a.v_page_stride = v_page_stride;
+  a.v_head_stride = v_head_stride; a.n_tokens = n_tokens; a.update = update;
+  const int esz = dtype == TLLM_F32 ? 4 : 2;
+  const auto ok16 = [](const void* p) { return ((uintptr_t)p % 16) == 0; };
+  const bool vec = kd % 8 == 0 && vd % 8 == 0 && ok16(proj) && ok16(q_out) && ok16(kcache) && ok16(vcache) && ok16(kept) &&
+                   ((long long)ld * esz) % 16 == 0 && (k_page_stride * esz) % 16 == 0 && (k_head_stride * esz) % 16 == 0 &&
+                   (v_page_stride * esz) % 16 == 0 && (v_head_stride * esz) % 16 == 0;
+  cudaStream_t s = (cudaStream_t)stream;
+  if (dtype == TLLM_F32) return launch_conv_sizes<float>(a, vec, s);
+  if (dtype == TLLM_BF16) return launch_conv_sizes<__nv_bfloat16>(a, vec, s);
+  TLLM_FAIL(TLLM_ERR_ARG, "conv_norm_kv_write: unknown dtype code %d", dtype);
 }
 
 extern "C" int tllm_sigmoid_gate(const float* x, const void* gate, int ldg, int per_head, void* out, long long n_tokens,

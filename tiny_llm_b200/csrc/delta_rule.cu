@@ -17,7 +17,8 @@
 //   request's earlier tokens in this step and, ahead of them, the inputs kept in the state; SiLU; query and key rows
 //   are divided by sqrt(sum(x^2) + unit_eps); the value rows' warps also leave the head's decay and step size:
 //   g = exp(-exp(A_log) softplus(a + dt_bias)), beta = sigmoid(b).  All outputs float32.
-// conv_state_update: the state's kept inputs after the step: the last taps - 1 of (kept inputs ++ the step's).
+// conv_state_update: the state's kept inputs after the step: the last taps - 1 of (kept inputs ++ the step's, plus their
+//   bias where the projection has one).
 // delta_rule_scan: a group of 8 lanes owns one value column of one (request, head): the column's state rows lie in
 //   the lanes' registers (a lane holds R consecutive rows).  Per token one round of shuffles gives the column's
 //   S^T k, S^T q and k . q from the state as it was; with those
@@ -135,7 +136,7 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(PrepArgs a) {
 template <typename T>
 __global__ void conv_state_update_kernel(const T* __restrict__ proj, int ld, float* __restrict__ kept_all,
                                          const int* __restrict__ slots, const int* __restrict__ cu_q, int n_taps,
-                                         int channels, int n_requests) {
+                                         int channels, int n_requests, const float* __restrict__ bias) {
   pdl_trigger();
   pdl_wait();
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
@@ -143,9 +144,10 @@ __global__ void conv_state_update_kernel(const T* __restrict__ proj, int ld, flo
   if (c >= channels || req >= n_requests) return;
   const int first = cu_q[req], n = cu_q[req + 1] - first;
   float* kept = kept_all + (size_t)slots[req] * (n_taps - 1) * channels;
+  const float add = bias ? bias[c] : 0.f;
   for (int j = 0; j < n_taps - 1; ++j) {
     const int i = n - (n_taps - 1) + j;   // index among this step's tokens; < 0: an input kept before
-    kept[(size_t)j * channels + c] = i >= 0 ? to_f32(proj[(size_t)(first + i) * ld + c]) : kept[(size_t)(j + n) * channels + c];
+    kept[(size_t)j * channels + c] = i >= 0 ? to_f32(proj[(size_t)(first + i) * ld + c]) + add : kept[(size_t)(j + n) * channels + c];
   }
 }
 
@@ -404,16 +406,16 @@ extern "C" int tllm_delta_prepare(const void* proj, int ld, const float* taps, i
 }
 
 extern "C" int tllm_conv_state_update(const void* proj, int ld, float* kept, const int* slots, const int* cu_q, int n_taps,
-                                      int channels, int n_requests, int dtype, void* stream) {
+                                      int channels, int n_requests, const float* bias, int dtype, void* stream) {
   TLLM_REQUIRE(n_requests > 0 && channels > 0 && n_taps >= 1 && n_requests <= 65535,
                "conv_state_update: %d requests, %d channels, %d taps", n_requests, channels, n_taps);
   if (n_taps == 1) return TLLM_OK;
   const dim3 grid((channels + 127) / 128, n_requests);
   cudaStream_t s = (cudaStream_t)stream;
   if (dtype == TLLM_F32)
-    TLLM_LAUNCH("conv_state_update", conv_state_update_kernel<float>, grid, 128, 0, s, (const float*)proj, ld, kept, slots, cu_q, n_taps, channels, n_requests);
+    TLLM_LAUNCH("conv_state_update", conv_state_update_kernel<float>, grid, 128, 0, s, (const float*)proj, ld, kept, slots, cu_q, n_taps, channels, n_requests, bias);
   else if (dtype == TLLM_BF16)
-    TLLM_LAUNCH("conv_state_update", conv_state_update_kernel<__nv_bfloat16>, grid, 128, 0, s, (const __nv_bfloat16*)proj, ld, kept, slots, cu_q, n_taps, channels, n_requests);
+    TLLM_LAUNCH("conv_state_update", conv_state_update_kernel<__nv_bfloat16>, grid, 128, 0, s, (const __nv_bfloat16*)proj, ld, kept, slots, cu_q, n_taps, channels, n_requests, bias);
   else TLLM_FAIL(TLLM_ERR_ARG, "conv_state_update: unknown dtype code %d", dtype);
   return TLLM_OK;
 }

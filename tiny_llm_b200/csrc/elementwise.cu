@@ -11,16 +11,24 @@ TLLM_DEFINE_LAST_ERROR
 namespace tllm {
 
 // ---------------------------------------------------------------- embedding: out[t,:] = table[tokens[t],:] * scale
+// `twin` (float32) and `copy` (bfloat16), where given, receive the same rows: a model that comes back to the embedding
+// output later, and a first layer that reads the stream itself.
 template <typename T>
 __global__ void embedding_kernel(const int* __restrict__ tokens, const T* __restrict__ table,
-                                 float* __restrict__ out, int n_tokens, int hidden, float scale) {
+                                 float* __restrict__ out, int n_tokens, int hidden, float scale,
+                                 float* __restrict__ twin, __nv_bfloat16* __restrict__ copy) {
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
   if (t >= n_tokens) return;
   const T* row = table + (size_t)tokens[t] * hidden;
   float* dst = out + (size_t)t * hidden;
-  for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = __fmul_rn(to_f32(row[i]), scale);
+  for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+    const float v = __fmul_rn(to_f32(row[i]), scale);
+    dst[i] = v;
+    if (twin) twin[(size_t)t * hidden + i] = v;
+    if (copy) copy[(size_t)t * hidden + i] = __float2bfloat16_rn(v);
+  }
 }
 
 // ---------------------------------------------------------------- RMSNorm
@@ -125,12 +133,24 @@ __global__ void rms_norm_vec_kernel(const float* __restrict__ x, const float* __
   }
 }
 
-// ---------------------------------------------------------------- act(gate) * up, act = SiLU (0) or ReLU (1)
+// What a gated feed-forward makes of a gate value and an up value: SiLU(g) u (act 0), ReLU(g) u (act 1), or the clamped
+// form (act 2): g <- min(g, limit), u <- clamp(u, -limit, limit), g sigmoid(1.702 g) (u + 1).
+__device__ __forceinline__ float glu_value(float g, float u, int act, float limit) {
+  if (act == 1) return fmaxf(g, 0.f) * u;
+  if (act == 2) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
+  }
+  return g / (1.f + expf(-g)) * u;
+}
+
+// ---------------------------------------------------------------- act(gate) * up, act as in glu_value
 // `gu` rows hold gate and up interleaved in blocks: [2 g B, 2 g B + B) gate, next B up.  With
 // ZERO the source is a float32 accumulation buffer (split-K partial sums land there) that this
 // kernel hands back cleared: every element is read once, by the thread that then zeroes it.
 template <typename TIn, typename TOut, bool ZERO>
-__global__ void silu_mul_kernel(TIn* __restrict__ gu, TOut* __restrict__ out, int m, int inter, int blk, int act) {
+__global__ void silu_mul_kernel(TIn* __restrict__ gu, TOut* __restrict__ out, int m, int inter, int blk, int act, float limit) {
   pdl_trigger();
   pdl_wait();
   const size_t total = (size_t)m * inter;
@@ -141,7 +161,7 @@ __global__ void silu_mul_kernel(TIn* __restrict__ gu, TOut* __restrict__ out, in
     TIn* src = gu + (size_t)row * 2 * inter + (size_t)g * 2 * blk;
     const float gate = to_f32(src[j]), up = to_f32(src[blk + j]);
     if (ZERO) { src[j] = from_f32<TIn>(0.f); src[blk + j] = from_f32<TIn>(0.f); }
-    out[idx] = from_f32<TOut>((act == 1 ? fmaxf(gate, 0.f) : gate / (1.f + expf(-gate))) * up);
+    out[idx] = from_f32<TOut>(glu_value(gate, up, act, limit));
   }
 }
 
@@ -149,7 +169,7 @@ __global__ void silu_mul_kernel(TIn* __restrict__ gu, TOut* __restrict__ out, in
 // and the rows 16-byte aligned): two 16-byte loads, one store.  ZERO hands the sums back cleared.
 template <typename TOut, bool ZERO>
 __global__ void __launch_bounds__(256) silu_mul_f32x4_kernel(float* __restrict__ gu, TOut* __restrict__ out, int m, int inter,
-                                                             int blk, int act) {
+                                                             int blk, int act, float limit) {
   pdl_trigger();
   pdl_wait();
   const int per_row = inter >> 2;
@@ -166,7 +186,7 @@ __global__ void __launch_bounds__(256) silu_mul_f32x4_kernel(float* __restrict__
     const float gv[4] = {gate.x, gate.y, gate.z, gate.w}, uv[4] = {up.x, up.y, up.z, up.w};
     float r[4];
 #pragma unroll
-    for (int i = 0; i < 4; ++i) r[i] = (act == 1 ? fmaxf(gv[i], 0.f) : gv[i] / (1.f + expf(-gv[i]))) * uv[i];
+    for (int i = 0; i < 4; ++i) r[i] = glu_value(gv[i], uv[i], act, limit);
     TOut* dst = out + (size_t)row * inter + col;
     if constexpr (sizeof(TOut) == 2) {
       __nv_bfloat162 lo = __floats2bfloat162_rn(r[0], r[1]), hi = __floats2bfloat162_rn(r[2], r[3]);
@@ -560,14 +580,14 @@ extern "C" int tllm_diff_combine(const float* a, const float* lq1, const float* 
 }
 
 extern "C" int tllm_embedding(const int* tokens, const void* table, float* out, int n_tokens, int hidden,
-                              int dtype, float scale, void* stream) {
+                              int dtype, float scale, float* twin, void* copy_bf16, void* stream) {
   TLLM_REQUIRE(n_tokens > 0 && hidden > 0, "embedding: empty input (%d tokens, width %d)", n_tokens, hidden);
   const int threads = hidden >= 1024 ? 256 : 128;
   cudaStream_t s = (cudaStream_t)stream;
   if (dtype == TLLM_F32)
-    TLLM_LAUNCH("embedding", embedding_kernel<float>, n_tokens, threads, 0, s, tokens, (const float*)table, out, n_tokens, hidden, scale);
+    TLLM_LAUNCH("embedding", embedding_kernel<float>, n_tokens, threads, 0, s, tokens, (const float*)table, out, n_tokens, hidden, scale, twin, (__nv_bfloat16*)copy_bf16);
   else if (dtype == TLLM_BF16)
-    TLLM_LAUNCH("embedding", embedding_kernel<__nv_bfloat16>, n_tokens, threads, 0, s, tokens, (const __nv_bfloat16*)table, out, n_tokens, hidden, scale);
+    TLLM_LAUNCH("embedding", embedding_kernel<__nv_bfloat16>, n_tokens, threads, 0, s, tokens, (const __nv_bfloat16*)table, out, n_tokens, hidden, scale, twin, (__nv_bfloat16*)copy_bf16);
   else
     TLLM_FAIL(TLLM_ERR_ARG, "embedding: unknown dtype code %d", dtype);
   return TLLM_OK;
@@ -619,9 +639,10 @@ extern "C" int tllm_rms_norm_add(float* x, const float* w, float* resid, int n_r
 // in_dtype: dtype of `gu`; out_dtype: dtype of `out`.  zero_src != 0 (float32 `gu` only): `gu` is a
 // split-K accumulation buffer and is handed back cleared.
 extern "C" int tllm_silu_mul(void* gu, void* out, int m, int inter, int blk, int in_dtype, int out_dtype, int zero_src,
-                             int act, void* stream) {
+                             int act, float limit, void* stream) {
   TLLM_REQUIRE(m > 0 && inter > 0 && blk > 0 && inter % blk == 0,
                "silu_mul: %d rows, width %d, block %d (the block must divide the width)", m, inter, blk);
+  TLLM_REQUIRE(act >= 0 && act <= 2 && (act != 2 || limit > 0.f), "silu_mul: activation code %d, limit %g", act, (double)limit);
   const size_t total = (size_t)m * inter;
   const int threads = 256;
   const int blocks = (int)((total + threads - 1) / threads < 148 * 16 ? (total + threads - 1) / threads : 148 * 16);
@@ -629,22 +650,22 @@ extern "C" int tllm_silu_mul(void* gu, void* out, int m, int inter, int blk, int
   if (in_dtype == TLLM_F32 && blk % 4 == 0 && ((uintptr_t)gu % 16) == 0 && ((uintptr_t)out % 16) == 0 && (out_dtype == TLLM_F32 || out_dtype == TLLM_BF16)) {
     const size_t quads = total / 4;
     const int vblocks = (int)((quads + threads - 1) / threads < 148 * 16 ? (quads + threads - 1) / threads : 148 * 16);
-    if (out_dtype == TLLM_F32 && zero_src) TLLM_LAUNCH("silu_mul", (silu_mul_f32x4_kernel<float, true>), vblocks, threads, 0, s, (float*)gu, (float*)out, m, inter, blk, act);
-    else if (out_dtype == TLLM_F32) TLLM_LAUNCH("silu_mul", (silu_mul_f32x4_kernel<float, false>), vblocks, threads, 0, s, (float*)gu, (float*)out, m, inter, blk, act);
-    else if (zero_src) TLLM_LAUNCH("silu_mul", (silu_mul_f32x4_kernel<__nv_bfloat16, true>), vblocks, threads, 0, s, (float*)gu, (__nv_bfloat16*)out, m, inter, blk, act);
-    else TLLM_LAUNCH("silu_mul", (silu_mul_f32x4_kernel<__nv_bfloat16, false>), vblocks, threads, 0, s, (float*)gu, (__nv_bfloat16*)out, m, inter, blk, act);
+    if (out_dtype == TLLM_F32 && zero_src) TLLM_LAUNCH("silu_mul", (silu_mul_f32x4_kernel<float, true>), vblocks, threads, 0, s, (float*)gu, (float*)out, m, inter, blk, act, limit);
+    else if (out_dtype == TLLM_F32) TLLM_LAUNCH("silu_mul", (silu_mul_f32x4_kernel<float, false>), vblocks, threads, 0, s, (float*)gu, (float*)out, m, inter, blk, act, limit);
+    else if (zero_src) TLLM_LAUNCH("silu_mul", (silu_mul_f32x4_kernel<__nv_bfloat16, true>), vblocks, threads, 0, s, (float*)gu, (__nv_bfloat16*)out, m, inter, blk, act, limit);
+    else TLLM_LAUNCH("silu_mul", (silu_mul_f32x4_kernel<__nv_bfloat16, false>), vblocks, threads, 0, s, (float*)gu, (__nv_bfloat16*)out, m, inter, blk, act, limit);
     return TLLM_OK;
   }
   if (in_dtype == TLLM_F32 && out_dtype == TLLM_F32 && !zero_src)
-    TLLM_LAUNCH("silu_mul", (silu_mul_kernel<float, float, false>), blocks, threads, 0, s, (float*)gu, (float*)out, m, inter, blk, act);
+    TLLM_LAUNCH("silu_mul", (silu_mul_kernel<float, float, false>), blocks, threads, 0, s, (float*)gu, (float*)out, m, inter, blk, act, limit);
   else if (in_dtype == TLLM_BF16 && out_dtype == TLLM_BF16 && !zero_src)
-    TLLM_LAUNCH("silu_mul", (silu_mul_kernel<__nv_bfloat16, __nv_bfloat16, false>), blocks, threads, 0, s, (__nv_bfloat16*)gu, (__nv_bfloat16*)out, m, inter, blk, act);
+    TLLM_LAUNCH("silu_mul", (silu_mul_kernel<__nv_bfloat16, __nv_bfloat16, false>), blocks, threads, 0, s, (__nv_bfloat16*)gu, (__nv_bfloat16*)out, m, inter, blk, act, limit);
   else if (in_dtype == TLLM_F32 && out_dtype == TLLM_BF16 && zero_src)
-    TLLM_LAUNCH("silu_mul", (silu_mul_kernel<float, __nv_bfloat16, true>), blocks, threads, 0, s, (float*)gu, (__nv_bfloat16*)out, m, inter, blk, act);
+    TLLM_LAUNCH("silu_mul", (silu_mul_kernel<float, __nv_bfloat16, true>), blocks, threads, 0, s, (float*)gu, (__nv_bfloat16*)out, m, inter, blk, act, limit);
   else if (in_dtype == TLLM_F32 && out_dtype == TLLM_BF16 && !zero_src)
-    TLLM_LAUNCH("silu_mul", (silu_mul_kernel<float, __nv_bfloat16, false>), blocks, threads, 0, s, (float*)gu, (__nv_bfloat16*)out, m, inter, blk, act);
+    TLLM_LAUNCH("silu_mul", (silu_mul_kernel<float, __nv_bfloat16, false>), blocks, threads, 0, s, (float*)gu, (__nv_bfloat16*)out, m, inter, blk, act, limit);
   else if (in_dtype == TLLM_F32 && out_dtype == TLLM_F32 && zero_src)
-    TLLM_LAUNCH("silu_mul", (silu_mul_kernel<float, float, true>), blocks, threads, 0, s, (float*)gu, (float*)out, m, inter, blk, act);
+    TLLM_LAUNCH("silu_mul", (silu_mul_kernel<float, float, true>), blocks, threads, 0, s, (float*)gu, (float*)out, m, inter, blk, act, limit);
   else
     TLLM_FAIL(TLLM_ERR_ARG, "silu_mul: dtype codes %d -> %d with zero_src %d are not built", in_dtype, out_dtype, zero_src);
   return TLLM_OK;

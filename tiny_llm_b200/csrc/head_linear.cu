@@ -1,5 +1,6 @@
 // One small product per head in one launch:
 //   out[t, h * o_hs + n] = sum_k a[t, h * a_hs + k] * w[h, n, k]        t < T, h < heads, n < N, k < K
+// and, with a gate, out times sigmoid(gate[t, h * g_hs + n]) in 32-bit before the one rounding.
 // `a` and `out` are rows of tokens whose heads lie side by side (any row stride, any distance between heads), `w` is
 // [heads, N, K] with rows contiguous.  It serves projections that differ from head to head and are too small to be
 // worth a launch each: a latent attention's queries into the latent's space and its values out of it.
@@ -29,7 +30,16 @@ struct HeadLinearArgs {
   long long o_ld;
   int o_hs;
   int tokens, heads, n, k;
+  const void* gate;    // null, or rows of a's type: one gate per output
+  long long g_ld;
+  int g_hs;
 };
+
+template <typename T>
+__device__ __forceinline__ float gated(const HeadLinearArgs& p, float v, int row, int h, int n) {
+  if (p.gate == nullptr) return v;
+  return v / (1.f + expf(-to_f32(((const T*)p.gate)[(size_t)row * p.g_ld + (size_t)h * p.g_hs + n])));
+}
 
 __device__ __forceinline__ void mma_bf16_16816(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
   asm volatile(
@@ -85,8 +95,8 @@ __global__ void __launch_bounds__(128) head_linear_mma_kernel(HeadLinearArgs p) 
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       if (n + i >= p.n) continue;
-      if (lo_ok) out[(size_t)r_lo * p.o_ld + n + i] = from_f32<TO>(acc[j][i]);
-      if (hi_ok) out[(size_t)r_hi * p.o_ld + n + i] = from_f32<TO>(acc[j][2 + i]);
+      if (lo_ok) out[(size_t)r_lo * p.o_ld + n + i] = from_f32<TO>(gated<__nv_bfloat16>(p, acc[j][i], r_lo, h, n + i));
+      if (hi_ok) out[(size_t)r_hi * p.o_ld + n + i] = from_f32<TO>(gated<__nv_bfloat16>(p, acc[j][2 + i], r_hi, h, n + i));
     }
   }
 }
@@ -126,7 +136,7 @@ __global__ void __launch_bounds__(256) head_linear_simt_kernel(HeadLinearArgs p)
 #pragma unroll
   for (int j = 0; j < 4; ++j) {
     const int r = row0 + tq * 4 + j;
-    if (r < p.tokens) out[(size_t)r * p.o_ld + n0 + nl] = from_f32<TO>(acc[j]);
+    if (r < p.tokens) out[(size_t)r * p.o_ld + n0 + nl] = from_f32<TO>(gated<T>(p, acc[j], r, h, n0 + nl));
   }
 }
 
@@ -137,15 +147,15 @@ using namespace tllm;
 // dtype: of a and w; out_dtype: of out (the same, or float32).  tensor_cores != 0 lets bfloat16 inputs whose sizes
 // allow it take the mma.sync kernel.
 extern "C" int tllm_head_linear(const void* a, long long a_ld, int a_hs, const void* w, void* out, long long o_ld, int o_hs,
-                                int tokens, int heads, int n, int k, int dtype, int out_dtype, int tensor_cores,
-                                void* stream) {
+                                int tokens, int heads, int n, int k, const void* gate, long long g_ld, int g_hs, int dtype,
+                                int out_dtype, int tensor_cores, void* stream) {
   TLLM_REQUIRE(tokens > 0 && heads > 0 && heads <= 65535 && n > 0 && k > 0 && a && w && out,
                "head_linear: %d tokens, %d heads, %d outputs of %d inputs", tokens, heads, n, k);
   TLLM_REQUIRE((dtype == TLLM_F32 || dtype == TLLM_BF16) && (out_dtype == dtype || out_dtype == TLLM_F32),
                "head_linear: dtype codes %d -> %d", dtype, out_dtype);
   HeadLinearArgs p;
   p.a = a; p.a_ld = a_ld; p.a_hs = a_hs; p.w = w; p.out = out; p.o_ld = o_ld; p.o_hs = o_hs;
-  p.tokens = tokens; p.heads = heads; p.n = n; p.k = k;
+  p.tokens = tokens; p.heads = heads; p.n = n; p.k = k; p.gate = gate; p.g_ld = g_ld; p.g_hs = g_hs;
   cudaStream_t s = (cudaStream_t)stream;
   const bool mma = tensor_cores && dtype == TLLM_BF16 && k % 2 == 0 && a_ld % 2 == 0 && a_hs % 2 == 0 &&
                    ((uintptr_t)a % 4) == 0 && ((uintptr_t)w % 4) == 0;

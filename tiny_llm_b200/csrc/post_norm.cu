@@ -1,0 +1,263 @@
+// Layer norms of the 32-bit stream, on their own and behind a branch, and the depth average of a model whose layers read
+// a weighted sum of everything that came before them.  All float32; means and variances in two passes over values held
+// in registers or shared memory.
+//
+// layer_norm: out[r] = (x - mean) / sqrt(var + eps) * w + b with x = row rows[r] (or r), var the mean of the squared
+//   deviations, rounded once to the output's type.
+// post_norm_join: what a block does that norms the SUM of the stream and a branch (post-norm), one kernel per branch:
+//     y = n(alpha * x + branch + out_bias),   x <- y
+//   `branch` is a zeroed buffer that products added into and is handed back zeroed; `copy` receives the new stream in
+//   bfloat16 for the next branch to read.  With stages X_0 .. X_(n-1) (stage j of row r at stages + j * stage_stride +
+//   r * hidden) the row's result y is the next stage, stored behind them when `keep` says that a later layer reads it, and
+//   what goes on is the depth average
+//     x <- mix[0] X_0 + ... + mix[n-1] X_(n-1) + mix[n] y.
+//   The stages' sum does not wait for the row's statistics: its loads are in flight while they are taken.
+// depth_average: the same average behind a layer whose block does not norm the sum: x is the result, stored and averaged.
+// row_add: x[r, :] += bias.
+#include "common.cuh"
+
+TLLM_DEFINE_LAST_ERROR
+
+namespace tllm {
+
+struct JoinArgs {
+  float* branch;            // [rows, hidden]
+  float* x;                 // [rows, hidden]: the stream, in place
+  const float* out_bias;    // [hidden] or null
+  const float *w, *b;       // [hidden]
+  float alpha, eps;
+  __nv_bfloat16* copy;      // [rows, hidden] or null
+  float* stages;            // null: no depth average
+  long long stage_stride;
+  int n_stages, keep;
+  const float* mix;         // [n_stages + 1]
+  int n_rows, hidden;
+};
+
+__device__ __forceinline__ float4 fma4(float s, float4 v, float4 a) {
+  return make_float4(fmaf(s, v.x, a.x), fmaf(s, v.y, a.y), fmaf(s, v.z, a.z), fmaf(s, v.w, a.w));
+}
+
+// Rows in registers: hidden a multiple of 4, at most 4 * VEC * blockDim.
+template <int VEC>
+__global__ void post_norm_join_vec_kernel(JoinArgs a) {
+  __shared__ float scratch[33];
+  pdl_trigger();
+  const int n4 = a.hidden / 4, r = blockIdx.x;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 ob[VEC];   // constants of the model are read ahead of the wait
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    const int idx = threadIdx.x + i * blockDim.x;
+    ob[i] = a.out_bias != nullptr && idx < n4 ? __ldg(reinterpret_cast<const float4*>(a.out_bias) + idx) : zero;
+  }
+  pdl_wait();
+  if (r >= a.n_rows) return;
+  float4* br = reinterpret_cast<float4*>(a.branch + (size_t)r * a.hidden);
+  float4* xr = reinterpret_cast<float4*>(a.x + (size_t)r * a.hidden);
+  float4 z[VEC], acc[VEC];
+  float sum = 0.f;
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    const int idx = threadIdx.x + i * blockDim.x;
+    z[i] = zero;
+    if (idx < n4) {
+      const float4 v = br[idx];
+      z[i] = fma4(a.alpha, xr[idx], make_float4(v.x + ob[i].x, v.y + ob[i].y, v.z + ob[i].z, v.w + ob[i].w));
+      br[idx] = zero;
+    }
+    sum += (z[i].x + z[i].y) + (z[i].z + z[i].w);
+    acc[i] = zero;
+  }
+  if (a.stages != nullptr) {
+#pragma unroll 4
+    for (int j = 0; j < a.n_stages; ++j) {
+      const float4* st = reinterpret_cast<const float4*>(a.stages + j * a.stage_stride + (size_t)r * a.hidden);
+      const float m = a.mix[j];
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) {
+        const int idx = threadIdx.x + i * blockDim.x;
+        if (idx < n4) acc[i] = fma4(m, st[idx], acc[i]);
+      }
+    }
+  }
+  const float mean = block_sum(sum, scratch) / (float)a.hidden;
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    if (threadIdx.x + i * blockDim.x < n4) {
+      z[i] = make_float4(z[i].x - mean, z[i].y - mean, z[i].z - mean, z[i].w - mean);
+      ss += (z[i].x * z[i].x + z[i].y * z[i].y) + (z[i].z * z[i].z + z[i].w * z[i].w);
+    }
+  }
+  ss = block_sum(ss, scratch);
+  const float inv = 1.f / sqrtf(ss / (float)a.hidden + a.eps);
+  const float last = a.stages != nullptr ? a.mix[a.n_stages] : 0.f;
+  float4* own = a.stages != nullptr ? reinterpret_cast<float4*>(a.stages + a.n_stages * a.stage_stride + (size_t)r * a.hidden) : nullptr;
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    const int idx = threadIdx.x + i * blockDim.x;
+    if (idx >= n4) continue;
+    const float4 w = __ldg(reinterpret_cast<const float4*>(a.w) + idx), b = __ldg(reinterpret_cast<const float4*>(a.b) + idx);
+    float4 y = make_float4(fmaf(z[i].x * inv, w.x, b.x), fmaf(z[i].y * inv, w.y, b.y), fmaf(z[i].z * inv, w.z, b.z), fmaf(z[i].w * inv, w.w, b.w));
+    if (own != nullptr) {
+      if (a.keep) own[idx] = y;
+      y = fma4(last, y, acc[i]);
+    }
+    xr[idx] = y;
+    if (a.copy != nullptr) {
+      uint2 pk;
+      *reinterpret_cast<__nv_bfloat162*>(&pk.x) = __floats2bfloat162_rn(y.x, y.y);
+      *reinterpret_cast<__nv_bfloat162*>(&pk.y) = __floats2bfloat162_rn(y.z, y.w);
+      reinterpret_cast<uint2*>(a.copy + (size_t)r * a.hidden)[idx] = pk;
+    }
+  }
+}
+
+// Any width: the row waits in shared memory.
+__global__ void post_norm_join_kernel(JoinArgs a) {
+  extern __shared__ float row[];
+  __shared__ float scratch[33];
+  pdl_trigger();
+  pdl_wait();
+  const int r = blockIdx.x;
+  if (r >= a.n_rows) return;
+  float* br = a.branch + (size_t)r * a.hidden;
+  float* xr = a.x + (size_t)r * a.hidden;
+  float sum = 0.f;
+  for (int i = threadIdx.x; i < a.hidden; i += blockDim.x) {   // a thread meets the same elements in every pass
+    const float z = fmaf(a.alpha, xr[i], br[i] + (a.out_bias ? a.out_bias[i] : 0.f));
+    br[i] = 0.f;
+    row[i] = z;
+    sum += z;
+  }
+  const float mean = block_sum(sum, scratch) / (float)a.hidden;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < a.hidden; i += blockDim.x) {
+    const float d = row[i] - mean;
+    row[i] = d;
+    ss += d * d;
+  }
+  ss = block_sum(ss, scratch);
+  const float inv = 1.f / sqrtf(ss / (float)a.hidden + a.eps);
+  for (int i = threadIdx.x; i < a.hidden; i += blockDim.x) {
+    float y = fmaf(row[i] * inv, a.w[i], a.b[i]);
+    if (a.stages != nullptr) {
+      float acc = 0.f;
+      for (int j = 0; j < a.n_stages; ++j) acc = fmaf(a.mix[j], a.stages[j * a.stage_stride + (size_t)r * a.hidden + i], acc);
+      if (a.keep) a.stages[a.n_stages * a.stage_stride + (size_t)r * a.hidden + i] = y;
+      y = fmaf(a.mix[a.n_stages], y, acc);
+    }
+    xr[i] = y;
+    if (a.copy) a.copy[(size_t)r * a.hidden + i] = __float2bfloat16_rn(y);
+  }
+}
+
+template <typename T>
+__global__ void layer_norm_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ b,
+                                  T* __restrict__ out, const int* __restrict__ rows, int n_rows, int hidden, float eps) {
+  extern __shared__ float row[];
+  __shared__ float scratch[33];
+  pdl_trigger();
+  pdl_wait();
+  const int r = blockIdx.x;
+  if (r >= n_rows) return;
+  const float* src = x + (size_t)(rows ? rows[r] : r) * hidden;
+  float sum = 0.f;
+  for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+    row[i] = src[i];
+    sum += row[i];
+  }
+  const float mean = block_sum(sum, scratch) / (float)hidden;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+    const float d = row[i] - mean;
+    row[i] = d;
+    ss += d * d;
+  }
+  ss = block_sum(ss, scratch);
+  const float inv = 1.f / sqrtf(ss / (float)hidden + eps);
+  for (int i = threadIdx.x; i < hidden; i += blockDim.x) out[(size_t)r * hidden + i] = from_f32<T>(fmaf(row[i] * inv, w[i], b[i]));
+}
+
+__global__ void depth_average_kernel(float* __restrict__ x, float* __restrict__ stages, long long stage_stride, int n_stages,
+                                     int keep, const float* __restrict__ mix, long long n) {
+  pdl_trigger();
+  pdl_wait();
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+    const float y = x[i];
+    float acc = 0.f;
+    for (int j = 0; j < n_stages; ++j) acc = fmaf(mix[j], stages[j * stage_stride + i], acc);
+    if (keep) stages[n_stages * stage_stride + i] = y;
+    x[i] = fmaf(mix[n_stages], y, acc);
+  }
+}
+
+__global__ void row_add_kernel(float* __restrict__ x, const float* __restrict__ bias, long long n, int hidden) {
+  pdl_trigger();
+  pdl_wait();
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x)
+    x[i] += bias[i % hidden];
+}
+
+constexpr int MAX_WIDTH = (48 * 1024 - 256) / 4;   // values of a row that waits in shared memory beside the sums' scratch
+
+}  // namespace tllm
+
+using namespace tllm;
+
+extern "C" int tllm_post_norm_join(float* branch, float* x, const float* out_bias, const float* w, const float* b, float alpha,
+                                   float eps, void* copy_bf16, float* stages, long long stage_stride, int n_stages, int keep,
+                                   const float* mix, int n_rows, int hidden, void* stream) {
+  TLLM_REQUIRE(n_rows > 0 && hidden > 0 && branch && x && w && b, "post_norm_join: %d rows of %d values", n_rows, hidden);
+  TLLM_REQUIRE(stages == nullptr || (mix != nullptr && n_stages >= 0), "post_norm_join: a depth average of %d stages needs weights", n_stages);
+  JoinArgs a;
+  a.branch = branch; a.x = x; a.out_bias = out_bias; a.w = w; a.b = b; a.alpha = alpha; a.eps = eps;
+  a.copy = (__nv_bfloat16*)copy_bf16; a.stages = stages; a.stage_stride = stage_stride; a.n_stages = n_stages; a.keep = keep;
+  a.mix = mix; a.n_rows = n_rows; a.hidden = hidden;
+  cudaStream_t s = (cudaStream_t)stream;
+  const auto off = [](const void* p, int to) { return ((uintptr_t)p % to) != 0; };
+  if (hidden % 4 == 0 && hidden <= 4 * 4 * 512 && !off(branch, 16) && !off(x, 16) && !off(out_bias, 16) && !off(w, 16) && !off(b, 16) &&
+      !off(copy_bf16, 8) && !off(stages, 16) && stage_stride % 4 == 0) {
+    // the threads depend on the width alone, so that a row's sums have the same order in every batch
+    const int n4 = hidden / 4;
+    const int threads = n4 <= 128 ? (n4 + 31) / 32 * 32 : (n4 <= 512 ? 256 : 512);
+    const int vec = (n4 + threads - 1) / threads;
+    if (vec <= 1) TLLM_LAUNCH("post_norm_join", post_norm_join_vec_kernel<1>, n_rows, threads, 0, s, a);
+    else if (vec == 2) TLLM_LAUNCH("post_norm_join", post_norm_join_vec_kernel<2>, n_rows, threads, 0, s, a);
+    else TLLM_LAUNCH("post_norm_join", post_norm_join_vec_kernel<4>, n_rows, threads, 0, s, a);
+    return TLLM_OK;
+  }
+  TLLM_REQUIRE(hidden <= MAX_WIDTH, "post_norm_join: rows of %d values (at most %d)", hidden, MAX_WIDTH);
+  const int threads = hidden >= 2048 ? 512 : (hidden >= 512 ? 256 : 128);
+  TLLM_LAUNCH("post_norm_join", post_norm_join_kernel, n_rows, threads, hidden * 4, s, a);
+  return TLLM_OK;
+}
+
+extern "C" int tllm_layer_norm(const float* x, const float* w, const float* b, void* out, const int* rows, int n_rows,
+                               int hidden, float eps, int out_dtype, void* stream) {
+  TLLM_REQUIRE(n_rows > 0 && hidden > 0 && hidden <= MAX_WIDTH, "layer_norm: %d rows of %d values (at most %d)", n_rows, hidden, MAX_WIDTH);
+  const int threads = hidden >= 2048 ? 512 : (hidden >= 512 ? 256 : 128);
+  cudaStream_t s = (cudaStream_t)stream;
+  if (out_dtype == TLLM_F32) TLLM_LAUNCH("layer_norm", layer_norm_kernel<float>, n_rows, threads, hidden * 4, s, x, w, b, (float*)out, rows, n_rows, hidden, eps);
+  else if (out_dtype == TLLM_BF16) TLLM_LAUNCH("layer_norm", layer_norm_kernel<__nv_bfloat16>, n_rows, threads, hidden * 4, s, x, w, b, (__nv_bfloat16*)out, rows, n_rows, hidden, eps);
+  else TLLM_FAIL(TLLM_ERR_ARG, "layer_norm: unknown dtype code %d", out_dtype);
+  return TLLM_OK;
+}
+
+extern "C" int tllm_depth_average(float* x, float* stages, long long stage_stride, int n_stages, int keep, const float* mix,
+                                  long long n, void* stream) {
+  TLLM_REQUIRE(n > 0 && n_stages >= 0 && x && stages && mix, "depth_average: %lld values, %d stages", n, n_stages);
+  const int threads = 256;
+  const long long want = (n + threads - 1) / threads;
+  TLLM_LAUNCH("depth_average", depth_average_kernel, (unsigned)(want < 148 * 16 ? want : 148 * 16), threads, 0, (cudaStream_t)stream, x, stages, stage_stride, n_stages, keep, mix, n);
+  return TLLM_OK;
+}
+
+extern "C" int tllm_row_add(float* x, const float* bias, long long n_rows, int hidden, void* stream) {
+  TLLM_REQUIRE(n_rows > 0 && hidden > 0 && x && bias, "row_add: %lld rows of %d values", n_rows, hidden);
+  const int threads = 256;
+  const long long n = n_rows * hidden, want = (n + threads - 1) / threads;
+  TLLM_LAUNCH("row_add", row_add_kernel, (unsigned)(want < 148 * 16 ? want : 148 * 16), threads, 0, (cudaStream_t)stream, x, bias, n, hidden);
+  return TLLM_OK;
+}

@@ -98,9 +98,10 @@ class Scheduler:
         for g in self.cache.groups:
             # the fewest tokens the request must be able to hold pages for: all of them, or, in a group
             # with a window, the window and the token being written, rounded out to whole pages at both
-            # ends (pages behind the window come back only after the step that passed them)
+            # ends (pages behind the window come back only after the step that passed them), and the pages of
+            # the first positions that a window keeps
             reach = min(x for x in (g.need.window, g.need.chunk, total) if x is not None)
-            most = total if not g.need.bounded else min(total, reach + 2 * g.page_size)
+            most = total if not g.need.bounded else min(total, reach + (2 + g.kept_pages) * g.page_size)
             if g.pages_for(most) > g.pool.num_pages:
                 raise RequestRefused(f"request {request.rid!r}: {most} tokens need {g.pages_for(most)} pages, "
                                      f"the pool has {g.pool.num_pages}")

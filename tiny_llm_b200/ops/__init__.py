@@ -127,10 +127,15 @@ def trace_dump():
 
 
 def embedding(tokens: torch.Tensor, table: torch.Tensor, out: torch.Tensor, accumulate: bool = False,
-              scale: float = 1.0) -> None:
+              scale: float = 1.0, twin: Optional[torch.Tensor] = None, copy: Optional[torch.Tensor] = None) -> None:
     """out[t, :] = table[tokens[t], :] * scale as float32 (the residual stream is 32-bit; the product is taken in
-    32-bit); accumulate=True adds the rows into `out` instead (unscaled)."""
-    _need_cuda(tokens, table, out)
+    32-bit); accumulate=True adds the rows into `out` instead (unscaled).  `twin` (float32) and `copy` (bfloat16), of
+    out's shape: also receive the rows, for a model that comes back to them and for a first layer that reads the
+    stream itself."""
+    _need_cuda(tokens, table, out, twin, copy)
+    for other, dt in ((twin, torch.float32), (copy, torch.bfloat16)):
+        if other is not None and (accumulate or other.dtype != dt or other.shape != out.shape or not other.is_contiguous()):
+            raise KernelError("embedding: a further output has the rows' shape, float32 (twin) or bfloat16 (copy)")
     _i32(tokens, "tokens")
     t, h = out.shape
     if out.dtype != torch.float32 or not out.is_contiguous() or not table.is_contiguous() or table.shape[1] != h \
@@ -143,7 +148,7 @@ def embedding(tokens: torch.Tensor, table: torch.Tensor, out: torch.Tensor, accu
         _call(lib, lib.tllm_embedding_add, _ptr(tokens), _ptr(table), _ptr(out), t, h, _code(table.dtype), _stream())
         return
     _call(lib, lib.tllm_embedding, _ptr(tokens), _ptr(table), _ptr(out), t, h, _code(table.dtype), ctypes.c_float(scale),
-          _stream())
+          _ptr(twin), _ptr(copy), _stream())
 
 
 def rms_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
@@ -257,11 +262,15 @@ def min_gru_scan(zug: torch.Tensor, bias_z: torch.Tensor, bias_u: torch.Tensor, 
           _ptr(summary), _code(zug.dtype), _stream())
 
 
-GLU_ACTS = {"silu": 0, "relu": 1}
+# what a gated feed-forward makes of gate and up: silu(g) u, relu(g) u, or the clamped form
+# min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u, -limit, limit) + 1)
+GLU_ACTS = {"silu": 0, "relu": 1, "clamped": 2}
 
 
-def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, block: int, consume: bool = False, act: str = "silu") -> None:
-    """out[m, g*block + j] = act(gate_up[m, 2*g*block + j]) * gate_up[m, 2*g*block + block + j], act = silu or relu.
+def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, block: int, consume: bool = False, act: str = "silu",
+             limit: float = 0.0) -> None:
+    """out[m, g*block + j] = act(gate_up[m, 2*g*block + j]) * gate_up[m, 2*g*block + block + j], act one of GLU_ACTS
+    (`limit` belongs to "clamped").
     `gate_up` is of out's dtype or float32 (a product's 32-bit sums).  consume=True: `gate_up` is a float32
     accumulation buffer (split-K sums) and is handed back zeroed."""
     _need_cuda(gate_up, out)
@@ -273,7 +282,7 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, block: int, consume: bool
     if act not in GLU_ACTS:
         raise KernelError(f"silu_mul: unknown activation {act!r} (known: {', '.join(GLU_ACTS)})")
     _call(lib, lib.tllm_silu_mul, _ptr(gate_up), _ptr(out), m, inter, block, _code(gate_up.dtype), _code(out.dtype),
-                                  1 if consume else 0, GLU_ACTS[act], _stream())
+                                  1 if consume else 0, GLU_ACTS[act], ctypes.c_float(limit), _stream())
 
 
 def rope_kv_write(qkv: torch.Tensor, positions: torch.Tensor, cos: Optional[torch.Tensor],
@@ -723,11 +732,11 @@ def qk_norm_kv_write(proj: torch.Tensor, positions: torch.Tensor, num_heads: int
 def latent_kv_write(proj: torch.Tensor, positions: torch.Tensor, num_heads: int, plain_dim: int, rot_part: int,
                     rank: int, rot_dims: int, freq: Optional[torch.Tensor], norm_weight: Optional[torch.Tensor], eps: float,
                     q_out: torch.Tensor, k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor],
-                    slot_mapping: Optional[torch.Tensor], rot_mag: float = 1.0) -> None:
+                    slot_mapping: Optional[torch.Tensor], rot_mag: float = 1.0, rot_pairs: bool = True) -> None:
     """Rows of `proj`: num_heads query heads of [plain_dim | rot_part] values, then `rank` latent values and rot_part
     key values shared by the heads.  The latent, normed with `norm_weight`, becomes the first `rank` values of the
     token's key row and its whole value row; the key's part and every query head's part are rotated pairwise (value
-    2i with 2i + 1, i < rot_dims / 2) by positions[t] * freq[i]; the key part is written behind the latent, the query
+    2i with 2i + 1, or, with rot_pairs=False, value i with i + rot_dims / 2; i < rot_dims / 2) by positions[t] * freq[i]; the key part is written behind the latent, the query
     parts to q_out[t, head, rank:] (q_out [T, num_heads, rank + rot_part]).  cos and sin are multiplied by rot_mag.
     Without caches (k_cache None) the rows hold the query heads only and only their parts are turned: the form of a
     mixer that reads what another layer cached."""
@@ -745,7 +754,7 @@ def latent_kv_write(proj: torch.Tensor, positions: torch.Tensor, num_heads: int,
         _call(lib, lib.tllm_latent_kv_write, _ptr(proj), proj.stride(0), num_heads, plain_dim, rot_part, rank, rot_dims,
               _ptr(None), _ptr(freq if rot_dims else None), ctypes.c_float(eps), _ptr(positions), _ptr(q_out),
               _ptr(None), _ptr(None), _ptr(None), 1, ctypes.c_longlong(0), ctypes.c_longlong(0), t,
-              ctypes.c_float(rot_mag), _code(proj.dtype), _stream())
+              ctypes.c_float(rot_mag), 1 if rot_pairs else 0, _code(proj.dtype), _stream())
         return
     if proj.stride(1) != 1 or proj.shape[1] < num_heads * (plain_dim + rot_part) + kd or \
             q_out.shape != (t, num_heads, kd) or not q_out.is_contiguous() or q_out.dtype != proj.dtype:
@@ -761,25 +770,72 @@ def latent_kv_write(proj: torch.Tensor, positions: torch.Tensor, num_heads: int,
     _call(lib, lib.tllm_latent_kv_write, _ptr(proj), proj.stride(0), num_heads, plain_dim, rot_part, rank, rot_dims,
           _ptr(norm_weight), _ptr(freq if rot_dims else None), ctypes.c_float(eps), _ptr(positions), _ptr(q_out),
           _ptr(k_cache), _ptr(v_cache), _ptr(slot_mapping), k_cache.shape[2], ll(k_cache.stride(0)), ll(v_cache.stride(0)),
-          t, ctypes.c_float(rot_mag), _code(proj.dtype), _stream())
+          t, ctypes.c_float(rot_mag), 1 if rot_pairs else 0, _code(proj.dtype), _stream())
 
 
-def head_linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
+def conv_norm_kv_write(proj: torch.Tensor, batch, num_heads: int, num_kv_heads: int, key_dim: int, value_dim: int,
+                       k_cache: torch.Tensor, v_cache: torch.Tensor, slot_mapping: torch.Tensor, q_out: torch.Tensor,
+                       bias: Optional[torch.Tensor] = None, taps: Optional[torch.Tensor] = None,
+                       kept: Optional[torch.Tensor] = None, norm_q: Optional[torch.Tensor] = None,
+                       norm_k: Optional[torch.Tensor] = None, eps: float = 0.0) -> None:
+    """Rows of `proj` begin with num_heads query heads and num_kv_heads key heads of key_dim values, then num_kv_heads
+    value heads of value_dim values.  With x = row + bias (float32 [channels]) every channel is filtered over time,
+    y_t = sum_j taps[:, j] x_(t - n + 1 + j) (taps float32 [channels, n], zeros before the sequence's start; the last
+    n - 1 inputs lie in kept[slot], float32 [slots, n - 1, channels], and are brought up to date); then all query values
+    of a token together become y / sqrt(mean(y^2) + eps) * norm_q (float32 [num_heads * key_dim]), and all its key values
+    the same with norm_k.  Queries go to q_out [T, num_heads * key_dim], keys and values to their pages; `proj` stays as
+    it is.  Without taps there is no filter, without norm weights no norm."""
+    _need_cuda(proj, k_cache, v_cache, slot_mapping, q_out, bias, taps, kept, norm_q, norm_k)
+    _i32(slot_mapping, "slot_mapping")
+    t = proj.shape[0]
+    nqc, nkc = num_heads * key_dim, num_kv_heads * key_dim
+    channels = nqc + nkc + num_kv_heads * value_dim
+    n = 1 if taps is None else taps.shape[1]
+    if proj.stride(1) != 1 or proj.shape[1] < channels or q_out.shape != (t, nqc) or not q_out.is_contiguous() or \
+            q_out.dtype != proj.dtype:
+        raise KernelError("conv_norm_kv_write: the rows of the projection or of the query buffer do not fit")
+    _paged("conv_norm_kv_write", k_cache, num_kv_heads, key_dim)
+    _paged("conv_norm_kv_write", v_cache, num_kv_heads, value_dim)
+    if k_cache.dtype != proj.dtype or v_cache.dtype != proj.dtype or k_cache.shape[2] != v_cache.shape[2]:
+        raise KernelError("conv_norm_kv_write: cache dtype or page size does not fit")
+    for name, b, shape in (("bias", bias, (channels,)), ("filter", taps, (channels, n)), ("query norm", norm_q, (nqc,)),
+                           ("key norm", norm_k, (nkc,))):
+        if b is not None and (b.dtype != torch.float32 or tuple(b.shape) != shape or not b.is_contiguous()):
+            raise KernelError(f"conv_norm_kv_write: the {name} must be contiguous float32 of shape {shape}")
+    if n > 1 and (kept is None or kept.dtype != torch.float32 or not kept.is_contiguous() or tuple(kept.shape[1:]) != (n - 1, channels)):
+        raise KernelError(f"conv_norm_kv_write: the kept inputs must be contiguous float32 [slots, {n - 1}, {channels}]")
+    single = batch.max_q_len == 1     # then the one token of a request also moves its kept inputs up
+    ll = ctypes.c_longlong
+    lib = build.load_library("attention_prep")
+    _call(lib, lib.tllm_conv_norm_kv_write, _ptr(proj), proj.stride(0), num_heads, num_kv_heads, key_dim, value_dim,
+          _ptr(bias), _ptr(taps), n, _ptr(kept if n > 1 else None), _ptr(batch.slots), _ptr(batch.cu_q), _ptr(batch.token_request),
+          _ptr(norm_q), _ptr(norm_k), ctypes.c_float(eps), _ptr(q_out), _ptr(k_cache), _ptr(v_cache), _ptr(slot_mapping),
+          k_cache.shape[2], ll(k_cache.stride(0)), ll(k_cache.stride(1)), ll(v_cache.stride(0)), ll(v_cache.stride(1)), t,
+          1 if single else 0, _code(proj.dtype), _stream())
+    if n > 1 and not single:
+        conv_state_update(proj, kept, batch, n, channels, bias=bias)
+
+
+def head_linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor] = None) -> None:
     """One small product per head in one launch: out[t, h, :] = w[h] . a[t, h, :].  a [T, heads, K] and out
     [T, heads, N] are views whose last dimension is contiguous (rows of tokens with the heads side by side, at any
     row stride and any distance between heads); w [heads, N, K] contiguous, of a's dtype; out of a's dtype or float32.
     bfloat16 with even K and even offsets runs on mma.sync tiles read straight from global memory, everything else
-    on FFMA tiles; either way an output's sum runs over ascending k whatever else is in the batch."""
-    _need_cuda(a, w, out)
+    on FFMA tiles; either way an output's sum runs over ascending k whatever else is in the batch.
+    `gate` [T, heads, N] (a view like the others, of a's dtype): the sums are multiplied by sigmoid(gate) in 32-bit."""
+    _need_cuda(a, w, out, gate)
     t, heads, k = a.shape
     n = w.shape[1]
     if w.shape != (heads, n, k) or not w.is_contiguous() or w.dtype != a.dtype or out.shape != (t, heads, n) or \
             a.stride(2) != 1 or out.stride(2) != 1 or out.dtype not in (a.dtype, torch.float32):
         raise KernelError("head_linear: shapes or dtypes do not fit")
+    if gate is not None and (gate.shape != (t, heads, n) or gate.dtype != a.dtype or gate.stride(2) != 1):
+        raise KernelError("head_linear: the gate does not fit")
     lib = build.load_library("head_linear")
     ll = ctypes.c_longlong
     _call(lib, lib.tllm_head_linear, _ptr(a), ll(a.stride(0)), a.stride(1), _ptr(w), _ptr(out), ll(out.stride(0)),
-          out.stride(1), t, heads, n, k, _code(a.dtype), _code(out.dtype), 0 if force_generic else 1, _stream())
+          out.stride(1), t, heads, n, k, _ptr(gate), ll(0 if gate is None else gate.stride(0)),
+          0 if gate is None else gate.stride(1), _code(a.dtype), _code(out.dtype), 0 if force_generic else 1, _stream())
 
 
 def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor, heads: int, value_dim: int, out: torch.Tensor) -> None:
@@ -844,16 +900,19 @@ def delta_prepare(proj: torch.Tensor, taps: torch.Tensor, kept: torch.Tensor, ba
           _code(proj.dtype), _stream())
 
 
-def conv_state_update(proj: torch.Tensor, kept: torch.Tensor, batch, n_taps: int, channels: int) -> None:
+def conv_state_update(proj: torch.Tensor, kept: torch.Tensor, batch, n_taps: int, channels: int,
+                      bias: Optional[torch.Tensor] = None) -> None:
     """kept[slot] <- the last n_taps - 1 inputs of every channel after the step's tokens (what was kept before moves
-    up when the step brought fewer tokens than that)."""
-    _need_cuda(proj, kept)
+    up when the step brought fewer tokens than that); with `bias` (float32 [channels]) an input is the projection plus it."""
+    _need_cuda(proj, kept, bias)
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != channels or not bias.is_contiguous()):
+        raise KernelError("conv_state_update: one contiguous float32 bias per channel")
     if proj.stride(1) != 1 or proj.shape[1] < channels or kept.dtype != torch.float32 or not kept.is_contiguous() or \
             tuple(kept.shape[1:]) != (max(n_taps - 1, 1), channels):
         raise KernelError("conv_state_update: shapes or dtypes do not fit")
     lib = build.load_library("delta_rule")
     _call(lib, lib.tllm_conv_state_update, _ptr(proj), proj.stride(0), _ptr(kept), _ptr(batch.slots), _ptr(batch.cu_q),
-          n_taps, channels, batch.num_requests, _code(proj.dtype), _stream())
+          n_taps, channels, batch.num_requests, _ptr(bias), _code(proj.dtype), _stream())
 
 
 def delta_rule_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gb: torch.Tensor, state: torch.Tensor, batch,
@@ -895,6 +954,73 @@ def bigram_add(tokens: torch.Tensor, table: torch.Tensor, last: torch.Tensor, ba
     _call(lib, lib.tllm_bigram_add, _ptr(tokens), _ptr(batch.token_request), _ptr(batch.cu_q), _ptr(batch.q_start),
           _ptr(batch.slots), _ptr(last), _ptr(table), _ptr(out), t, h, ll(table.shape[0] - 1), ll(mul_prev), ll(mul_cur),
           _code(table.dtype), _stream())
+
+
+def layer_norm(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, eps: float, out: torch.Tensor,
+               rows: Optional[torch.Tensor] = None) -> None:
+    """out[r, :] = (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps) * weight + bias with v = x[rows[r], :]; x, weight
+    and bias are float32."""
+    _need_cuda(x, weight, bias, out, rows)
+    _i32(rows, "rows")
+    h, n = x.shape[1], out.shape[0]
+    if any(v.dtype != torch.float32 or not v.is_contiguous() for v in (x, weight, bias)) or not out.is_contiguous() or \
+            out.shape[1] != h or weight.numel() != h or bias.numel() != h or \
+            (rows is None and n != x.shape[0]) or (rows is not None and rows.numel() != n):
+        raise KernelError("layer_norm: shapes or dtypes do not fit")
+    lib = build.load_library("post_norm")
+    _call(lib, lib.tllm_layer_norm, _ptr(x), _ptr(weight), _ptr(bias), _ptr(out), _ptr(rows), n, h, ctypes.c_float(eps),
+          _code(out.dtype), _stream())
+
+
+def _check_stages(name: str, x: torch.Tensor, stages: torch.Tensor, done: int, mix: torch.Tensor, keep: bool) -> None:
+    if stages.dtype != torch.float32 or not stages.is_contiguous() or tuple(stages.shape[1:]) != tuple(x.shape) or \
+            stages.shape[0] < done + (1 if keep else 0) or mix.dtype != torch.float32 or not mix.is_contiguous() or \
+            mix.numel() != done + 1:
+        raise KernelError(f"{name}: {done} stages of the stream's shape (and room for one more to keep) and {done + 1} weights")
+
+
+def post_norm_join(branch: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, eps: float,
+                   stream_scale: float = 1.0, out_bias: Optional[torch.Tensor] = None, copy: Optional[torch.Tensor] = None,
+                   stages: Optional[torch.Tensor] = None, done: int = 0, mix: Optional[torch.Tensor] = None,
+                   keep: bool = False) -> None:
+    """y = layer_norm(stream_scale * x + branch + out_bias) (weight, bias, eps), x <- y, row by row, all float32; `branch`
+    is handed back zeroed (products add into it) and `copy` (bfloat16) receives the new stream rounded.  With `stages`
+    (float32 [S, T, H], of which `done` hold earlier results) y becomes stages[done] when `keep` says so, and
+    x <- sum_(j < done) mix[j] stages[j] + mix[done] y."""
+    _need_cuda(branch, x, weight, bias, out_bias, copy, stages, mix)
+    h = x.shape[1]
+    if any(v.dtype != torch.float32 or not v.is_contiguous() for v in (branch, x, weight, bias)) or branch.shape != x.shape or \
+            weight.numel() != h or bias.numel() != h or \
+            (out_bias is not None and (out_bias.dtype != torch.float32 or out_bias.numel() != h or not out_bias.is_contiguous())) or \
+            (copy is not None and (copy.dtype != torch.bfloat16 or copy.shape != x.shape or not copy.is_contiguous())):
+        raise KernelError("post_norm_join: shapes or dtypes do not fit")
+    if stages is not None:
+        _check_stages("post_norm_join", x, stages, done, mix, keep)
+    lib = build.load_library("post_norm")
+    _call(lib, lib.tllm_post_norm_join, _ptr(branch), _ptr(x), _ptr(out_bias), _ptr(weight), _ptr(bias),
+          ctypes.c_float(stream_scale), ctypes.c_float(eps), _ptr(copy), _ptr(stages),
+          ctypes.c_longlong(0 if stages is None else stages.stride(0)), done, 1 if keep else 0, _ptr(mix), x.shape[0], h, _stream())
+
+
+def depth_average(x: torch.Tensor, stages: torch.Tensor, done: int, mix: torch.Tensor, keep: bool = False) -> None:
+    """x <- sum_(j < done) mix[j] stages[j] + mix[done] x, all float32; with `keep` the x that came in becomes stages[done]."""
+    _need_cuda(x, stages, mix)
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise KernelError("depth_average: the stream is contiguous float32")
+    _check_stages("depth_average", x, stages, done, mix, keep)
+    lib = build.load_library("post_norm")
+    _call(lib, lib.tllm_depth_average, _ptr(x), _ptr(stages), ctypes.c_longlong(stages.stride(0)), done, 1 if keep else 0,
+          _ptr(mix), ctypes.c_longlong(x.numel()), _stream())
+
+
+def row_add(x: torch.Tensor, bias: torch.Tensor) -> None:
+    """x[r, :] += bias, float32."""
+    _need_cuda(x, bias)
+    if x.dtype != torch.float32 or bias.dtype != torch.float32 or not x.is_contiguous() or not bias.is_contiguous() or \
+            bias.numel() != x.shape[1]:
+        raise KernelError("row_add: shapes or dtypes do not fit")
+    lib = build.load_library("post_norm")
+    _call(lib, lib.tllm_row_add, _ptr(x), _ptr(bias), ctypes.c_longlong(x.shape[0]), x.shape[1], _stream())
 
 
 UNARY_ACTS = {"copy": 0, "relu2": 1}
@@ -1209,8 +1335,8 @@ def linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate: bool
 
 
 def linear_swiglu(a: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, block: int, workspace,
-                  act: str = "silu") -> None:
-    """out = act(a Wg^T) * (a Wu^T) with Wg, Wu interleaved in `w_gate_up` in row blocks of `block`; act = silu or relu.
+                  act: str = "silu", limit: float = 0.0) -> None:
+    """out = act(a Wg^T) * (a Wu^T) with Wg, Wu interleaved in `w_gate_up` in row blocks of `block`; act one of GLU_ACTS.
     With blocks of 128 and more than 128 rows the product and SiLU*up are one tensor-core kernel (SiLU only: another
     activation takes the product and the element-wise kernel)."""
     m = a.shape[0]
@@ -1219,11 +1345,11 @@ def linear_swiglu(a: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, b
         if prefers_split(a, w_gate_up):
             acc = workspace.get_zeroed("gate_up_f32", (m, n2))
             linear(a, w_gate_up, acc, accumulate=True)
-            silu_mul(acc, out, block, consume=True, act=act)
+            silu_mul(acc, out, block, consume=True, act=act, limit=limit)
             return
         gu = workspace.get("gate_up", (m, n2), a.dtype)
         linear(a, w_gate_up, gu)
-        silu_mul(gu, out, block, act=act)
+        silu_mul(gu, out, block, act=act, limit=limit)
         return
     if _tc_ok(a, w_gate_up, out) and block == 128 and m > 128 and n2 % 256 == 0 and out.is_contiguous():
         _need_cuda(a, w_gate_up, out)
@@ -1416,13 +1542,18 @@ attention_maps_splits = int(os.environ.get("TLLM_ATTENTION_MAPS_SPLITS", "16"))
 def paged_attention_maps(qkv: torch.Tensor, num_heads: int, num_kv_heads: int, maps: int, key_dim: int, value_dim: int,
                          k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor, batch,
                          out: torch.Tensor, scale: float, window: Optional[int] = None,
-                         chunk: Optional[int] = None, sink: Optional[torch.Tensor] = None, workspace=None) -> None:
+                         chunk: Optional[int] = None, sink: Optional[torch.Tensor] = None, workspace=None,
+                         keep_first: int = 0, rel: Optional[torch.Tensor] = None,
+                         rel_log2: Optional[torch.Tensor] = None) -> None:
     """Attention with `maps` score maps per head over the same values, key rows of key_dim and value rows of
     value_dim values: query rows [head][map][key_dim] at the front of each `qkv` row, k_cache
     [pages, num_kv_heads * maps, page_size, key_dim], v_cache [pages, num_kv_heads, page_size, value_dim]; out
     [T, num_heads * maps * value_dim] in the cache's dtype or float32.  `chunk`: a key is visible only inside the
     query's chunk of that many positions (counted from position 0).  `sink` (float32 [num_heads]): a learned score
-    per head whose exponential joins the softmax's denominator; it stands for no key and has no value.
+    per head whose exponential joins the softmax's denominator; it stands for no key and has no value.  `keep_first`:
+    with a window, the sequence's first positions that stay visible to every later token.  `rel` (float32 [num_heads, n]):
+    rel[h, min(distance, n - 1)] is added to every scaled score of head h; `rel_log2` is the same table times log2(e)
+    (the tensor-core kernel's units; without it that kernel is not taken).
     `batch`: token_request and positions per token
     (the CUDA-core kernel); cu_q, q_start per request, num_requests, max_q_len (the tensor-core kernel).
     bfloat16 with a float32 output and sizes that are multiples of 16 runs on the tensor cores, everything else on
@@ -1433,6 +1564,13 @@ def paged_attention_maps(qkv: torch.Tensor, num_heads: int, num_kv_heads: int, m
     t = qkv.shape[0]
     if sink is not None and (sink.dtype != torch.float32 or sink.numel() != num_heads or not sink.is_contiguous()):
         raise KernelError("paged_attention_maps: the sink is one float32 per head")
+    _need_cuda(rel, rel_log2)
+    for tab in (rel, rel_log2):
+        if tab is not None and (rel is None or tab.dtype != torch.float32 or tab.dim() != 2 or tab.shape[0] != num_heads or
+                                tab.shape != rel.shape or not tab.is_contiguous()):
+            raise KernelError("paged_attention_maps: the distance bias is a contiguous float32 [heads, distances] table")
+    keep_first = int(keep_first) if window else 0
+    rel_len = 0 if rel is None else rel.shape[1]
     if out.shape != (t, num_heads * maps * value_dim) or not out.is_contiguous() or \
             out.dtype not in (qkv.dtype, torch.float32) or k_cache.dtype != qkv.dtype or v_cache.dtype != qkv.dtype or \
             k_cache.stride(3) != 1 or k_cache.stride(2) != key_dim or k_cache.shape[1] != num_kv_heads * maps or \
@@ -1441,13 +1579,13 @@ def paged_attention_maps(qkv: torch.Tensor, num_heads: int, num_kv_heads: int, m
         raise KernelError("paged_attention_maps: shapes or dtypes do not fit")
     few = getattr(batch, "max_q_len", 0) == 1 and t * num_heads * maps <= attention_maps_decode_pairs
     if qkv.dtype == torch.bfloat16 and out.dtype == torch.float32 and not force_generic and attention_maps_tc and \
-            not few and scale > 0 and key_dim % 16 == 0 and value_dim % 16 == 0 and 16 <= key_dim <= 256 and 16 <= value_dim <= 256 and \
+            (rel is None or rel_log2 is not None) and not few and scale > 0 and key_dim % 16 == 0 and value_dim % 16 == 0 and 16 <= key_dim <= 256 and 16 <= value_dim <= 256 and \
             qkv.stride(0) % 8 == 0 and qkv.data_ptr() % 16 == 0:
         # bfloat16: the tensor-core kernel compiled for this pair of sizes (prompt portions and decoded tokens alike)
         lib = build.load_library("attention_maps_mma", flags=(f"-DTLLM_HEAD_DIM={key_dim}", f"-DTLLM_VALUE_DIM={value_dim}"))
         splits, part = 1, None
         if workspace is not None and batch.max_q_len == 1 and attention_maps_splits > 1 and num_heads // num_kv_heads <= 64:
-            seen = batch.max_kv_len if not window else min(batch.max_kv_len, window + 64)
+            seen = batch.max_kv_len if not window else min(batch.max_kv_len, window + 64 + keep_first)
             if chunk:
                 seen = min(seen, chunk)
             ctas = batch.num_requests * num_kv_heads * maps
@@ -1460,7 +1598,7 @@ def paged_attention_maps(qkv: torch.Tensor, num_heads: int, num_kv_heads: int, m
               num_kv_heads, maps, key_dim, value_dim, k_cache.shape[2], ctypes.c_longlong(k_cache.stride(0)),
               ctypes.c_longlong(k_cache.stride(1)), ctypes.c_longlong(v_cache.stride(0)),
               ctypes.c_longlong(v_cache.stride(1)), ctypes.c_float(scale), int(window or 0), int(chunk or 0), _ptr(sink),
-              splits, _ptr(part), _stream())
+              splits, _ptr(part), keep_first, _ptr(rel_log2), rel_len, _stream())
         return
     lib = build.load_library("attention_generic")
     _call(lib, lib.tllm_paged_attention_maps,
@@ -1469,7 +1607,8 @@ def paged_attention_maps(qkv: torch.Tensor, num_heads: int, num_kv_heads: int, m
           value_dim, k_cache.shape[2], ctypes.c_longlong(k_cache.stride(0)), ctypes.c_longlong(k_cache.stride(1)),
           ctypes.c_longlong(v_cache.stride(0)), ctypes.c_longlong(v_cache.stride(1)), ctypes.c_float(scale),
           int(window or 0), int(chunk or 0), _code(qkv.dtype), 1 if out.dtype == torch.float32 else 0,
-          -1 if generic_attention_split is None else int(generic_attention_split), _ptr(sink), _stream())
+          -1 if generic_attention_split is None else int(generic_attention_split), _ptr(sink), keep_first, _ptr(rel), rel_len,
+          _stream())
 
 
 def attention_tc_timing(head_dim: int = 64) -> Optional[dict]:
@@ -1527,7 +1666,7 @@ def sample(logits: torch.Tensor, work: torch.Tensor, temperature: torch.Tensor, 
 
 
 ALL_LIBRARIES = ("elementwise", "linear_generic", "linear_tc", "attention_generic", "attention_prep", "recurrence",
-                 "linear_attention", "delta_rule", "head_linear", "window_attention", "attention_talk", "moe", "sampling")
+                 "linear_attention", "delta_rule", "head_linear", "window_attention", "attention_talk", "moe", "post_norm", "sampling")
 
 
 ATTENTION_HEAD_DIMS = (16, 32, 48, 64, 128)   # head sizes `build_all` compiles ahead; others compile on first use

@@ -49,6 +49,10 @@ class GQAttention:
     def cache_need(self):
         return None if self.shares_cache else KVNeed(self.num_kv_heads, self.head_dim, self.window)
 
+    def cache_reach(self):
+        """Which of the keys it reads this mixer can still see, for the owner of the cache."""
+        return KVNeed(self.num_kv_heads, self.head_dim, self.window)
+
     def weight_specs(self, prefix: str):
         specs = [WeightSpec(prefix + "q_proj.weight", (self.q_dim, self.hidden_size), COMPUTE)]
         if not self.shares_cache:

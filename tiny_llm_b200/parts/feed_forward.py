@@ -42,10 +42,15 @@ class SwiGLU:
 
     def __init__(self, hidden_size: int, intermediate_size: int,
                  names=("gate_proj.weight", "up_proj.weight", "down_proj.weight"), out_scale: float = 1.0,
-                 act: str = "silu"):
+                 act: str = "silu", limit: float = 0.0):
         """`names`: what the gate, up and down matrices are called behind the part's prefix.  `out_scale`: a
         constant the part's output is multiplied by; it is folded into the down matrix when that is loaded.
-        `act`: the gate's activation, "silu" or "relu" (m = (act(y Wg^T) * (y Wu^T)) Wd^T)."""
+        `act`: the gate's activation, "silu" or "relu" (m = (act(y Wg^T) * (y Wu^T)) Wd^T), or "clamped", which bounds
+        both sides by `limit`: with g = min(y Wg^T, limit) and u = clamp(y Wu^T, -limit, limit),
+        m = (g sigmoid(1.702 g) (u + 1)) Wd^T."""
+        if act == "clamped" and not limit > 0:
+            raise ValueError("a clamped feed-forward needs a positive limit")
+        self.limit = float(limit)
         if act not in ops.GLU_ACTS:
             raise ValueError(f"unknown gate activation {act!r}; known: {', '.join(ops.GLU_ACTS)}")
         self.act = act
@@ -71,7 +76,7 @@ class SwiGLU:
     def forward(self, ctx, h, resid) -> None:
         t = h.shape[0]
         act = ctx.workspace.get("ffn_act", (t, self.intermediate_size), ctx.dtype)
-        ops.linear_swiglu(h, self.w_gate_up, act, self.block, ctx.workspace, act=self.act)
+        ops.linear_swiglu(h, self.w_gate_up, act, self.block, ctx.workspace, act=self.act, limit=self.limit)
         ops.linear(act, self.w_down, resid, accumulate=True)
 
 

@@ -11,7 +11,8 @@ import torch
 
 from .. import ops
 from ..config.spec import LayerSpec, ModelSpec
-from ..weights import COMPUTE, WeightSpec
+from ..cache import KVNeed
+from ..weights import COMPUTE, FLOAT32, WeightSpec
 from .registry import build_block, build_part, register_block
 
 
@@ -196,6 +197,54 @@ class BranchNormBlock:
 register_block("branch_norm", BranchNormBlock)
 
 
+class PostNormBlock:
+    """The norm of the SUM: x <- norm1(s x + mixer(x)); x <- norm2(s x + ffn(x)), s the layer's `stream_scale`.  The
+    branches read the stream itself, as in the branch_norm block: the float32 engine hands them the stream, the bfloat16
+    engine the rounded copy that the kernel before left.  A branch adds its output into a zeroed float32 buffer; one kernel
+    adds the scaled stream (and an output bias that the mixer leaves to the block), norms the sum, hands the buffer back
+    zeroed and leaves the next branch's input.  Where the model averages its layers' results over the depth, the layer's
+    last norm does that on its way into the stream (`forward(..., depth=...)`)."""
+
+    leaves_stream_copy = True
+    averages_depth = True        # forward takes the model's depth average
+
+    def __init__(self, spec: LayerSpec, shares_cache: bool = False):
+        for role in ("norm1", "mixer"):
+            if getattr(spec, role) is None:
+                raise ValueError(f"layer {spec.prefix!r}: a post_norm block needs a {role}")
+        if (spec.ffn is None) != (spec.norm2 is None):
+            raise ValueError(f"layer {spec.prefix!r}: a post_norm block has a norm2 exactly when it has a feed-forward")
+        self.spec = spec
+        scale = {} if spec.residual_scale == 1.0 else {"out_scale": spec.residual_scale}
+        self.norm1 = build_part("norm", spec.norm1)
+        self.mixer = build_part("mixer", spec.mixer, **scale, **({"shares_cache": True} if shares_cache else {}))
+        self.norm2 = None if spec.ffn is None else build_part("norm", spec.norm2)
+        self.ffn = None if spec.ffn is None else build_part("ffn", spec.ffn, **scale)
+        if hasattr(self.mixer, "defer_out_bias"):
+            self.mixer.defer_out_bias = True
+
+    parts, _named = BranchNormBlock.parts, BranchNormBlock._named
+    weight_specs, load = BranchNormBlock.weight_specs, BranchNormBlock.load
+    _input = staticmethod(BranchNormBlock._input)
+
+    def _join(self, ctx, norm, branch, resid, out_bias=None, depth=None) -> None:
+        copy = None if ctx.dtype != torch.bfloat16 else ctx.workspace.get("stream_copy", tuple(resid.shape), ctx.dtype)
+        norm.join(ctx, branch, resid, self.spec.stream_scale, out_bias=out_bias, copy=copy, depth=depth)
+        ctx.stream_copy = None if copy is None else (resid.data_ptr(), copy)
+
+    def forward(self, ctx, resid, cache, depth=None) -> None:
+        branch = ctx.workspace.get_zeroed("branch_out", tuple(resid.shape))
+        self.mixer.forward(ctx, self._input(ctx, resid), branch, cache)
+        self._join(ctx, self.norm1, branch, resid, out_bias=getattr(self.mixer, "w_ob", None),
+                   depth=depth if self.ffn is None else None)
+        if self.ffn is not None:
+            self.ffn.forward(ctx, self._input(ctx, resid), branch)
+            self._join(ctx, self.norm2, branch, resid, depth=depth)
+
+
+register_block("post_norm", PostNormBlock)
+
+
 class DecoderModel:
     def __init__(self, spec: ModelSpec):
         self.spec = spec
@@ -210,6 +259,9 @@ class DecoderModel:
         if spec.after_embedding is not None and any(c.add_embedding for c in spec.order):
             raise ValueError("a run order that adds the embedding output again cannot be combined with a hook that "
                              "rewrites the stream after the embedding")
+        if spec.depth_average is not None and ([c.layer for c in spec.order] != list(range(len(spec.layers))) or
+                                               any(c.add_embedding for c in spec.order)):
+            raise ValueError("a depth average takes every layer once, in order, without the embedding output added again")
         shared = {c.layer for c in spec.order if c.reads_cache_of is not None}
         owning = {c.layer for c in spec.order if c.reads_cache_of is None}
         if shared & owning:
@@ -220,6 +272,7 @@ class DecoderModel:
         self.on_logits = None if spec.on_logits is None else build_part("hook", spec.on_logits)
         self._hook_keeps = self.after_embedding is not None and hasattr(self.after_embedding, "cache_need")
         self.embed = None
+        self.depth_weights = []      # per layer, when the model averages its results over the depth
         self.lm_head = None
         self.loaded = False
         # a callable(position in the run order, float32 stream [T, H]) called after every layer call: for tests and
@@ -236,6 +289,9 @@ class DecoderModel:
         specs = [WeightSpec(s.embed_name, (s.vocab_size, s.hidden_size), COMPUTE)]
         for b in self.blocks:
             specs += b.weight_specs()
+        if s.depth_average is not None:
+            specs += [WeightSpec(ls.prefix + s.depth_average, (i + 2,), FLOAT32, init=("uniform", -0.2, 0.8))
+                      for i, ls in enumerate(s.layers)]
         specs += self.final_norm.weight_specs(s.final_norm_name)
         if self.after_embedding is not None:
             specs += self.after_embedding.weight_specs(s.after_embedding_name)
@@ -257,6 +313,10 @@ class DecoderModel:
         def need(block):
             return None if block.mixer is None else block.mixer.cache_need()
         needs = [None if c.reads_cache_of is not None else need(self.blocks[c.layer]) for c in self.spec.order]
+        for c in self.spec.order:    # a cache holds its keys as long as the farthest-seeing of its readers needs them
+            reach = getattr(self.blocks[c.layer].mixer, "cache_reach", None)
+            if c.reads_cache_of is not None and reach is not None and isinstance(needs[c.reads_cache_of], KVNeed):
+                needs[c.reads_cache_of] = needs[c.reads_cache_of].reaching(reach())
         if self._hook_keeps:   # what the hook after the embedding keeps per request comes behind the layer calls' entries
             needs.append(self.after_embedding.cache_need())
         return needs
@@ -266,6 +326,8 @@ class DecoderModel:
         self.embed = weights[s.embed_name]
         for b in self.blocks:
             b.load(weights)
+        if s.depth_average is not None:
+            self.depth_weights = [weights[ls.prefix + s.depth_average] for ls in s.layers]
         self.final_norm.load(s.final_norm_name, weights)
         if self.after_embedding is not None:
             self.after_embedding.load(s.after_embedding_name, weights)
@@ -281,19 +343,40 @@ class DecoderModel:
         s = self.spec
         b = ctx.batch
         resid = ctx.workspace.get("resid", (b.num_tokens, s.hidden_size), torch.float32)
-        ops.embedding(b.tokens, self.embed, resid, scale=s.embedding_scale)
-        ctx.stream_copy = None     # a rounded copy of the stream that a block may leave for the next one
+        # what a depth average comes back to: the embedding output and every layer's result but the last's
+        stages = None if s.depth_average is None else \
+            ctx.workspace.get("depth_stages", (len(s.order), b.num_tokens, s.hidden_size), torch.float32)
+        copy = None
+        if ctx.dtype == torch.bfloat16 and getattr(self.blocks[s.order[0].layer], "leaves_stream_copy", False) and \
+                self.after_embedding is None:
+            copy = ctx.workspace.get("stream_copy", tuple(resid.shape), ctx.dtype)
+        ops.embedding(b.tokens, self.embed, resid, scale=s.embedding_scale, copy=copy,
+                      twin=None if stages is None or self.after_embedding is not None else stages[0])
+        # a rounded copy of the stream that a block may leave for the next one
+        ctx.stream_copy = None if copy is None else (resid.data_ptr(), copy)
         if self._hook_keeps:
             self.after_embedding.forward(ctx, resid, ctx.cache_view(len(s.order)))
         elif self.after_embedding is not None:
             self.after_embedding.forward(ctx, resid)
+        if stages is not None and self.after_embedding is not None:
+            ops.unary(resid, stages[0])
         for pos, call in enumerate(s.order):
             owner = pos if call.reads_cache_of is None else call.reads_cache_of
             if call.add_embedding:   # the embedding output is the table's rows again: gathered and added in one kernel
                 ops.embedding(b.tokens, self.embed, resid, accumulate=True)
                 ctx.stream_copy = None
-            self.blocks[call.layer].forward(ctx, resid, ctx.cache_view(owner))
-            if not getattr(self.blocks[call.layer], "leaves_stream_copy", False):
+            block = self.blocks[call.layer]
+            if stages is None:
+                block.forward(ctx, resid, ctx.cache_view(owner))
+            else:
+                depth = (stages, pos + 1, self.depth_weights[pos], pos + 1 < len(s.order))
+                if getattr(block, "averages_depth", False):
+                    block.forward(ctx, resid, ctx.cache_view(owner), depth=depth)
+                else:
+                    block.forward(ctx, resid, ctx.cache_view(owner))
+                    ops.depth_average(resid, *depth)
+                    ctx.stream_copy = None
+            if not getattr(block, "leaves_stream_copy", False):
                 ctx.stream_copy = None
             if self.probe is not None:
                 self.probe(pos, resid)

@@ -1,6 +1,6 @@
 """Norms.  RMSNorm: y_j = (w_j x_j) / sqrt(mean_j(x_j^2) + eps), statistics in 32-bit
 (tiny_llm/ops/cuda/norm.cu:16-49).  Any width; the reference stops at 2048.  With `one_plus` the stored weight lies
-around zero and the norm multiplies by 1 + w_j."""
+around zero and the norm multiplies by 1 + w_j.  LayerNorm: y_j = (x_j - mean) / sqrt(var + eps) w_j + b_j."""
 from __future__ import annotations
 
 from .. import ops
@@ -74,5 +74,38 @@ class DynamicTanh:
         return out
 
 
+class LayerNorm:
+    """y_j = (x_j - mean) / sqrt(mean((x - mean)^2) + eps) * w_j + b_j, all in 32-bit.  The weight is stored under the
+    part's own name, the bias beside it as `<name>.b`."""
+    graph_safe = True
+
+    def __init__(self, size: int, eps: float):
+        self.size, self.eps = size, float(eps)
+        self.weight = self.bias = None
+
+    def weight_specs(self, prefix: str):
+        return [WeightSpec(prefix, (self.size,), FLOAT32, init=("uniform", 0.5, 1.5)),
+                WeightSpec(prefix + ".b", (self.size,), FLOAT32, init=("normal", 0.2))]
+
+    def load(self, prefix: str, weights) -> None:
+        self.weight, self.bias = weights[prefix], weights[prefix + ".b"]
+
+    def join(self, ctx, branch, resid, stream_scale, out_bias=None, copy=None, depth=None) -> None:
+        """resid <- norm(stream_scale * resid + branch + out_bias): for a block that norms the sum.  `branch` is a zeroed
+        float32 buffer that products added into; it is handed back zeroed.  `copy` (bfloat16) also receives the new
+        stream, rounded.  `depth` (stages, how many hold results, weights, whether to keep this one): the result is
+        averaged with the earlier ones on its way into the stream."""
+        stages, done, mix, keep = depth if depth is not None else (None, 0, None, False)
+        ops.post_norm_join(branch, resid, self.weight, self.bias, self.eps, stream_scale, out_bias=out_bias, copy=copy,
+                           stages=stages, done=done, mix=mix, keep=keep)
+
+    def forward(self, ctx, x, rows=None):
+        n = x.shape[0] if rows is None else rows.shape[0]
+        out = ctx.workspace.get("norm_out", (n, self.size), ctx.dtype)
+        ops.layer_norm(x, self.weight, self.bias, self.eps, out, rows)
+        return out
+
+
 register_part("norm", "rms_norm", RMSNorm)
+register_part("norm", "layer_norm", LayerNorm)
 register_part("norm", "dynamic_tanh", DynamicTanh)

@@ -23,8 +23,11 @@ Interfaces (duck-typed; `ctx` is the step's StepContext):
 A block arranges a layer's parts.  `register_block(kind, factory)`; factory(layer_spec, shares_cache)
 returns an object with
             parts() -> every part it built (the model asks each whether its steps may be captured);
-            mixer (the part whose cache_need() the cache manager reads, or None);
+            mixer (the part whose cache_need() the cache manager reads, or None; a mixer that reads another call's
+            cache says with cache_reach() -> KVNeed how far back it looks);
             weight_specs() -> [WeightSpec]; load(weights); forward(ctx, resid_f32[T, H], cache).
+A block that sets `averages_depth` takes the model's depth average as forward(..., depth=(stages, done, weights, keep)) and
+leaves the averaged stream; behind any other block the model runs the average as a kernel of its own.
 `resid` passed to a mixer or ffn need not be the residual stream itself: a block that norms a branch
 before it joins the stream hands the part a zeroed float32 buffer and joins it itself.
 """

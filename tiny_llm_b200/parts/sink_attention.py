@@ -14,7 +14,13 @@ size may differ.  The gate has one value per output value, or one per head (`gat
 `head_temp` multiplies head h's scores by a learned number `temp`[h]; `talk` mixes the heads' scores before the softmax,
 z_h = sum_g talk[h, g] s_g with a learned heads x heads matrix.  With either of the last two the scores of all heads
 meet in one kernel (`ops.attention_talk`), which takes scale, temperatures and mixing as ONE matrix
-M[h, g] = talk[h, g] * temp[g] * scale (made in 32-bit at load).
+M[h, g] = talk[h, g] * temp[g] * scale (made in 32-bit at load).  `conv` > 0 passes every channel of q, k and v (projection
+plus bias) through a causal filter of that many taps before the norms; the last conv - 1 inputs of a request are state
+beside its keys and values.  `qk_norm="whole"` norms all query rows of a token at once, and all its key rows, with a
+weight per channel.  `bias_max` adds a learned bias `rel`[bucket(distance), head] to the scaled scores (`distance_buckets`;
+the number of buckets is the stored table's).  `keep_first` leaves the first positions visible to every token whatever
+the window.  `out_bias` adds `o.b` behind the output projection (a block that joins the branch itself takes it over:
+`defer_out_bias`).
 
 `LatentAttention`: keys and values of all heads are projections of ONE small latent vector per token,
     c = norm(first `rank` rows of Wdkv h),   k_h = [Wuk_h c | rot(last rows of Wdkv h)],   v_h = Wuv_h c,
@@ -22,8 +28,10 @@ and the queries are [plain | rotated] per head.  Only c and the rotated key part
 against the cache as it is: with q'_h = Wuk_h^T q_plain_h the score q_plain_h . (Wuk_h c) equals q'_h . c, so every
 head attends with the query [q'_h | q_rot_h] over one shared key row [c | k_rot] and one shared value row c, and the
 head's value projection is applied to the weighted sum of latents afterwards: o_h = Wuv_h (sum_j p_j c_j).  The rotated
-parts turn in pairs (2i, 2i + 1) by p * base^(-2i / rot_dims).  A key is visible while 0 <= i - j < window.  The gate
-has one value per head (`gate=False`: none).  Built with `shares_cache=True` (a run-order entry that reads another
+parts turn in pairs (2i, 2i + 1), or in halves (i, i + rot_dims / 2) with `rot_layout="halves"`, by
+p * base^(-2i / rot_dims).  A key is visible while 0 <= i - j < window.  The gate has one value per head, applied to the
+weighted sums of latents (`gate=False`: none), or with `gate="value"` one per output value, applied behind the value
+projection.  Built with `shares_cache=True` (a run-order entry that reads another
 entry's cache) the mixer has no Wdkv and no latent norm: it attends over the latents and rotated key parts that the
 other layer cached, with its own Wuk, Wuv, queries and sink."""
 from __future__ import annotations
@@ -34,7 +42,7 @@ from typing import Optional
 import torch
 
 from .. import ops
-from ..cache import KVNeed
+from ..cache import KVNeed, StateNeed
 from ..weights import COMPUTE, FLOAT32, WeightSpec
 from .feed_forward import scaled_matrix
 from .registry import register_part
@@ -70,6 +78,18 @@ def stretched_frequencies(dims: int, base: float, scaling: Optional[dict] = None
     return f.to(torch.float32).contiguous(), mag
 
 
+def distance_buckets(buckets: int, far: float):
+    """The bucket of every distance n = 0, 1, ... up to the first that falls into the last bucket (all beyond do): one
+    bucket per distance below buckets // 2 = h, then h + floor(ln(n / h) / ln(far / h) (buckets - h)), at most the last."""
+    h = buckets // 2
+    if h < 1 or far <= h:
+        raise ValueError(f"a distance bias of {buckets} buckets needs at least two, and a largest distance above {h} (found {far})")
+    out = list(range(h))
+    while out[-1] < buckets - 1:
+        out.append(min(buckets - 1, h + math.floor(math.log(len(out) / h) / math.log(far / h) * (buckets - h))))
+    return out
+
+
 def _padded(n: int) -> int:
     return -(-n // 8) * 8
 
@@ -81,7 +101,8 @@ class SinkAttention:
                  eps: float, bias: bool = True, qk_norm: bool = True, sink: bool = True, gate: bool = True,
                  stretch_coef: float = 0.0, stretch_every: int = 0, window: Optional[int] = None,
                  rot_dims: int = 0, rot_base: float = 10000.0, rot_scaling: Optional[dict] = None,
-                 rot_layout: str = "halves", head_temp: bool = False, talk: bool = False,
+                 rot_layout: str = "halves", head_temp: bool = False, talk: bool = False, conv: int = 0,
+                 bias_max: Optional[float] = None, keep_first: int = 0, out_bias: bool = False,
                  out_scale: float = 1.0, shares_cache: bool = False):
         if shares_cache:
             raise ValueError("this attention does not read another layer call's cache")
@@ -91,6 +112,18 @@ class SinkAttention:
             raise ValueError(f"{rot_dims} rotated values must be even and at most the key size {key_dim}; layouts: halves, pairs")
         if gate not in (True, False, "head"):
             raise ValueError(f"unknown gate kind {gate!r} (True: one per value, \"head\": one per head, False: none)")
+        if qk_norm not in (True, False, "whole"):
+            raise ValueError(f"unknown query/key norm {qk_norm!r} (True: per head, \"whole\": all heads at once, False: none)")
+        # filters and whole-row norms leave q, k, v through one kernel that knows neither rotations nor stretched queries
+        self.filtered = conv > 0 or qk_norm == "whole"
+        if self.filtered and (qk_norm is True or rot_dims or stretch_every):
+            raise ValueError("short filters and norms over all heads go without norms per head, rotations and stretched queries")
+        if (head_temp or talk) and (bias_max is not None or keep_first or self.filtered):
+            raise ValueError("mixed scores go without filters, distance biases and kept first positions")
+        self.conv, self.bias_max, self.out_bias = int(conv), bias_max, out_bias
+        self.keep_first = int(keep_first) if window is not None else 0
+        self.defer_out_bias = False     # set by a block that adds `w_ob` where it joins the branch
+        self.taps = self.w_ob = self.rel = self.rel_log2 = self.bias_row = None
         self.rot_dims, self.rot_base, self.rot_scaling, self.rot_layout = rot_dims, float(rot_base), rot_scaling, rot_layout
         self.head_temp, self.talk = head_temp, talk
         self.freq, self.rot_mag, self.mix, self.mix_log2 = None, 1.0, None, None
@@ -107,7 +140,10 @@ class SinkAttention:
         self.w_in = self.w_o = self.biases = self.norms = self.w_sink = None
 
     def cache_need(self):
-        return KVNeed(self.num_kv_heads, self.key_dim, self.window, value_dim=self.value_dim)
+        kv = KVNeed(self.num_kv_heads, self.key_dim, self.window, value_dim=self.value_dim, keep_first=self.keep_first)
+        if self.conv > 1:
+            return kv, StateNeed((self.conv - 1, self.q_dim + self.k_dim + self.v_dim), torch.float32)
+        return kv
 
     def weight_specs(self, prefix: str):
         h = self.hidden_size
@@ -116,7 +152,10 @@ class SinkAttention:
         if self.bias:
             specs += [WeightSpec(prefix + n + ".b", (d,), FLOAT32, init=("normal", 0.3))
                       for n, d in (("q", self.q_dim), ("k", self.k_dim), ("v", self.v_dim))]
-        if self.qk_norm:
+        if self.qk_norm == "whole":
+            specs += [WeightSpec(prefix + "q.norm", (self.q_dim,), FLOAT32, init=("uniform", 0.5, 1.5)),
+                      WeightSpec(prefix + "k.norm", (self.k_dim,), FLOAT32, init=("uniform", 0.5, 1.5))]
+        elif self.qk_norm:
             specs += [WeightSpec(prefix + "q.norm", (self.key_dim,), FLOAT32, init=("uniform", 0.5, 1.5)),
                       WeightSpec(prefix + "k.norm", (self.key_dim,), FLOAT32, init=("uniform", 0.5, 1.5))]
         if self.sink:
@@ -125,6 +164,13 @@ class SinkAttention:
             specs.append(WeightSpec(prefix + "g", (self.g_dim, h), COMPUTE))
         if self.head_temp:
             specs.append(WeightSpec(prefix + "temp", (self.num_heads,), FLOAT32, init=("uniform", 0.6, 1.6)))
+        if self.conv:
+            specs += [WeightSpec(prefix + n + ".conv", (d, self.conv), FLOAT32, init=("normal", 0.5))
+                      for n, d in (("q", self.q_dim), ("k", self.k_dim), ("v", self.v_dim))]
+        if self.bias_max is not None:
+            specs.append(WeightSpec(prefix + "rel", (None, self.num_heads), FLOAT32, init=("normal", 1.0)))
+        if self.out_bias:
+            specs.append(WeightSpec(prefix + "o.b", (h,), FLOAT32, init=("normal", 0.3)))
         if self.talk:
             specs.append(WeightSpec(prefix + "talk", (self.num_heads, self.num_heads), FLOAT32, init=("normal", 0.4)))
         return specs
@@ -146,18 +192,40 @@ class SinkAttention:
         self.biases = [weights[prefix + n + ".b"] for n in ("q", "k", "v")] if self.bias else [None] * 3
         self.norms = [weights[prefix + "q.norm"], weights[prefix + "k.norm"]] if self.qk_norm else [None, None]
         self.w_sink = weights[prefix + "sink"] if self.sink else None
+        if self.filtered:
+            self.bias_row = torch.cat(self.biases).contiguous() if self.bias else None
+            self.taps = torch.cat([weights[prefix + n + ".conv"] for n in ("q", "k", "v")]).contiguous() if self.conv else None
+        if self.bias_max is not None:   # a row of biases by distance per head; distances past the row take its last value
+            table = weights[prefix + "rel"]
+            rows = torch.tensor(distance_buckets(table.shape[0], float(self.bias_max)), device=table.device)
+            self.rel = table[rows].T.contiguous()
+            self.rel_log2 = (self.rel.double() * math.log2(math.e)).to(torch.float32).contiguous()
+        self.w_ob = weights[prefix + "o.b"] * self.out_scale if self.out_bias else None
+
+    def _project_out(self, out, resid) -> None:
+        ops.linear(out, self.w_o, resid, accumulate=True)
+        if self.w_ob is not None and not self.defer_out_bias:
+            ops.row_add(resid, self.w_ob)
 
     def forward(self, ctx, h, resid, cache) -> None:
         t = h.shape[0]
+        cache, kept = cache if self.conv > 1 else (cache, None)
         nh, nkv, kd, vd = self.num_heads, self.num_kv_heads, self.key_dim, self.value_dim
         width = self.w_in.shape[0]
         # the row stride is a multiple of 8 values so that the rows can feed the tensor-core kernels
         proj = ctx.workspace.get("qkv", (t, _padded(width)), ctx.dtype)[:, :width]
         ops.linear(h, self.w_in, proj, cluster_slices=True)
-        ops.qk_norm_kv_write(proj, ctx.batch.positions, nh, nkv, kd, vd, cache.k, cache.v, cache.slot_mapping,
-                             *self.biases, *self.norms, eps=self.eps, stretch_coef=self.stretch_coef,
-                             stretch_every=self.stretch_every, freq=self.freq, rot_pairs=self.rot_layout == "pairs",
-                             rot_mag=self.rot_mag)
+        q = proj
+        if self.filtered:
+            q = ctx.workspace.get("filtered_q", (t, self.q_dim), ctx.dtype)
+            ops.conv_norm_kv_write(proj, ctx.batch, nh, nkv, kd, vd, cache.k, cache.v, cache.slot_mapping, q,
+                                   bias=self.bias_row, taps=self.taps, kept=None if kept is None else kept.state,
+                                   norm_q=self.norms[0], norm_k=self.norms[1], eps=self.eps)
+        else:
+            ops.qk_norm_kv_write(proj, ctx.batch.positions, nh, nkv, kd, vd, cache.k, cache.v, cache.slot_mapping,
+                                 *self.biases, *self.norms, eps=self.eps, stretch_coef=self.stretch_coef,
+                                 stretch_every=self.stretch_every, freq=self.freq, rot_pairs=self.rot_layout == "pairs",
+                                 rot_mag=self.rot_mag)
         out = ctx.workspace.get("attn_out", (t, self.o_dim), ctx.dtype)
         off = self.q_dim + self.k_dim + self.v_dim
         if self.mix is not None:    # all heads' scores meet: one kernel, which also applies a gate per head
@@ -168,15 +236,16 @@ class SinkAttention:
                                mix_log2=self.mix_log2, workspace=ctx.workspace)
             if self.gate and not per_head:
                 ops.sigmoid_gate(attn, proj[:, off:off + self.o_dim], nh, vd, out)
-            ops.linear(out, self.w_o, resid, accumulate=True)
+            self._project_out(out, resid)
             return
         # with a gate the attention leaves float32 rows and the gate kernel rounds them; without, it writes `out` itself
         attn = ctx.workspace.get("attn_maps", (t, self.o_dim), torch.float32) if self.gate else out
-        ops.paged_attention_maps(proj, nh, nkv, 1, kd, vd, cache.k, cache.v, cache.block_table, ctx.batch, attn,
-                                 self.scale, self.window, None, sink=self.w_sink, workspace=ctx.workspace)
+        ops.paged_attention_maps(q, nh, nkv, 1, kd, vd, cache.k, cache.v, cache.block_table, ctx.batch, attn,
+                                 self.scale, self.window, None, sink=self.w_sink, workspace=ctx.workspace,
+                                 keep_first=self.keep_first, rel=self.rel, rel_log2=self.rel_log2)
         if self.gate:
             ops.sigmoid_gate(attn, proj[:, off:off + self.g_dim], nh, vd, out)
-        ops.linear(out, self.w_o, resid, accumulate=True)
+        self._project_out(out, resid)
 
 
 class LatentAttention:
@@ -184,9 +253,13 @@ class LatentAttention:
 
     def __init__(self, hidden_size: int, num_heads: int, plain_dim: int, rot_part: int, value_dim: int, rank: int,
                  scale: float, eps: float, rot_dims: int = 0, rot_base: float = 10000.0, window: Optional[int] = None,
-                 sink: bool = True, gate: bool = True, rot_scaling: Optional[dict] = None, out_scale: float = 1.0,
-                 shares_cache: bool = False):
+                 sink: bool = True, gate=True, rot_scaling: Optional[dict] = None, rot_layout: str = "pairs",
+                 out_scale: float = 1.0, shares_cache: bool = False):
+        if gate not in (True, False, "value") or rot_layout not in ("halves", "pairs"):
+            raise ValueError(f"unknown gate kind {gate!r} (True: one per head, \"value\": one per output value, False: none) "
+                             f"or rotation layout {rot_layout!r} (halves, pairs)")
         self.shares_cache, self.gate, self.rot_scaling, self.rot_mag = shares_cache, gate, rot_scaling, 1.0
+        self.rot_pairs = rot_layout == "pairs"
         if rot_dims % 2 or rot_dims > rot_part:
             raise ValueError(f"{rot_dims} rotated values must be even and at most the rotated part's size {rot_part}")
         if plain_dim < 1:
@@ -205,6 +278,8 @@ class LatentAttention:
     def cache_need(self):
         return KVNeed(1, self.key_dim, self.window, value_dim=self.rank)
 
+    cache_reach = cache_need     # a layer that reads another's latents may see farther back than their owner
+
     def weight_specs(self, prefix: str):
         h, nh = self.hidden_size, self.num_heads
         specs = [WeightSpec(prefix + "q", (self.q_dim, h), COMPUTE),
@@ -215,7 +290,7 @@ class LatentAttention:
             specs += [WeightSpec(prefix + "dkv", (self.key_dim, h), COMPUTE),
                       WeightSpec(prefix + "dkv.norm", (self.rank,), FLOAT32, init=("uniform", 0.5, 1.5))]
         if self.gate:
-            specs.append(WeightSpec(prefix + "g", (nh, h), COMPUTE))
+            specs.append(WeightSpec(prefix + "g", (nh * self.value_dim if self.gate == "value" else nh, h), COMPUTE))
         if self.sink:
             specs.append(WeightSpec(prefix + "sink", (nh,), FLOAT32, init=("normal", 1.0)))
         return specs
@@ -247,22 +322,24 @@ class LatentAttention:
         q_lat = ctx.workspace.get("latent_q", (t, nh, kd), ctx.dtype)
         if self.shares_cache:   # the other layer's step has written the token's rows already; only the queries turn
             ops.latent_kv_write(proj, ctx.batch.positions, nh, nd, rd, rank, self.rot_dims, self.freq, None, self.eps,
-                                q_lat, None, None, None, rot_mag=self.rot_mag)
+                                q_lat, None, None, None, rot_mag=self.rot_mag, rot_pairs=self.rot_pairs)
         else:
             ops.latent_kv_write(proj, ctx.batch.positions, nh, nd, rd, rank, self.rot_dims, self.freq, self.w_norm, self.eps,
-                                q_lat, cache.k, cache.v, cache.slot_mapping, rot_mag=self.rot_mag)
+                                q_lat, cache.k, cache.v, cache.slot_mapping, rot_mag=self.rot_mag,
+                                rot_pairs=self.rot_pairs)
         ops.head_linear(proj[:, :nh * qd].view(t, nh, qd)[:, :, :nd], self.w_uk_t, q_lat[:, :, :rank])
         attn = ctx.workspace.get("attn_maps", (t, nh * rank), torch.float32)
         ops.paged_attention_maps(q_lat.view(t, nh * kd), nh, 1, 1, kd, rank, cache.k, cache.v, cache.block_table,
                                  ctx.batch, attn, self.scale, self.window, None, sink=self.w_sink, workspace=ctx.workspace)
         gated = ctx.workspace.get("latent_o", (t, nh * rank), ctx.dtype)
-        if self.gate:
-            g0 = self.q_dim + (0 if self.shares_cache else kd)
+        g0 = self.q_dim + (0 if self.shares_cache else kd)
+        if self.gate is True:
             ops.sigmoid_gate(attn, proj[:, g0:g0 + nh], nh, rank, gated)
         else:
             ops.unary(attn, gated)
         out = ctx.workspace.get("attn_out", (t, nh * vd), ctx.dtype)
-        ops.head_linear(gated.view(t, nh, rank), self.w_uv, out.view(t, nh, vd))
+        ops.head_linear(gated.view(t, nh, rank), self.w_uv, out.view(t, nh, vd),
+                        gate=proj[:, g0:g0 + nh * vd].view(t, nh, vd) if self.gate == "value" else None)
         ops.linear(out, self.w_o, resid, accumulate=True)
 
 
