@@ -17,7 +17,8 @@ Dunelix model at the TinyLlama layer sizes beside the Llama decoder at equal siz
 like kernels, each against its roofline (`--only decode` with it: the decode points alone).  `--design zozenex` does
 the same for a Zozenex model (retention and gated linear attention, window attention with pooled blocks, routed
 experts) beside the Dunelix model at equal width, layers and vocabulary, `--design gevovik` for a Gevovik model beside
-the Fiponex model, `--design fiponex` for a Fiponex model (gated
+the Fiponex model, `--design vigodra` for a Vigodra model (attention behind short filters with a distance bias, latent
+attention with a gate per value, post-norm blocks with a depth average) beside the Gevovik model, `--design fiponex` for a Fiponex model (gated
 delta rule, latent attention, attention with a sink, dense and routed gated feed-forwards) beside the Zozenex model."""
 import argparse
 import json
@@ -748,7 +749,7 @@ def fiponex_decode_bytes(model, runner, batch, mean_ctx, itemsize):
         chosen = f.num_experts * (1.0 - (1.0 - f.top / f.num_experts) ** batch)
         total += (chosen - f.num_experts) * expert     # spec_weight_bytes counts every expert
     for g in runner.cache.groups:
-        seen = mean_ctx if g.need.window is None else min(mean_ctx, g.need.window)
+        seen = mean_ctx if g.need.window is None else min(mean_ctx, g.need.window + g.need.keep_first)
         total += batch * seen * g.bytes_per_token(itemsize)
     for n in runner.cache.slots.needs:
         numel = 1
@@ -756,6 +757,7 @@ def fiponex_decode_bytes(model, runner, batch, mean_ctx, itemsize):
             numel *= d
         total += 2 * batch * 4 * numel
     return int(total)
+
 
 def fiponex_kernels(dtype, device, pk, tokens=2048):
     """The design's kernels alone at the sizes of one layer of the --design shape and `tokens` tokens of one prompt, and
@@ -1099,6 +1101,154 @@ def gevovik_kernels(dtype, device, pk, tokens=2048):
     return out
 
 
+# `--design vigodra`: a Vigodra model (grouped-query attention behind short filters with norms over the whole projection, a
+# distance bias, a window that keeps the first positions and a sink; latent attention over a window with a gate per value,
+# every second one reading the cache of the one before; post-norm blocks whose results are averaged over the depth; clamped
+# gated feed-forwards) at the same width, layers and vocabulary, beside the Gevovik model above (the closest design the
+# engine has: latent attention with shared caches, a window attention, filters, branches that read the stream itself).
+def vigodra_shape(layers=DESIGN_LAYERS, width=2048, vocab=32000, ff=5632, window=1024):
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    att = {"heads": 16, "kv_heads": 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "conv": 4, "bias_max": 512,
+           "mask": {"size": window, "keep_first": 64}}
+    latent = {"heads": 16, "dim": 64, "rot_dim": 64, "vdim": 128, "kv_rank": 192, "scale": 128 ** -0.5,
+              "mask": {"size": window}, "rot": {"dims": 64, "base": 10000.0}}
+    out = []
+    for i in range(layers):
+        if i % 2 == 0:
+            out.append({"type": "attention", "mixer": att, "mlp": dense})
+        else:
+            out.append({"type": "latent_attention", "mixer": latent if i % 4 == 1 else dict(latent, kv_from=i - 2), "mlp": dense})
+    return {"architecture": "Vigodra", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "initializer_range": 0.02,
+            "embedding": {"scale": width ** 0.5}, "postln_alpha": (2 * layers) ** 0.25, "layers": out}
+
+
+def vigodra_kernels(dtype, device, pk, tokens=2048):
+    """The design's kernels alone at the sizes of one layer of the --design shape and `tokens` tokens of one prompt, and
+    their like kernels of the Gevovik and Fiponex paths: microseconds, achieved GB/s or TFLOP/s, share of the peak."""
+    import types
+    import torch
+    from tiny_llm_b200 import ops
+    from tiny_llm_b200.engine import Workspace
+    from tiny_llm_b200.parts import distance_buckets
+    t, width, page, window, keep = tokens, 2048, PAGE, 1024, 64
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=device)
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=device)
+    rnd = lambda *shape: torch.randn(*shape, device=device).to(dtype)
+    out = {}
+    isz = 2 if dtype == torch.bfloat16 else 4
+
+    def mem(name, us, nbytes):
+        out[name] = {"us": round(us, 2), "gbs": round(nbytes / us / 1e3, 1), "frac": round(nbytes / us / 1e3 / pk["hbm_gbs"], 3)}
+
+    def flop(name, us, flops):
+        out[name] = {"us": round(us, 2), "tflops": round(flops / us / 1e6, 1), "frac": round(flops / us / 1e6 / pk["bf16_tflops"], 3)}
+
+    ws = Workspace(torch.device(device))
+    pages = -(-t // page)
+    table = i32([list(range(pages))])
+    slots, pos = i32(list(range(t))), i32(list(range(t)))
+    meta = types.SimpleNamespace(token_request=i32([0] * t), positions=pos, cu_q=i32([0, t]), q_start=i32([0]), slots=i32([1]),
+                                 num_requests=1, num_tokens=t, max_q_len=t, max_kv_len=t, num_leading_decodes=0)
+
+    # attention: biases + filters + whole-row norms + cache write; the scores with a distance bias, kept keys and a sink
+    h, kvh, kd, vd, taps = 16, 4, 128, 128, 4
+    nqc, nkc, nvc = h * kd, kvh * kd, kvh * vd
+    ch = nqc + nkc + nvc
+    proj = rnd(t, ch)
+    kc = torch.zeros(pages, kvh, page, kd, dtype=dtype, device=device)
+    vc = torch.zeros(pages, kvh, page, vd, dtype=dtype, device=device)
+    q = torch.empty(t, nqc, dtype=dtype, device=device)
+    bias, w_taps = torch.zeros(ch, device=device), torch.randn(ch, taps, device=device) * 0.5
+    kept = torch.zeros(4, taps - 1, ch, device=device)
+    wq, wk = torch.ones(nqc, device=device), torch.ones(nkc, device=device)
+    mem("conv_norm_kv_write (biases, 4 taps, norms over all heads) + conv_state_update", time_kernel(lambda: ops.conv_norm_kv_write(
+        proj, meta, h, kvh, kd, vd, kc, vc, slots, q, bias=bias, taps=w_taps, kept=kept, norm_q=wq, norm_k=wk, eps=1e-6), flush),
+        t * ch * isz * 2)
+    qn, kn = torch.ones(kd, device=device), torch.ones(kd, device=device)
+    mem("qk_norm_kv_write (like: biases, norms per head)", time_kernel(lambda: ops.qk_norm_kv_write(
+        proj, pos, h, kvh, kd, vd, kc, vc, slots, bias[:nqc], bias[nqc:nqc + nkc].contiguous(), bias[nqc + nkc:].contiguous(), qn, kn,
+        eps=1e-6), flush), t * ch * isz * 2)
+    dh, dk = 8, 128
+    dch = 2 * dh * dk + 8 * 128
+    dq, dkk = torch.empty(t, dh * dk, device=device), torch.empty(t, dh * dk, device=device)
+    dv, gb = torch.empty(t, 8 * 128, device=device), torch.empty(t, 8, 2, device=device)
+    dproj, d_taps, d_kept = rnd(t, dch + 16), torch.randn(dch, taps, device=device) * 0.5, torch.zeros(4, taps - 1, dch, device=device)
+    z8 = torch.zeros(8, device=device)
+    mem("delta_prepare (like: filters, SiLU, unit norms)", time_kernel(lambda: ops.delta_prepare(
+        dproj, d_taps, d_kept, meta, 8, dh, dk, 128, dch, dch + 8, z8, z8, dk ** -0.5, 1e-6, dq, dkk, dv, gb), flush), t * dch * (isz + 4))
+    att = torch.empty(t, h * vd, dtype=torch.float32, device=device)
+    sink = torch.zeros(h, device=device)
+    rows = torch.tensor(distance_buckets(32, 512.0), device=device)
+    rel = torch.randn(32, h, device=device)[rows].T.contiguous()
+    rel2 = (rel * 1.4426950408889634).contiguous()
+    wpairs = sum(min(p + 1, window + min(keep, max(0, p - window + 1))) for p in range(t))
+    plain_pairs = sum(min(p + 1, window) for p in range(t))
+    kq = rnd(t, h * kd)
+    flop("attention, window 1024 + 64 kept keys, distance bias, sink (16 heads of 128)", time_kernel(lambda: ops.paged_attention_maps(
+        kq, h, kvh, 1, kd, vd, kc, vc, table, meta, att, kd ** -0.5, window, None, sink=sink, keep_first=keep, rel=rel, rel_log2=rel2,
+        workspace=ws), flush, repeats=5), 2.0 * wpairs * h * (kd + vd))
+    flop("attention with a sink, window 1024 (like)", time_kernel(lambda: ops.paged_attention_maps(
+        kq, h, kvh, 1, kd, vd, kc, vc, table, meta, att, kd ** -0.5, window, None, sink=sink, workspace=ws), flush, repeats=5),
+        2.0 * plain_pairs * h * (kd + vd))
+
+    # latent attention: rotation in halves, the gate per value in the value products' last lines
+    h, nd, rd, lvd, rank = 16, 64, 64, 128, 192
+    lkd = rank + rd
+    lproj = rnd(t, -(-(h * (nd + rd) + lkd + h * lvd) // 8) * 8)
+    lkc = torch.zeros(pages, 1, page, lkd, dtype=dtype, device=device)
+    lvc = torch.zeros(pages, 1, page, rank, dtype=dtype, device=device)
+    q_lat = torch.zeros(t, h, lkd, dtype=dtype, device=device)
+    freq = torch.pow(torch.tensor(10000.0), -torch.arange(rd // 2, dtype=torch.float32) * 2 / rd).to(device)
+    wl = torch.ones(rank, device=device)
+    for label, pairs_layout in (("rotation in halves", False), ("like: rotation in pairs", True)):
+        mem(f"latent_kv_write ({label})", time_kernel(lambda: ops.latent_kv_write(
+            lproj, pos, h, nd, rd, rank, rd, freq, wl, 1e-6, q_lat, lkc, lvc, slots, rot_pairs=pairs_layout), flush),
+            t * isz * (h * rd * 2 + lkd * 2 + rank))
+    w_uk_t, w_uv = rnd(h, rank, nd), rnd(h, lvd, rank)
+    flop("head_linear: latent query products (16 heads, 64 -> 192; shared with the like)", time_kernel(lambda: ops.head_linear(
+        lproj[:, :h * (nd + rd)].view(t, h, nd + rd)[:, :, :nd], w_uk_t, q_lat[:, :, :rank]), flush), 2.0 * t * h * nd * rank)
+    latt = torch.empty(t, h * rank, dtype=torch.float32, device=device)
+    flop("latent attention (key row 256, value row 192, window 1024; shared with the like)", time_kernel(
+        lambda: ops.paged_attention_maps(q_lat.view(t, h * lkd), h, 1, 1, lkd, rank, lkc, lvc, table, meta, latt, 0.0884, window, None,
+                                         workspace=ws), flush, repeats=5), 2.0 * plain_pairs * h * (lkd + rank))
+    lg = rnd(t, h * rank)
+    lout = torch.empty(t, h * lvd, dtype=dtype, device=device)
+    off = h * (nd + rd) + lkd
+    gate = lproj[:, off:off + h * lvd].view(t, h, lvd)
+    flop("head_linear: latent value products with the gate per value (16 heads, 192 -> 128)", time_kernel(lambda: ops.head_linear(
+        lg.view(t, h, rank), w_uv, lout.view(t, h, lvd), gate=gate), flush), 2.0 * t * h * rank * lvd)
+    flop("head_linear: latent value products (like)", time_kernel(lambda: ops.head_linear(
+        lg.view(t, h, rank), w_uv, lout.view(t, h, lvd)), flush), 2.0 * t * h * rank * lvd)
+
+    # the stream: the norm of the sum, with the depth average over 1, 4 and 8 earlier stages; the gate of the feed-forward
+    x, branch = torch.randn(t, width, device=device), torch.randn(t, width, device=device)
+    w1, b1 = torch.ones(width, device=device), torch.zeros(width, device=device)
+    cp = torch.empty(t, width, dtype=torch.bfloat16, device=device)
+    stages = torch.randn(9, t, width, device=device)
+    mem("post_norm_join (norm of the sum, output bias, rounded copy)", time_kernel(lambda: ops.post_norm_join(
+        branch, x, w1, b1, 1e-6, 2.0, out_bias=b1, copy=cp), flush), t * width * 18)
+    for n in (1, 4, 8):
+        mix = torch.full((n + 1,), 0.3, device=device)
+        mem(f"post_norm_join with the depth average over {n} earlier stages", time_kernel(lambda: ops.post_norm_join(
+            branch, x, w1, b1, 1e-6, 2.0, copy=cp, stages=stages, done=n, mix=mix, keep=True), flush), t * width * (22 + 4 * n))
+    resid = torch.zeros(t, width, device=device)
+    mem("rms_norm_add with a rounded copy (like)", time_kernel(lambda: ops.rms_norm_add(x, w1, 1e-6, 1.0, resid, copy=cp), flush), t * width * 18)
+    emb = rnd(32000, width)
+    toks = torch.randint(0, 32000, (t,), dtype=torch.int32, device=device)
+    mem("embedding, three outputs", time_kernel(lambda: ops.embedding(toks, emb, resid, scale=2.0, twin=stages[0], copy=cp), flush), t * width * (isz + 10))
+    mem("embedding (like)", time_kernel(lambda: ops.embedding(toks, emb, resid, scale=2.0), flush), t * width * (isz + 4))
+    yy = torch.empty(t, width, dtype=dtype, device=device)
+    mem("layer_norm", time_kernel(lambda: ops.layer_norm(x, w1, b1, 1e-6, yy), flush), t * width * (4 + isz))
+    mem("rms_norm (like)", time_kernel(lambda: ops.rms_norm(x, w1, 1e-6, yy), flush), t * width * (4 + isz))
+    ff = 5632
+    h_in, w_gu = rnd(t, width), rnd(2 * ff, width)
+    act = torch.empty(t, ff, dtype=dtype, device=device)
+    flop("gate and up product with the clamped gate", time_kernel(lambda: ops.linear_swiglu(h_in, w_gu, act, 128, ws, act="clamped", limit=7.0), flush),
+         2.0 * t * 2 * ff * width)
+    flop("gate and up product with SiLU (like)", time_kernel(lambda: ops.linear_swiglu(h_in, w_gu, act, 128, ws), flush), 2.0 * t * 2 * ff * width)
+    return out
+
+
 def design_run(args, dtype, device, pk):
     import gc
     import torch
@@ -1125,13 +1275,19 @@ def design_run(args, dtype, device, pk):
                         "key/value heads, keys and values of 128, window 1024, stretched rotation, gate per head) beside a delta "
                         "rule with decays per key channel (16 heads, 8 query/key heads, keys and values of 128, 4 taps); latent "
                         "attention reading the first one's cache; every layer with a relu-squared feed-forward of 5632; beside: "
-                        "the Fiponex model of --design fiponex at equal width, layers and vocabulary"}
+                        "the Fiponex model of --design fiponex at equal width, layers and vocabulary",
+             "vigodra": "width 2048, vocabulary 32000; layers in turn: attention (16 heads, 4 key/value heads, keys and values of 128, "
+                        "4 taps, window 1024 with 64 kept positions, distance bias, sink, biases); latent attention (16 heads, 64 "
+                        "plain + 64 rotated, values of 128, latent 192, window 1024, gate per value); attention; latent attention "
+                        "reading the cache of the one before; post-norm blocks averaged over the depth; every layer with a clamped "
+                        "gated feed-forward of 5632; beside: the Gevovik model of --design gevovik at equal width, layers and "
+                        "vocabulary"}
     result = {"design": args.design, "dtype": args.dtype, "layers": DESIGN_LAYERS, "peaks": pk["source"],
               "sizes": sizes[args.design],
               "l2": "whole steps: weights larger than L2; kernels alone: L2 flushed before every timed call"}
     sampler = ClockSampler().start()
     labels = {"dunelix": ("dunelix", "llama"), "zozenex": ("zozenex", "dunelix"), "fiponex": ("fiponex", "zozenex"),
-              "gevovik": ("gevovik", "fiponex")}[args.design]
+              "gevovik": ("gevovik", "fiponex"), "vigodra": ("vigodra", "gevovik")}[args.design]
     for label in labels[:1 if args.only == "decode" else 2]:
         if label == "dunelix":
             cfg, model = build_design(dunelix_shape(), dtype, device)
@@ -1141,6 +1297,8 @@ def design_run(args, dtype, device, pk):
             cfg, model = build_design(fiponex_shape(), dtype, device)
         elif label == "gevovik":
             cfg, model = build_design(gevovik_shape(), dtype, device)
+        elif label == "vigodra":
+            cfg, model = build_design(vigodra_shape(), dtype, device)
         else:
             cfg, model = build_model(DESIGN_LAYERS, dtype, device)
         runner = make_runner(model, dtype, device, max_tokens=64 * CONTEXT, page_size=PAGE, max_requests=64,
@@ -1153,7 +1311,7 @@ def design_run(args, dtype, device, pk):
             ms, launched, ctx = timed_decode(runner, bsz, CONTEXT - (REPEATS * steps + warmup), steps, warmup, out, repeats=REPEATS)
             moved = design_decode_bytes(model, runner, bsz, ctx, itemsize) if label == "dunelix" else \
                 zozenex_decode_bytes(model, runner, bsz, ctx, itemsize) if label == "zozenex" else \
-                fiponex_decode_bytes(model, runner, bsz, ctx, itemsize) if label in ("fiponex", "gevovik") else \
+                fiponex_decode_bytes(model, runner, bsz, ctx, itemsize) if label in ("fiponex", "gevovik", "vigodra") else \
                 decode_bytes(model, runner, bsz, ctx, itemsize)
             rec[f"decode_b{bsz}"] = {"ms_per_step": round(ms, 4), "tokens_per_s": round(bsz * 1e3 / ms, 1),
                                      "hbm_frac": round(moved / (ms * 1e-3) / 1e9 / pk["hbm_gbs"], 4), "gpu_launches": launched}
@@ -1164,7 +1322,7 @@ def design_run(args, dtype, device, pk):
     result["clocks"] = sampler.stop()
     if dtype == torch.bfloat16 and args.only == "all":
         result["kernels"] = {"dunelix": design_kernels, "zozenex": zozenex_kernels, "fiponex": fiponex_kernels,
-                             "gevovik": gevovik_kernels}[args.design](dtype, device, pk)
+                             "gevovik": gevovik_kernels, "vigodra": vigodra_kernels}[args.design](dtype, device, pk)
     ops.check_status()
     print(json.dumps(result))
     return 0
@@ -1189,7 +1347,7 @@ def main():
     ap.add_argument("--page-size", type=int, default=PAGE, help="tokens per page of the cache")
     ap.add_argument("--shape", default="tinyllama", choices=["tinyllama"] + list(OTHER_SHAPES),
                     help="layer sizes for --only runs (profiler captures of the other models' kernels)")
-    ap.add_argument("--design", default=None, choices=["dunelix", "zozenex", "fiponex", "gevovik"],
+    ap.add_argument("--design", default=None, choices=["dunelix", "zozenex", "fiponex", "gevovik", "vigodra"],
                     help="instead of the flagship run: this design's prefill and decode at real layer sizes beside the Llama "
                          "decoder at equal sizes, and its kernels beside their like kernels (one plain line, no record)")
     ap.add_argument("--quick", action="store_true",

@@ -1,5 +1,5 @@
-// Attention of the step's queries over the paged cache on the CUDA cores, any key size and any value
-// size up to 256 (the two may differ; key rows whose bytes are a multiple of 16 are read with 16-byte loads), any number of heads and groups, any
+// Attention of the step's queries over the paged cache on the CUDA cores, any key size up to 1,024 and any value
+// size up to 512 (the two may differ; above 256 every (token, head) pair takes eight warps; key rows whose bytes are a multiple of 16 are read with 16-byte loads), any number of heads and groups, any
 // page size.  It is the attention of the true 32-bit path and the fallback of the bfloat16 path.
 //
 // Heads.  A query head has `maps` score maps, each an attention of its own over the same values: the
@@ -34,7 +34,8 @@ TLLM_DEFINE_LAST_ERROR
 namespace tllm {
 
 constexpr int WARPS = 4;
-constexpr int MAX_HD = 256;
+constexpr int MAX_HD = 256;            // sizes of all three launches
+constexpr int MAX_KD = 1024, MAX_VD = 512;   // sizes of the launch with eight warps per pair
 
 // Where the rows of the cache lie and which keys are visible; `nq` and `nk` count (head, map) rows.
 struct Geometry {
@@ -340,7 +341,7 @@ paged_attention_generic_kernel(const T* __restrict__ q, int q_row_stride, const 
                                int max_blocks, const int* __restrict__ token_request,
                                const int* __restrict__ positions, TO* __restrict__ out, int n_tokens,
                                Geometry g, float scale, const float* __restrict__ sink) {
-  __shared__ __align__(16) float q_s[SPLIT ? 1 : WARPS][MAX_HD];
+  __shared__ __align__(16) float q_s[SPLIT ? 1 : WARPS][SPLIT ? MAX_KD : MAX_HD];
   __shared__ float merge_s[SPLIT ? WAYS : 1][SPLIT ? OD * 32 + 2 : 1];
   pdl_trigger();
   pdl_wait();
@@ -426,7 +427,8 @@ static int launch_attention(const void* q, int q_row_stride, const void* kcache,
               GroupedWarps<OD_>::N * 32, 0, s, (const T*)q, q_row_stride, (const T*)kcache, (const T*)vcache,          \
               block_table, max_blocks, token_request, positions, (TO*)out, n_tokens, g, scale, sink)
   if (split) {
-    if (od == 2) TLLM_ATT_GENERIC(true, 2); else if (od == 4) TLLM_ATT_GENERIC(true, 4); else TLLM_ATT_GENERIC(true, 8);
+    if (od == 2) TLLM_ATT_GENERIC(true, 2); else if (od == 4) TLLM_ATT_GENERIC(true, 4); else if (od == 8) TLLM_ATT_GENERIC(true, 8);
+    else TLLM_ATT_GENERIC(true, 16);
   } else if (grouped) {
     if (od == 2) TLLM_ATT_GROUPED(2); else if (od == 4) TLLM_ATT_GROUPED(4); else TLLM_ATT_GROUPED(8);
   } else {
@@ -456,8 +458,8 @@ extern "C" int tllm_paged_attention_maps(const void* q, int q_row_stride, const 
                                          int keep, const float* rel, int rel_len, void* stream) {
   TLLM_REQUIRE(n_tokens > 0 && nq > 0 && nkv > 0 && nq % nkv == 0 && maps > 0,
                "attention: %d tokens, %d heads, %d key/value heads (heads must be a multiple of key/value heads)", n_tokens, nq, nkv);
-  TLLM_REQUIRE(kd >= 1 && kd <= MAX_HD && vd >= 1 && vd <= MAX_HD,
-               "attention: key size %d / value size %d is not built (both up to %d)", kd, vd, MAX_HD);
+  TLLM_REQUIRE(kd >= 1 && kd <= MAX_KD && vd >= 1 && vd <= MAX_VD,
+               "attention: key size %d / value size %d is not built (up to %d / %d)", kd, vd, MAX_KD, MAX_VD);
   TLLM_REQUIRE(page_size > 0 && max_blocks > 0 && window >= 0 && chunk >= 0, "attention: page size %d, %d blocks, window %d, chunk %d", page_size, max_blocks, window, chunk);
   TLLM_REQUIRE(keep >= 0 && (rel == nullptr || rel_len >= 1), "attention: %d kept keys, %d distances of a bias", keep, rel_len);
   const int elem = dtype == TLLM_F32 ? 4 : 2;
@@ -475,10 +477,11 @@ extern "C" int tllm_paged_attention_maps(const void* q, int q_row_stride, const 
     TLLM_FAIL(TLLM_ERR_CUDA, "attention: cannot read the number of SMs");
   // split_override: -1 by the number of pairs; 1 eight warps per pair; 0 one warp per (token, key row, four query rows);
   // 2 one warp per pair (the plainest form, kept for comparison: all give the same bits)
-  const bool split = split_override >= 0 ? split_override == 1 : tasks <= 8LL * sms;
+  const bool large = kd > MAX_HD || vd > MAX_HD;
+  const bool split = large || (split_override >= 0 ? split_override == 1 : tasks <= 8LL * sms);
   const bool grouped = !split && split_override != 2;
   const int hd = kd > vd ? kd : vd;
-  const int od = hd <= 64 ? 2 : (hd <= 128 ? 4 : 8);
+  const int od = large ? 16 : (hd <= 64 ? 2 : (hd <= 128 ? 4 : 8));
   const int gw = od <= 2 ? 4 : (od <= 4 ? 2 : 1);
   const long long gtasks = (long long)n_tokens * g.nk * ((nq / nkv + GH - 1) / GH);
   const long long blocks = split ? tasks : (grouped ? (gtasks + gw - 1) / gw : (tasks + WARPS - 1) / WARPS);

@@ -11,8 +11,8 @@
 // Scores, the running softmax (max, sum, rescale; exp2 on scores scaled by scale * log2 e) and the weights P stay
 // 32-bit: P enters the P V product as the sum of two bfloat16 numbers, P = hi + lo with hi = bf16(P) and
 // lo = bf16(P - hi), so the product sees 16 bits of every weight's mantissa (relative error 2^-17, the size of the
-// 32-bit rounding of the sums themselves) where a single bfloat16 operand would keep 8.  The output rows are float32
-// [token][head][map][VD], for the kernel that combines a head's maps.
+// 32-bit rounding of the sums themselves) where a single bfloat16 operand would keep 8.  The output rows
+// [token][head][map][VD] are float32, for the kernel that combines a head's maps or gates them, or bfloat16, for a product.
 //
 // With a sink (a learned score per head) the softmax's denominator also holds exp(sink); it has no value row.
 //
@@ -46,7 +46,8 @@ struct MapsParams {
   const int* block_table;        // [R, max_blocks]
   const int* cu_q;               // [R + 1]
   const int* q_start;            // [R]: position of the request's first token in this step
-  float* out;                    // [T, nq * maps, VD]
+  void* out;                     // [T, nq * maps, VD], float32 or bfloat16
+  int out_bf16;
   const float* sink;             // [nq] or null: exp(sink) joins the denominator of every softmax of the head
   long long k_page_stride, k_head_stride, v_page_stride, v_head_stride;
   int q_row_stride, max_blocks, nq, nkv, maps, page_size, window, chunk, tiles_per_req, n_requests;
@@ -346,17 +347,25 @@ attention_maps_kernel(const MapsParams p) {
       const float top = fmaxf(m, sk), f = ex2(m - top);
       inv = f / fmaf(half ? l_b : l_a, f, ex2(sk - top));
     }
-    float* dst = p.out + ((size_t)(tok0 + row / group) * p.nq * p.maps + (size_t)((kvh * group + row % group) * p.maps + map)) * VD;
+    const size_t at = ((size_t)(tok0 + row / group) * p.nq * p.maps + (size_t)((kvh * group + row % group) * p.maps + map)) * VD + t4 * 2;
+    if (p.out_bf16) {
+      __nv_bfloat16* dst = (__nv_bfloat16*)p.out + at;
 #pragma unroll
-    for (int i = 0; i < VD / 8; ++i)
-      *reinterpret_cast<float2*>(dst + i * 8 + t4 * 2) = make_float2(o[i][half * 2] * inv, o[i][half * 2 + 1] * inv);
+      for (int i = 0; i < VD / 8; ++i)
+        *reinterpret_cast<uint32_t*>(dst + i * 8) = pack_bf16(o[i][half * 2] * inv, o[i][half * 2 + 1] * inv);
+    } else {
+      float* dst = (float*)p.out + at;
+#pragma unroll
+      for (int i = 0; i < VD / 8; ++i)
+        *reinterpret_cast<float2*>(dst + i * 8) = make_float2(o[i][half * 2] * inv, o[i][half * 2 + 1] * inv);
+    }
   }
 }
 
 // Joins the runs of one row: with M the largest of the runs' maxima (and the sink), out = sum_s o_s 2^(m_s - M) /
 // (sum_s l_s 2^(m_s - M) + 2^(sink - M)), runs in ascending order.  One warp per row.
-__global__ void __launch_bounds__(128) attention_maps_merge_kernel(const float* __restrict__ part, float* __restrict__ out,
-                                                                   const float* __restrict__ sink, int total_rows, int splits,
+__global__ void __launch_bounds__(128) attention_maps_merge_kernel(const float* __restrict__ part, void* __restrict__ out,
+                                                                   int out_bf16, const float* __restrict__ sink, int total_rows, int splits,
                                                                    int heads_maps, int maps) {
   pdl_trigger();
   pdl_wait();
@@ -383,7 +392,8 @@ __global__ void __launch_bounds__(128) attention_maps_merge_kernel(const float* 
       const float* src = part + ((size_t)s * total_rows + row) * LD;
       acc = fmaf(src[d], ex2(src[VD] - top), acc);
     }
-    out[(size_t)row * VD + d] = acc * inv;
+    if (out_bf16) ((__nv_bfloat16*)out)[(size_t)row * VD + d] = __float2bfloat16_rn(acc * inv);
+    else ((float*)out)[(size_t)row * VD + d] = acc * inv;
   }
 }
 
@@ -393,7 +403,7 @@ using namespace tllm;
 
 extern "C" int tllm_attention_maps_mma(const void* q, int q_row_stride, const void* kcache, const void* vcache,
                                        const int* block_table, int max_blocks, const int* cu_q, const int* q_start,
-                                       float* out, int n_tokens, int n_requests, int max_q_len, int nq, int nkv, int maps,
+                                       void* out, int out_bf16, int n_tokens, int n_requests, int max_q_len, int nq, int nkv, int maps,
                                        int kd, int vd, int page_size, long long k_page_stride, long long k_head_stride,
                                        long long v_page_stride, long long v_head_stride, float scale, int window, int chunk,
                                        const float* sink, int splits, float* part, int keep, const float* rel, int rel_len,
@@ -413,7 +423,7 @@ extern "C" int tllm_attention_maps_mma(const void* q, int q_row_stride, const vo
   MapsParams p;
   p.keep = window > 0 ? keep : 0; p.rel = rel; p.rel_len = rel_len;
   p.q = (const __nv_bfloat16*)q; p.kcache = (const __nv_bfloat16*)kcache; p.vcache = (const __nv_bfloat16*)vcache;
-  p.block_table = block_table; p.cu_q = cu_q; p.q_start = q_start; p.out = out; p.sink = sink;
+  p.block_table = block_table; p.cu_q = cu_q; p.q_start = q_start; p.out = out; p.out_bf16 = out_bf16; p.sink = sink;
   p.k_page_stride = k_page_stride; p.k_head_stride = k_head_stride; p.v_page_stride = v_page_stride; p.v_head_stride = v_head_stride;
   p.q_row_stride = q_row_stride; p.max_blocks = max_blocks; p.nq = nq; p.nkv = nkv; p.maps = maps; p.page_size = page_size;
   p.window = window; p.chunk = chunk; p.n_requests = n_requests;
@@ -436,6 +446,6 @@ extern "C" int tllm_attention_maps_mma(const void* q, int q_row_stride, const vo
   else TLLM_LAUNCH("attention_maps_mma", (attention_maps_kernel<ST, false>), grid, 128, smem, (cudaStream_t)stream, p);
   if (splits > 1)
     TLLM_LAUNCH("attention_maps_merge", attention_maps_merge_kernel, dim3((unsigned)((p.total_rows + 3) / 4)), 128, 0,
-                (cudaStream_t)stream, (const float*)part, out, sink, p.total_rows, splits, nq * maps, maps);
+                (cudaStream_t)stream, (const float*)part, out, out_bf16, sink, p.total_rows, splits, nq * maps, maps);
   return TLLM_OK;
 }

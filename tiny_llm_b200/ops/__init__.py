@@ -1556,8 +1556,8 @@ def paged_attention_maps(qkv: torch.Tensor, num_heads: int, num_kv_heads: int, m
     (the tensor-core kernel's units; without it that kernel is not taken).
     `batch`: token_request and positions per token
     (the CUDA-core kernel); cu_q, q_start per request, num_requests, max_q_len (the tensor-core kernel).
-    bfloat16 with a float32 output and sizes that are multiples of 16 runs on the tensor cores, everything else on
-    the CUDA cores in 32-bit.  `workspace` (the step's named buffers): lets a step of decoded tokens cut the keys of a
+    bfloat16 with sizes that are multiples of 16 up to 256 runs on the tensor cores, everything else on the CUDA cores
+    in 32-bit.  `workspace` (the step's named buffers): lets a step of decoded tokens cut the keys of a
     row tile into runs that separate CTAs walk (needs batch.max_kv_len, an upper bound of the contexts)."""
     _need_cuda(qkv, k_cache, v_cache, block_table, out, sink)
     _i32(block_table, "block_table")
@@ -1578,7 +1578,7 @@ def paged_attention_maps(qkv: torch.Tensor, num_heads: int, num_kv_heads: int, m
             v_cache.shape[1] != num_kv_heads or v_cache.shape[3] != value_dim or k_cache.shape[2] != v_cache.shape[2]:
         raise KernelError("paged_attention_maps: shapes or dtypes do not fit")
     few = getattr(batch, "max_q_len", 0) == 1 and t * num_heads * maps <= attention_maps_decode_pairs
-    if qkv.dtype == torch.bfloat16 and out.dtype == torch.float32 and not force_generic and attention_maps_tc and \
+    if qkv.dtype == torch.bfloat16 and not force_generic and attention_maps_tc and \
             (rel is None or rel_log2 is not None) and not few and scale > 0 and key_dim % 16 == 0 and value_dim % 16 == 0 and 16 <= key_dim <= 256 and 16 <= value_dim <= 256 and \
             qkv.stride(0) % 8 == 0 and qkv.data_ptr() % 16 == 0:
         # bfloat16: the tensor-core kernel compiled for this pair of sizes (prompt portions and decoded tokens alike)
@@ -1594,8 +1594,8 @@ def paged_attention_maps(qkv: torch.Tensor, num_heads: int, num_kv_heads: int, m
                 part = workspace.get("attn_maps_part", (splits, t * num_heads * maps, value_dim + 2), torch.float32)
         _call(lib, lib.tllm_attention_maps_mma,
               _ptr(qkv), qkv.stride(0), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1],
-              _ptr(batch.cu_q), _ptr(batch.q_start), _ptr(out), t, batch.num_requests, batch.max_q_len, num_heads,
-              num_kv_heads, maps, key_dim, value_dim, k_cache.shape[2], ctypes.c_longlong(k_cache.stride(0)),
+              _ptr(batch.cu_q), _ptr(batch.q_start), _ptr(out), 1 if out.dtype == torch.bfloat16 else 0, t, batch.num_requests,
+              batch.max_q_len, num_heads, num_kv_heads, maps, key_dim, value_dim, k_cache.shape[2], ctypes.c_longlong(k_cache.stride(0)),
               ctypes.c_longlong(k_cache.stride(1)), ctypes.c_longlong(v_cache.stride(0)),
               ctypes.c_longlong(v_cache.stride(1)), ctypes.c_float(scale), int(window or 0), int(chunk or 0), _ptr(sink),
               splits, _ptr(part), keep_first, _ptr(rel_log2), rel_len, _stream())

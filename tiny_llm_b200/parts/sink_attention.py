@@ -328,15 +328,14 @@ class LatentAttention:
                                 q_lat, cache.k, cache.v, cache.slot_mapping, rot_mag=self.rot_mag,
                                 rot_pairs=self.rot_pairs)
         ops.head_linear(proj[:, :nh * qd].view(t, nh, qd)[:, :, :nd], self.w_uk_t, q_lat[:, :, :rank])
-        attn = ctx.workspace.get("attn_maps", (t, nh * rank), torch.float32)
+        # a gate per head reads the attention's 32-bit rows; without one the rows are rounded as they are stored
+        gated = ctx.workspace.get("latent_o", (t, nh * rank), ctx.dtype)
+        attn = ctx.workspace.get("attn_maps", (t, nh * rank), torch.float32) if self.gate is True else gated
         ops.paged_attention_maps(q_lat.view(t, nh * kd), nh, 1, 1, kd, rank, cache.k, cache.v, cache.block_table,
                                  ctx.batch, attn, self.scale, self.window, None, sink=self.w_sink, workspace=ctx.workspace)
-        gated = ctx.workspace.get("latent_o", (t, nh * rank), ctx.dtype)
         g0 = self.q_dim + (0 if self.shares_cache else kd)
         if self.gate is True:
             ops.sigmoid_gate(attn, proj[:, g0:g0 + nh], nh, rank, gated)
-        else:
-            ops.unary(attn, gated)
         out = ctx.workspace.get("attn_out", (t, nh * vd), ctx.dtype)
         ops.head_linear(gated.view(t, nh, rank), self.w_uv, out.view(t, nh, vd),
                         gate=proj[:, g0:g0 + nh * vd].view(t, nh, vd) if self.gate == "value" else None)
