@@ -1158,7 +1158,7 @@ def vigodra_kernels(dtype, device, pk, tokens=2048):
     kc = torch.zeros(pages, kvh, page, kd, dtype=dtype, device=device)
     vc = torch.zeros(pages, kvh, page, vd, dtype=dtype, device=device)
     q = torch.empty(t, nqc, dtype=dtype, device=device)
-    bias, w_taps = torch.zeros(ch, device=device), torch.randn(ch, taps, device=device) * 0.5
+    bias, w_taps = torch.zeros(ch, device=device), torch.randn(taps, ch, device=device) * 0.5
     kept = torch.zeros(4, taps - 1, ch, device=device)
     wq, wk = torch.ones(nqc, device=device), torch.ones(nkc, device=device)
     mem("conv_norm_kv_write (biases, 4 taps, norms over all heads) + conv_state_update", time_kernel(lambda: ops.conv_norm_kv_write(

@@ -363,35 +363,39 @@ attention_maps_kernel(const MapsParams p) {
 }
 
 // Joins the runs of one row: with M the largest of the runs' maxima (and the sink), out = sum_s o_s 2^(m_s - M) /
-// (sum_s l_s 2^(m_s - M) + 2^(sink - M)), runs in ascending order.  One warp per row.
+// (sum_s l_s 2^(m_s - M) + 2^(sink - M)), runs in ascending order.  One CTA per row; lane s of every warp holds run s's
+// maximum and factor, a thread owns one value (or two) and asks for the runs' sums eight at a time.
+constexpr int MERGE_RUNS = 32;
 __global__ void __launch_bounds__(128) attention_maps_merge_kernel(const float* __restrict__ part, void* __restrict__ out,
-                                                                   int out_bf16, const float* __restrict__ sink, int total_rows, int splits,
-                                                                   int heads_maps, int maps) {
+                                                                   int out_bf16, const float* __restrict__ sink, int total_rows,
+                                                                   int splits, int heads_maps, int maps) {
+  __shared__ float factor[MERGE_RUNS];
   pdl_trigger();
   pdl_wait();
-  const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (row >= total_rows) return;
+  const int row = blockIdx.x, lane = threadIdx.x & 31;
   constexpr int LD = VD + 2;
-  float top = -CUDART_INF_F;
-  for (int s = 0; s < splits; ++s) top = fmaxf(top, part[((size_t)s * total_rows + row) * LD + VD]);
+  const float* src = part + (size_t)row * LD;
+  const size_t step = (size_t)total_rows * LD;
+  const bool has = lane < splits;
+  const float m = has ? src[lane * step + VD] : -CUDART_INF_F;
+  const float l = has ? src[lane * step + VD + 1] : 0.f;
+  float top = m;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
   float extra = 0.f;
   if (sink != nullptr) {
     const float sk = sink[(row % heads_maps) / maps] * 1.4426950408889634f;
     top = fmaxf(top, sk);
     extra = ex2(sk - top);
   }
-  float denom = 0.f;
-  for (int s = 0; s < splits; ++s) {
-    const float* src = part + ((size_t)s * total_rows + row) * LD;
-    denom = fmaf(src[VD + 1], ex2(src[VD] - top), denom);     // an empty run: 2^(-inf) = 0
-  }
-  const float inv = 1.f / (denom + extra);
-  for (int d = lane; d < VD; d += 32) {
+  const float f = has ? ex2(m - top) : 0.f;     // an empty run: 2^(-inf) = 0
+  if (threadIdx.x < 32) factor[lane] = f;
+  const float inv = 1.f / (warp_sum(l * f) + extra);
+  __syncthreads();
+  for (int d = threadIdx.x; d < VD; d += 128) {
     float acc = 0.f;
-    for (int s = 0; s < splits; ++s) {
-      const float* src = part + ((size_t)s * total_rows + row) * LD;
-      acc = fmaf(src[d], ex2(src[VD] - top), acc);
-    }
+#pragma unroll 8
+    for (int s = 0; s < splits; ++s) acc = fmaf(src[s * step + d], factor[s], acc);
     if (out_bf16) ((__nv_bfloat16*)out)[(size_t)row * VD + d] = __float2bfloat16_rn(acc * inv);
     else ((float*)out)[(size_t)row * VD + d] = acc * inv;
   }
@@ -408,7 +412,7 @@ extern "C" int tllm_attention_maps_mma(const void* q, int q_row_stride, const vo
                                        long long v_page_stride, long long v_head_stride, float scale, int window, int chunk,
                                        const float* sink, int splits, float* part, int keep, const float* rel, int rel_len,
                                        void* stream) {
-  TLLM_REQUIRE(splits >= 1 && splits <= 65535 && (splits == 1 || (part != nullptr && max_q_len * (nq / nkv) <= BM)),
+  TLLM_REQUIRE(splits >= 1 && splits <= MERGE_RUNS && (splits == 1 || (part != nullptr && max_q_len * (nq / nkv) <= BM)),
                "attention_maps_mma: %d runs of key tiles need a buffer and rows that fit one tile", splits);
   TLLM_REQUIRE(kd == KD && vd == VD, "attention_maps_mma: built for key size %d and value size %d, called with %d and %d", KD, VD, kd, vd);
   TLLM_REQUIRE(n_tokens > 0 && n_requests > 0 && max_q_len > 0 && nq > 0 && nkv > 0 && nq % nkv == 0 && maps > 0,
@@ -445,7 +449,7 @@ extern "C" int tllm_attention_maps_mma(const void* q, int q_row_stride, const vo
   if (rel != nullptr) TLLM_LAUNCH("attention_maps_mma", (attention_maps_kernel<ST, true>), grid, 128, smem, (cudaStream_t)stream, p);
   else TLLM_LAUNCH("attention_maps_mma", (attention_maps_kernel<ST, false>), grid, 128, smem, (cudaStream_t)stream, p);
   if (splits > 1)
-    TLLM_LAUNCH("attention_maps_merge", attention_maps_merge_kernel, dim3((unsigned)((p.total_rows + 3) / 4)), 128, 0,
+    TLLM_LAUNCH("attention_maps_merge", attention_maps_merge_kernel, dim3((unsigned)p.total_rows), 128, 0,
                 (cudaStream_t)stream, (const float*)part, out, out_bf16, sink, p.total_rows, splits, nq * maps, maps);
   return TLLM_OK;
 }

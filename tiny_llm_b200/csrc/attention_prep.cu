@@ -16,7 +16,7 @@
 //   latent in the key row, the query parts to q_out[t, head, rank : rank + rd].  (The plain query parts reach q_out through a product with the
 //   keys' up-projection, which is not this kernel's.)
 // conv_norm_kv_write: rows are [nq query heads | nkv key heads] of kd values, then nkv value heads of vd values, all of
-//   them channels of a short causal filter over time: y_t[c] = sum_j taps[c, j] x_(t - n_taps + 1 + j)[c] with x the
+//   them channels of a short causal filter over time: y_t[c] = sum_j taps[j, c] x_(t - n_taps + 1 + j)[c] with x the
 //   projection plus its bias, zero before the sequence's start; the last n_taps - 1 inputs of every channel are the
 //   request's state.  The filtered queries TOGETHER (all heads of the token) are divided by sqrt(mean(y^2) + eps) and
 //   multiplied by a weight per channel, and so are the keys.  Queries go to a buffer of their own (other tokens' filters
@@ -224,7 +224,7 @@ struct ConvArgs {
   const void* proj;             // [T, ld], channels [queries | keys | values] first
   int ld, nq, nkv, kd, vd;
   const float* bias;            // [channels] or null
-  const float* taps;            // [channels, n_taps]; null: no filter (n_taps = 1)
+  const float* taps;            // [n_taps, channels]; null: no filter (n_taps = 1)
   int n_taps;
   float* kept;                  // [slots, n_taps - 1, channels]: inputs of the tokens before this step, oldest first
   const int *slots, *cu_q, *token_request;
@@ -245,10 +245,12 @@ template <> struct __align__(16) Piece<__nv_bfloat16, 8> { __nv_bfloat16 v[8]; }
 
 // A CTA takes TOK consecutive tokens of the step with all their channels, V channels per thread and turn; the filtered
 // queries and keys wait in shared memory for their sums of squares.  NT: the number of taps (0: any).  Which thread meets
-// which channel depends on the sizes alone, so a token's sums have the same order in every batch.
+// which channel depends on the sizes alone, so a token's sums have the same order in every batch.  Where a tile's tokens
+// are one request's and their filters reach no kept input, the inputs of the tile are all asked for at once.
+constexpr int CONV_THREADS = 384;
 template <typename T, int V, int TOK, int NT>
-__global__ void conv_norm_kv_write_kernel(ConvArgs a) {
-  extern __shared__ float ys[];        // [TOK, (nq + nkv) * kd]
+__global__ void __launch_bounds__(CONV_THREADS) conv_norm_kv_write_kernel(ConvArgs a) {
+  extern __shared__ __align__(16) float ys[];        // [TOK, (nq + nkv) * kd]
   __shared__ float part[2 * TOK][33];
   pdl_trigger();
   const int nqc = a.nq * a.kd, nkc = a.nkv * a.kd, nvc = a.nkv * a.vd, channels = nqc + nkc + nvc, nqk = nqc + nkc;
@@ -259,26 +261,31 @@ __global__ void conv_norm_kv_write_kernel(ConvArgs a) {
   float ssq[TOK], ssk[TOK];
 #pragma unroll
   for (int i = 0; i < TOK; ++i) ssq[i] = ssk[i] = 0.f;
-  int first[TOK];
-  float* kept[TOK];
-  long long slot[TOK];
-#pragma unroll
-  for (int i = 0; i < TOK; ++i) {
-    const int t = min(t0 + i, a.n_tokens - 1);
-    const int req = a.token_request[t];
-    first[i] = a.cu_q[req];
-    kept[i] = taps_n > 1 ? a.kept + (size_t)a.slots[req] * (taps_n - 1) * channels : nullptr;
-    slot[i] = a.slot_mapping[t];
+  bool inside = false;
+  if (TOK > 1 && NT > 0 && t0 + TOK <= a.n_tokens) {
+    const int req = a.token_request[t0];
+    inside = req == a.token_request[t0 + TOK - 1] && t0 - a.cu_q[req] >= NT - 1;
   }
   for (int c = threadIdx.x * V; c < channels; c += blockDim.x * V) {
-    float w[NT ? NT * V : 1];
+    Piece<T, V> in[NT && TOK > 1 ? TOK + NT - 1 : 1];
+    if (inside) {
+#pragma unroll
+      for (int j = 0; j < (NT && TOK > 1 ? TOK + NT - 1 : 1); ++j)
+        in[j] = *reinterpret_cast<const Piece<T, V>*>(proj + (size_t)(t0 - (NT - 1) + j) * a.ld + c);
+    }
+    Piece<float, V> w[NT ? NT : 1];
     if (NT) {
 #pragma unroll
-      for (int j = 0; j < NT * V; ++j) w[j] = a.taps[(size_t)c * NT + j];
+      for (int j = 0; j < NT; ++j) w[j] = *reinterpret_cast<const Piece<float, V>*>(a.taps + (size_t)j * channels + c);
     }
-    float bias[V];
+    Piece<float, V> add;
+    if (a.bias) {
+      add = *reinterpret_cast<const Piece<float, V>*>(a.bias + c);
+    } else {
 #pragma unroll
-    for (int e = 0; e < V; ++e) bias[e] = a.bias ? a.bias[c + e] : 0.f;
+      for (int e = 0; e < V; ++e) add.v[e] = 0.f;
+    }
+    const float* bias = add.v;
 #pragma unroll
     for (int i = 0; i < TOK; ++i) {
       const int t = t0 + i;
@@ -286,47 +293,62 @@ __global__ void conv_norm_kv_write_kernel(ConvArgs a) {
       float y[V], x[V];
 #pragma unroll
       for (int e = 0; e < V; ++e) y[e] = 0.f;
+      if (inside) {
 #pragma unroll
-      for (int j = 0; j < taps_n; ++j) {
-        const int n = t - first[i] - (taps_n - 1) + j;   // index among the request's tokens of this step; < 0: kept ones
-        if (n >= 0) {
-          const Piece<T, V> p = *reinterpret_cast<const Piece<T, V>*>(proj + (size_t)(first[i] + n) * a.ld + c);
+        for (int j = 0; j < NT; ++j)
 #pragma unroll
-          for (int e = 0; e < V; ++e) x[e] = to_f32(p.v[e]) + bias[e];
-        } else {
-          const Piece<float, V> p = *reinterpret_cast<const Piece<float, V>*>(kept[i] + (size_t)(taps_n - 1 + n) * channels + c);
+          for (int e = 0; e < V; ++e)
+            y[e] = fmaf(w[NT ? j : 0].v[e], to_f32(in[NT && TOK > 1 ? i + j : 0].v[e]) + bias[e], y[e]);
+      } else {
+        const int req = a.token_request[t], first = a.cu_q[req];
+        float* kept = taps_n > 1 ? a.kept + (size_t)a.slots[req] * (taps_n - 1) * channels : nullptr;
 #pragma unroll
-          for (int e = 0; e < V; ++e) x[e] = p.v[e];
-          // the entry just read is the only reader's: what it holds next is the entry behind it
-          if (a.update && j > 0) *reinterpret_cast<Piece<float, V>*>(kept[i] + (size_t)(j - 1) * channels + c) = p;
+        for (int j = 0; j < taps_n; ++j) {
+          const int n = t - first - (taps_n - 1) + j;   // index among the request's tokens of this step; < 0: kept ones
+          if (n >= 0) {
+            const Piece<T, V> p = *reinterpret_cast<const Piece<T, V>*>(proj + (size_t)(first + n) * a.ld + c);
+#pragma unroll
+            for (int e = 0; e < V; ++e) x[e] = to_f32(p.v[e]) + bias[e];
+          } else {
+            const Piece<float, V> p = *reinterpret_cast<const Piece<float, V>*>(kept + (size_t)(taps_n - 1 + n) * channels + c);
+#pragma unroll
+            for (int e = 0; e < V; ++e) x[e] = p.v[e];
+            // this thread is the entry's only reader: what it holds next is the entry behind it
+            if (a.update && j > 0) *reinterpret_cast<Piece<float, V>*>(kept + (size_t)(j - 1) * channels + c) = p;
+          }
+#pragma unroll
+          for (int e = 0; e < V; ++e) {
+            const float f = NT ? w[NT ? j : 0].v[e] : (a.taps ? a.taps[(size_t)j * channels + c + e] : 1.f);
+            y[e] = fmaf(f, x[e], y[e]);
+          }
         }
+        if (a.update && taps_n > 1) {   // x is the token's own input now
+          Piece<float, V> p;
 #pragma unroll
-        for (int e = 0; e < V; ++e) {
-          const float f = NT ? w[e * (NT ? NT : 1) + (NT ? j : 0)] : (a.taps ? a.taps[(size_t)(c + e) * taps_n + j] : 1.f);
-          y[e] = fmaf(f, x[e], y[e]);
+          for (int e = 0; e < V; ++e) p.v[e] = x[e];
+          *reinterpret_cast<Piece<float, V>*>(kept + (size_t)(taps_n - 2) * channels + c) = p;
         }
-      }
-      if (a.update && taps_n > 1) {   // x is the token's own input now
-        Piece<float, V> p;
-#pragma unroll
-        for (int e = 0; e < V; ++e) p.v[e] = x[e];
-        *reinterpret_cast<Piece<float, V>*>(kept[i] + (size_t)(taps_n - 2) * channels + c) = p;
       }
       if (c >= nqk) {   // values have no norm
-        if (slot[i] < 0) continue;
+        const int slot = a.slot_mapping[t];
+        if (slot < 0) continue;
         const int h = (c - nqk) / a.vd, d = (c - nqk) % a.vd;
         Piece<T, V> p;
 #pragma unroll
         for (int e = 0; e < V; ++e) p.v[e] = from_f32<T>(y[e]);
-        *reinterpret_cast<Piece<T, V>*>((T*)a.vcache + slot[i] / a.page_size * a.v_page_stride + (long long)h * a.v_head_stride +
-                                        slot[i] % a.page_size * a.vd + d) = p;
+        *reinterpret_cast<Piece<T, V>*>((T*)a.vcache + (long long)(slot / a.page_size) * a.v_page_stride +
+                                        (long long)h * a.v_head_stride + (long long)(slot % a.page_size) * a.vd + d) = p;
         continue;
       }
       float ss = 0.f;
+      float* keep_y = ys + (size_t)i * nqk + c;
 #pragma unroll
-      for (int e = 0; e < V; ++e) {
-        ys[(size_t)i * nqk + c + e] = y[e];
-        ss = fmaf(y[e], y[e], ss);
+      for (int e = 0; e < V; ++e) ss = fmaf(y[e], y[e], ss);
+      if (V == 8) {
+        *reinterpret_cast<float4*>(keep_y) = make_float4(y[0], y[1 % V], y[2 % V], y[3 % V]);
+        *reinterpret_cast<float4*>(keep_y + 4) = make_float4(y[4 % V], y[5 % V], y[6 % V], y[7 % V]);
+      } else {
+        keep_y[0] = y[0];
       }
       if (c < nqc) ssq[i] += ss; else ssk[i] += ss;
     }
@@ -346,21 +368,39 @@ __global__ void conv_norm_kv_write_kernel(ConvArgs a) {
   for (int c = threadIdx.x * V; c < nqk; c += blockDim.x * V) {
     const bool is_q = c < nqc;
     const float* wn = is_q ? a.wq : a.wk;
-    float w[V];
+    Piece<float, V> w;
+    if (wn) {
+      w = *reinterpret_cast<const Piece<float, V>*>(wn + (is_q ? c : c - nqc));
+    } else {
 #pragma unroll
-    for (int e = 0; e < V; ++e) w[e] = wn ? wn[(is_q ? c : c - nqc) + e] : 1.f;
+      for (int e = 0; e < V; ++e) w.v[e] = 1.f;
+    }
     const int h = (c - nqc) / a.kd, d = (c - nqc) % a.kd;
 #pragma unroll
     for (int i = 0; i < TOK; ++i) {
       const int t = t0 + i;
-      if (t >= a.n_tokens || (!is_q && slot[i] < 0)) continue;
+      if (t >= a.n_tokens) continue;
+      T* dst;
+      if (is_q) {
+        dst = (T*)a.q_out + (size_t)t * nqc + c;
+      } else {
+        const int slot = a.slot_mapping[t];
+        if (slot < 0) continue;
+        dst = (T*)a.kcache + (long long)(slot / a.page_size) * a.k_page_stride + (long long)h * a.k_head_stride +
+              (long long)(slot % a.page_size) * a.kd + d;
+      }
       const float f = wn ? part[2 * i + (is_q ? 0 : 1)][32] : 1.f;
+      const float* keep_y = ys + (size_t)i * nqk + c;   // this thread wrote these values itself
+      float y[V];
+      if (V == 8) {
+        const float4 lo = *reinterpret_cast<const float4*>(keep_y), hi = *reinterpret_cast<const float4*>(keep_y + 4);
+        y[0] = lo.x; y[1 % V] = lo.y; y[2 % V] = lo.z; y[3 % V] = lo.w; y[4 % V] = hi.x; y[5 % V] = hi.y; y[6 % V] = hi.z; y[7 % V] = hi.w;
+      } else {
+        y[0] = keep_y[0];
+      }
       Piece<T, V> p;
 #pragma unroll
-      for (int e = 0; e < V; ++e) p.v[e] = from_f32<T>(__fmul_rn(__fmul_rn(ys[(size_t)i * nqk + c + e], f), w[e]));
-      T* dst = is_q ? (T*)a.q_out + (size_t)t * nqc + c
-                    : (T*)a.kcache + slot[i] / a.page_size * a.k_page_stride + (long long)h * a.k_head_stride +
-                          slot[i] % a.page_size * a.kd + d;
+      for (int e = 0; e < V; ++e) p.v[e] = from_f32<T>(__fmul_rn(__fmul_rn(y[e], f), w.v[e]));
       *reinterpret_cast<Piece<T, V>*>(dst) = p;
     }
   }
@@ -369,7 +409,7 @@ __global__ void conv_norm_kv_write_kernel(ConvArgs a) {
 template <typename T, int V, int TOK, int NT>
 static int launch_conv(const ConvArgs& a, cudaStream_t s) {
   const int channels = (a.nq + a.nkv) * a.kd + a.nkv * a.vd, pieces = channels / V;
-  const int threads = pieces >= 512 ? 512 : (pieces + 31) / 32 * 32;
+  const int threads = pieces >= CONV_THREADS ? CONV_THREADS : (pieces + 31) / 32 * 32;
   const size_t smem = (size_t)TOK * (a.nq + a.nkv) * a.kd * 4;
   static size_t configured = 48 * 1024;
   if (smem + 2 * TOK * 33 * 4 > configured) {
@@ -479,7 +519,7 @@ extern "C" int tllm_conv_norm_kv_write(const void* proj, int ld, int nq, int nkv
   a.v_head_stride = v_head_stride; a.n_tokens = n_tokens; a.update = update;
   const int esz = dtype == TLLM_F32 ? 4 : 2;
   const auto ok16 = [](const void* p) { return ((uintptr_t)p % 16) == 0; };
-  const bool vec = kd % 8 == 0 && vd % 8 == 0 && ok16(proj) && ok16(q_out) && ok16(kcache) && ok16(vcache) && ok16(kept) &&
+  const bool vec = kd % 8 == 0 && vd % 8 == 0 && ok16(proj) && ok16(q_out) && ok16(kcache) && ok16(vcache) && ok16(kept) && ok16(bias) && ok16(taps) && ok16(wq) && ok16(wk) &&
                    ((long long)ld * esz) % 16 == 0 && (k_page_stride * esz) % 16 == 0 && (k_head_stride * esz) % 16 == 0 &&
                    (v_page_stride * esz) % 16 == 0 && (v_head_stride * esz) % 16 == 0;
   cudaStream_t s = (cudaStream_t)stream;

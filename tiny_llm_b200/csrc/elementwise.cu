@@ -165,6 +165,32 @@ __global__ void silu_mul_kernel(TIn* __restrict__ gu, TOut* __restrict__ out, in
   }
 }
 
+// The same between bfloat16 rows, eight neighbouring outputs per thread (block and row multiples of eight values, the
+// rows 16-byte aligned).
+__global__ void __launch_bounds__(256) silu_mul_bf16x8_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ out,
+                                                              int m, int inter, int blk, int act, float limit) {
+  pdl_trigger();
+  pdl_wait();
+  const int per_row = inter >> 3;
+  const long long total = (long long)m * per_row;
+  for (long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (long long)gridDim.x * blockDim.x) {
+    const int row = (int)(idx / per_row), col = (int)(idx - (long long)row * per_row) << 3;
+    const int g = col / blk, j = col - g * blk;
+    const __nv_bfloat16* src = gu + (size_t)row * 2 * inter + (size_t)g * 2 * blk + j;
+    const uint4 gv = *reinterpret_cast<const uint4*>(src), uv = *reinterpret_cast<const uint4*>(src + blk);
+    const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gv);
+    const __nv_bfloat162* u2 = reinterpret_cast<const __nv_bfloat162*>(&uv);
+    uint4 pk;
+    __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&pk);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 a = __bfloat1622float2(g2[i]), b = __bfloat1622float2(u2[i]);
+      o2[i] = __floats2bfloat162_rn(glu_value(a.x, b.x, act, limit), glu_value(a.y, b.y, act, limit));
+    }
+    *reinterpret_cast<uint4*>(out + (size_t)row * inter + col) = pk;
+  }
+}
+
 // The same from float32 sums, four neighbouring outputs per thread (the block and the row are multiples of four values
 // and the rows 16-byte aligned): two 16-byte loads, one store.  ZERO hands the sums back cleared.
 template <typename TOut, bool ZERO>
@@ -654,6 +680,12 @@ extern "C" int tllm_silu_mul(void* gu, void* out, int m, int inter, int blk, int
     else if (out_dtype == TLLM_F32) TLLM_LAUNCH("silu_mul", (silu_mul_f32x4_kernel<float, false>), vblocks, threads, 0, s, (float*)gu, (float*)out, m, inter, blk, act, limit);
     else if (zero_src) TLLM_LAUNCH("silu_mul", (silu_mul_f32x4_kernel<__nv_bfloat16, true>), vblocks, threads, 0, s, (float*)gu, (__nv_bfloat16*)out, m, inter, blk, act, limit);
     else TLLM_LAUNCH("silu_mul", (silu_mul_f32x4_kernel<__nv_bfloat16, false>), vblocks, threads, 0, s, (float*)gu, (__nv_bfloat16*)out, m, inter, blk, act, limit);
+    return TLLM_OK;
+  }
+  if (in_dtype == TLLM_BF16 && out_dtype == TLLM_BF16 && !zero_src && blk % 8 == 0 && ((uintptr_t)gu % 16) == 0 && ((uintptr_t)out % 16) == 0) {
+    const size_t pieces = total / 8;
+    const int vblocks = (int)((pieces + threads - 1) / threads < 148 * 16 ? (pieces + threads - 1) / threads : 148 * 16);
+    TLLM_LAUNCH("silu_mul", silu_mul_bf16x8_kernel, vblocks, threads, 0, s, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, m, inter, blk, act, limit);
     return TLLM_OK;
   }
   if (in_dtype == TLLM_F32 && out_dtype == TLLM_F32 && !zero_src)

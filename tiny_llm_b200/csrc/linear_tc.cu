@@ -41,11 +41,25 @@ enum Epilogue { EPI_BF16 = 0, EPI_F32 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU = 3, EPI_
                 EPI_CL_ADD_F32 = 5, EPI_CL_ROPE_KV = 6, EPI_CL_SWIGLU = 7, EPI_CL_BF16 = 8,
                 // NORMAL orientation: Q/K/V projection with rotation and cache write (head size 64 or 128)
                 EPI_ROPE_KV = 9,
-                EPI_GELU_BF16 = 10 };   // bfloat16 store of the exact GELU of the sums (the grouped expert product)
+                EPI_GELU_BF16 = 10,    // bfloat16 store of the exact GELU of the sums (the grouped expert product)
+                EPI_GLU_CLAMPED = 11 };   // like EPI_SWIGLU with the clamped gate (glu_f)
 
 constexpr int ERR_PRODUCER = 1, ERR_MMA = 2, ERR_EPILOGUE = 3;
 
-__device__ __forceinline__ float silu_f(float x) { return x / (1.f + __expf(-x)); }
+__device__ __forceinline__ float silu_f(float x) { return __fdividef(x, 1.f + __expf(-x)); }
+
+// What the gate/up epilogues store: SiLU(g) u, or, clamped, with g <- min(g, limit) and u <- clamp(u, -limit, limit),
+// g sigmoid(1.702 g) (u + 1).
+constexpr bool is_glu(int epi) { return epi == EPI_SWIGLU || epi == EPI_GLU_CLAMPED; }
+__device__ __forceinline__ float clamped_glu_f(float g, float u, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return __fdividef(g * (u + 1.f), 1.f + __expf(-1.702f * g));
+}
+template <int EPI>
+__device__ __forceinline__ float glu_f(float g, float u, float limit) {
+  return EPI == EPI_GLU_CLAMPED ? clamped_glu_f(g, u, limit) : silu_f(g) * u;
+}
 
 template <int BN, int STAGES>
 struct SmemLayout {
@@ -78,6 +92,9 @@ struct ClusterArgs {
   // every role), whose weights are rows [expert * expert_rows, +rows_b) of the stacked B matrix (null: one B for all)
   const int* tile_expert;
   int expert_rows;
+  // gate/up epilogues: the clamped gate's limit; the cluster kernel's gate: 0 SiLU, 1 clamped
+  float limit;
+  int clamped;
 };
 
 // Epilogue of one 128 x BN tile of C in the NORMAL orientation: this thread owns row `row` of the
@@ -156,12 +173,12 @@ __device__ __forceinline__ void store_tile_rope_kv(uint32_t taddr, int m, int n_
 
 template <int BN, int EPI>
 __device__ __forceinline__ void store_tile_normal(uint32_t taddr, int row, int tile_a, int tile_b, int rows_a,
-                                                  int rows_b, void* __restrict__ out, int ldo) {
+                                                  int rows_b, void* __restrict__ out, int ldo, float limit = 0.f) {
   // 16-byte stores need an aligned base and row stride
   const bool vec_ok = (reinterpret_cast<uintptr_t>(out) & 15) == 0 &&
-                      ((EPI == EPI_BF16 || EPI == EPI_GELU_BF16 || EPI == EPI_SWIGLU) ? (ldo & 7) == 0 : (ldo & 3) == 0);
+                      ((EPI == EPI_BF16 || EPI == EPI_GELU_BF16 || is_glu(EPI)) ? (ldo & 7) == 0 : (ldo & 3) == 0);
   const int m = tile_a * BM + row;
-  if (EPI == EPI_SWIGLU) {
+  if (is_glu(EPI)) {
     // columns [0, BN/2) are gate, [BN/2, BN) the matching up columns; output tile is BN/2 wide
     const int n0 = tile_b * (BN / 2);
     const int n_out = rows_b / 2;
@@ -179,13 +196,13 @@ __device__ __forceinline__ void store_tile_normal(uint32_t taddr, int row, int t
             __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&pk);
 #pragma unroll
             for (int e = 0; e < 4; ++e)
-              h[e] = __floats2bfloat162_rn(silu_f(g[j + 2 * e]) * u[j + 2 * e], silu_f(g[j + 2 * e + 1]) * u[j + 2 * e + 1]);
+              h[e] = __floats2bfloat162_rn(glu_f<EPI>(g[j + 2 * e], u[j + 2 * e], limit), glu_f<EPI>(g[j + 2 * e + 1], u[j + 2 * e + 1], limit));
             *reinterpret_cast<uint4*>(dst + j) = pk;
           }
         } else {
 #pragma unroll
           for (int j = 0; j < 32; ++j)
-            if (n0 + c + j < n_out) dst[j] = __float2bfloat16_rn(silu_f(g[j]) * u[j]);
+            if (n0 + c + j < n_out) dst[j] = __float2bfloat16_rn(glu_f<EPI>(g[j], u[j], limit));
         }
       }
     }
@@ -247,8 +264,9 @@ __device__ __forceinline__ void store_tile_normal(uint32_t taddr, int row, int t
 
 // SiLU(gate) * up for a STRIP of a gate/up tile: the accumulator holds `w` gate columns and, behind them, the `w`
 // matching up columns; the strip's results go to output columns [out_col, out_col + w).  This thread owns row m.
+template <int EPI>
 __device__ __forceinline__ void store_strip_swiglu(uint32_t taddr, int m, int out_col, int w, int rows_a, int n_out,
-                                                   __nv_bfloat16* __restrict__ out, int ldo) {
+                                                   __nv_bfloat16* __restrict__ out, int ldo, float limit) {
   const bool vec_ok = (reinterpret_cast<uintptr_t>(out) & 15) == 0 && (ldo & 7) == 0;
 #pragma unroll 1
   for (int c = 0; c < w; c += 32) {
@@ -264,13 +282,13 @@ __device__ __forceinline__ void store_strip_swiglu(uint32_t taddr, int m, int ou
           __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&pk);
 #pragma unroll
           for (int e = 0; e < 4; ++e)
-            h[e] = __floats2bfloat162_rn(silu_f(g[j + 2 * e]) * u[j + 2 * e], silu_f(g[j + 2 * e + 1]) * u[j + 2 * e + 1]);
+            h[e] = __floats2bfloat162_rn(glu_f<EPI>(g[j + 2 * e], u[j + 2 * e], limit), glu_f<EPI>(g[j + 2 * e + 1], u[j + 2 * e + 1], limit));
           *reinterpret_cast<uint4*>(dst + j) = pk;
         }
       } else {
 #pragma unroll
         for (int j = 0; j < 32; ++j)
-          if (out_col + c + j < n_out) dst[j] = __float2bfloat16_rn(silu_f(g[j]) * u[j]);
+          if (out_col + c + j < n_out) dst[j] = __float2bfloat16_rn(glu_f<EPI>(g[j], u[j], limit));
       }
     }
   }
@@ -628,7 +646,8 @@ linear_tc_cluster_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
 #pragma unroll
       for (int e = 0; e < 4; ++e)
         if (2 * col0 + BM + r + e < rows_a)   // the matching up row exists
-          dst[e] = __float2bfloat16_rn((gate[e] / (1.f + expf(-gate[e]))) * up[e]);
+          dst[e] = __float2bfloat16_rn(ca.clamped ? clamped_glu_f(gate[e], up[e], ca.limit)
+                                                  : (gate[e] / (1.f + expf(-gate[e]))) * up[e]);
     }
   } else if (EPI == EPI_CL_ROPE_KV) {
     // pairs (d, d + hd/2) of whole heads: 64 pairs per tile, dealt to the CZ CTAs, four neighbouring pairs per item
@@ -775,7 +794,7 @@ linear_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const __g
   auto item_kbn = [&](int i) { return k_splits > 1 ? max(0, min(k_blocks, (i / n_tiles + 1) * k_per) - (i / n_tiles) * k_per) : k_blocks; };
   // (a strip of a gate/up tile: tail_width / 2 gate rows from item_col on, and the matching up rows BN / 2 further on)
   auto item_col = [&](int i) {
-    return (item_tile(i) / tiles_m) * BN + (i < whole ? 0 : ((i - whole) % strips) * (EPI == EPI_SWIGLU ? ca.tail_width / 2 : ca.tail_width));
+    return (item_tile(i) / tiles_m) * BN + (i < whole ? 0 : ((i - whole) % strips) * (is_glu(EPI) ? ca.tail_width / 2 : ca.tail_width));
   };
   auto item_width = [&](int i) { return i < whole ? BN : ca.tail_width; };
   // grouped product: the expert of an item's row tile (read after the wait for earlier kernels, which write the list)
@@ -826,7 +845,7 @@ linear_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const __g
         if (!pre) {
           if (!mbar_wait(&empty_bar[s], ((it / STAGES) & 1) ^ 1, abort_flag)) { *abort_flag = 1; atomicExch(status, ERR_PRODUCER); ok = false; break; }
           mbar_expect_tx(&full_bar[s], (uint32_t)(L::A_BYTES + width * BK * 2));
-          if (EPI == EPI_SWIGLU && width != BN) {   // the strip's gate rows, then its up rows behind them
+          if (is_glu(EPI) && width != BN) {   // the strip's gate rows, then its up rows behind them
             tma_load_2d(a_dst + L::A_BYTES, &map_b_strip, kb * BK, col, &full_bar[s]);
             tma_load_2d(a_dst + L::A_BYTES + (width / 2) * BK * 2, &map_b_strip, kb * BK, col + BN / 2, &full_bar[s]);
           } else {
@@ -914,11 +933,11 @@ linear_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const __g
           }
         }
       }
-      else if (EPI == EPI_SWIGLU && item_width(t) != BN)
-        store_strip_swiglu(taddr, (item_tile(t) % tiles_m) * BM + row,
+      else if (is_glu(EPI) && item_width(t) != BN)
+        store_strip_swiglu<EPI>(taddr, (item_tile(t) % tiles_m) * BM + row,
                            (item_tile(t) / tiles_m) * (BN / 2) + (item_col(t) - (item_tile(t) / tiles_m) * BN), item_width(t) / 2,
-                           rows_a, rows_b / 2, reinterpret_cast<__nv_bfloat16*>(out), ldo);
-      else store_tile_normal<BN, EPI>(taddr, row, item_tile(t) % tiles_m, item_tile(t) / tiles_m, rows_a, rows_b, out, ldo);
+                           rows_a, rows_b / 2, reinterpret_cast<__nv_bfloat16*>(out), ldo, ca.limit);
+      else store_tile_normal<BN, EPI>(taddr, row, item_tile(t) % tiles_m, item_tile(t) / tiles_m, rows_a, rows_b, out, ldo, ca.limit);
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&acc_empty[buf]);   // four arrivals free the accumulator
@@ -1051,7 +1070,7 @@ static int launch_persistent(const CUtensorMap& ma, const CUtensorMap& mb, void*
       strip_map = &ms;
     }
   }
-  if (EPI == EPI_SWIGLU && tiles > sm_count && tiles % sm_count != 0 && w_ptr != nullptr && n % BN == 0) {
+  if (is_glu(EPI) && tiles > sm_count && tiles % sm_count != 0 && w_ptr != nullptr && n % BN == 0) {
     // gate/up: the tiles of the incomplete last round as 4 or 2 strips (32 or 64 gate columns with their up columns),
     // as many as still fit one round
     const int left = tiles % sm_count;
@@ -1105,7 +1124,8 @@ using namespace tllm;
 
 // out[M, N] (row stride ldo) = / += a[M, K] (row stride lda) . w[N, K]^T, bfloat16 operands.
 //   epi: 0 store bfloat16, 1 store float32, 2 add into float32, 3 SiLU(gate)*up with gate/up rows of w
-//        interleaved in blocks of 128 (out is [M, N/2] bfloat16), 4 atomic add into float32.
+//        interleaved in blocks of 128 (out is [M, N/2] bfloat16), 4 atomic add into float32, 11 the same as 3
+//        with the clamped gate and its `limit`.
 //   swap: 0 = 128 x 256 tiles of C per CTA (large M); 1 = weights on the 128-row side, M <= 128,
 //        `splits` slices of K per weight tile (epi 4 when splits > 1).
 // `status` is a device int that receives a non-zero code if a bounded wait expired.
@@ -1134,7 +1154,7 @@ extern "C" int tllm_linear_tc_grouped(const void* a, const void* w, void* out, i
 }
 
 extern "C" int tllm_linear_tc(const void* a, const void* w, void* out, int m, int n, int k, int lda, int ldo, int epi,
-                              int swap, int splits, int* status, void* stream) {
+                              int swap, int splits, float limit, int* status, void* stream) {
   TLLM_REQUIRE(m > 0 && n > 0 && k > 0, "linear_tc: empty product %d x %d x %d", m, n, k);
   TLLM_REQUIRE(k % 8 == 0 && lda % 8 == 0, "linear_tc: K (%d) and the row stride of A (%d) must be multiples of 8 (16-byte rule of TMA)", k, lda);
   TLLM_REQUIRE(((uintptr_t)a % 16) == 0 && ((uintptr_t)w % 16) == 0, "linear_tc: operands must be 16-byte aligned");
@@ -1144,7 +1164,7 @@ extern "C" int tllm_linear_tc(const void* a, const void* w, void* out, int m, in
   if (!swap) {
     TLLM_REQUIRE(splits == 1, "linear_tc: K is split only in the swapped orientation");
     TLLM_REQUIRE(epi != EPI_ATOMIC_F32, "linear_tc: atomic output belongs to the swapped orientation");
-    if (epi == EPI_SWIGLU) TLLM_REQUIRE(n % 256 == 0, "linear_tc: the fused SiLU*up epilogue needs gate/up blocks of 128 rows (N = %d)", n);
+    if (is_glu(epi)) TLLM_REQUIRE(n % 256 == 0, "linear_tc: the fused SiLU*up epilogue needs gate/up blocks of 128 rows (N = %d)", n);
     if (!make_map(&ma, a, m, k, lda, BM) || !make_map(&mb, w, n, k, k, 256))
       TLLM_FAIL(TLLM_ERR_CUDA, "linear_tc: cuTensorMapEncodeTiled failed");
     switch (epi) {
@@ -1152,11 +1172,16 @@ extern "C" int tllm_linear_tc(const void* a, const void* w, void* out, int m, in
       case EPI_F32: return launch_persistent<EPI_F32>(ma, mb, out, m, n, k, ldo, status, s);
       case EPI_ADD_F32: return launch_persistent<EPI_ADD_F32>(ma, mb, out, m, n, k, ldo, status, s);
       case EPI_SWIGLU: return launch_persistent<EPI_SWIGLU>(ma, mb, out, m, n, k, ldo, status, s, ClusterArgs(), w);
+      case EPI_GLU_CLAMPED: {
+        ClusterArgs ca = ClusterArgs();
+        ca.limit = limit;
+        return launch_persistent<EPI_GLU_CLAMPED>(ma, mb, out, m, n, k, ldo, status, s, ca, w);
+      }
     }
     TLLM_FAIL(TLLM_ERR_ARG, "linear_tc: unknown epilogue %d", epi);
   }
   TLLM_REQUIRE(m <= 128, "linear_tc: the swapped orientation takes at most 128 rows of A (got %d)", m);
-  TLLM_REQUIRE(epi != EPI_SWIGLU, "linear_tc: SiLU*up is fused only in the unswapped orientation");
+  TLLM_REQUIRE(!is_glu(epi), "linear_tc: SiLU*up is fused only in the unswapped orientation");
   TLLM_REQUIRE(splits >= 1 && (splits == 1 || epi == EPI_ATOMIC_F32), "linear_tc: split K needs the atomic epilogue");
   const int bn = m <= 16 ? 16 : (m <= 32 ? 32 : (m <= 64 ? 64 : 128));
   if (!make_map(&ma, w, n, k, k, BM) || !make_map(&mb, a, m, k, lda, bn))
@@ -1189,13 +1214,13 @@ extern "C" int tllm_linear_tc(const void* a, const void* w, void* out, int m, in
 //      hd 16, 32, 64 or 128; cos/sin null: no rotation.  This one also takes more than 128 rows (head size
 //      64 or 128): then it runs as 128 x 256 tiles of C with the same epilogue per tile;
 //   7: SiLU(gate) * up with gate/up rows of w interleaved in blocks of 128, out bfloat16 [M, N/2]
-//      (slices <= 4: the cluster also spans the gate tile and the up tile);
+//      (slices <= 4: the cluster also spans the gate tile and the up tile); with `limit` > 0 the clamped gate instead;
 //   8: out (bfloat16 [M, N]) = product.
 extern "C" int tllm_linear_tc_cluster(const void* a, const void* w, void* out, int m, int n, int k, int lda, int ldo,
                                       int epi, int slices, const int* positions, const float* cos, const float* sin,
                                       int nq, int nkv, int hd, void* kcache, void* vcache, const int* slot_mapping,
-                                      int page_size, long long page_stride, long long head_stride, int* status,
-                                      void* stream) {
+                                      int page_size, long long page_stride, long long head_stride, float limit,
+                                      int* status, void* stream) {
   TLLM_REQUIRE(m > 0 && n > 0 && k > 0 && (m <= 128 || epi == EPI_CL_ROPE_KV),
                "linear_tc_cluster: product %d x %d x %d (at most 128 rows, except for the Q/K/V projection)", m, n, k);
   TLLM_REQUIRE(k % 8 == 0 && lda % 8 == 0, "linear_tc_cluster: K (%d) and the row stride of A (%d) must be multiples of 8", k, lda);
@@ -1205,6 +1230,7 @@ extern "C" int tllm_linear_tc_cluster(const void* a, const void* w, void* out, i
   TLLM_REQUIRE(slices <= (k + BK - 1) / BK, "linear_tc_cluster: %d slices of a K of %d", slices, k);
   ClusterArgs ca = {};
   ca.cy = 1; ca.cz = slices;
+  ca.limit = limit; ca.clamped = limit > 0.f;
   if (epi == EPI_CL_SWIGLU) {
     TLLM_REQUIRE(n % 256 == 0 && slices <= 4, "linear_tc_cluster: SiLU*up needs gate/up blocks of 128 rows (N = %d) and at most 4 slices", n);
     ca.cy = 2;

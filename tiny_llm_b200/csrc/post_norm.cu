@@ -38,10 +38,55 @@ __device__ __forceinline__ float4 fma4(float s, float4 v, float4 a) {
   return make_float4(fmaf(s, v.x, a.x), fmaf(s, v.y, a.y), fmaf(s, v.z, a.z), fmaf(s, v.w, a.w));
 }
 
+// Mean of a row of 4 * n4 values that the block holds in registers (thread t's i-th piece is piece t + i * blockDim; pieces
+// past the row are zero) and its summed squared deviations, with ONE barrier: every warp takes those of its own values
+// (shuffles only), and the warps' pairs are joined by
+//   mean = sum_w n_w mean_w / N,   M2 = sum_w (M2_w + n_w (mean_w - mean)^2).
+template <int VEC>
+__device__ __forceinline__ void row_moments(const float4* z, int n4, float2* moments, float* counts, float& mean, float& m2) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  float sum = 0.f, count = 0.f;
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    sum += (z[i].x + z[i].y) + (z[i].z + z[i].w);
+    count += 4.f * fminf(32.f, fmaxf(0.f, (float)(n4 - (warp * 32 + i * (int)blockDim.x))));
+  }
+  const float own_mean = count > 0.f ? warp_sum(sum) / count : 0.f;
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    if (threadIdx.x + i * blockDim.x < n4) {
+      const float dx = z[i].x - own_mean, dy = z[i].y - own_mean, dz = z[i].z - own_mean, dw = z[i].w - own_mean;
+      ss += (dx * dx + dy * dy) + (dz * dz + dw * dw);
+    }
+  }
+  ss = warp_sum(ss);
+  if (lane == 0) { moments[warp] = make_float2(own_mean, ss); counts[warp] = count; }
+  __syncthreads();
+  const bool has = lane < (int)(blockDim.x >> 5);
+  const float2 pair = has ? moments[lane] : make_float2(0.f, 0.f);
+  const float cnt = has ? counts[lane] : 0.f;
+  mean = warp_sum(cnt * pair.x) / (4.f * (float)n4);
+  const float off = pair.x - mean;
+  m2 = warp_sum(fmaf(cnt * off, off, pair.y));
+}
+
+__device__ __forceinline__ void put4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void put4(__nv_bfloat16* p, float4 v) {
+  uint2 pk;
+  *reinterpret_cast<__nv_bfloat162*>(&pk.x) = __floats2bfloat162_rn(v.x, v.y);
+  *reinterpret_cast<__nv_bfloat162*>(&pk.y) = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = pk;
+}
+
+// The threads of a row depend on the width alone, so that a row's sums have the same order in every batch.
+inline int row_threads(int n4) { return n4 <= 128 ? (n4 + 31) / 32 * 32 : (n4 <= 512 ? 256 : 512); }
+
 // Rows in registers: hidden a multiple of 4, at most 4 * VEC * blockDim.
 template <int VEC>
 __global__ void post_norm_join_vec_kernel(JoinArgs a) {
-  __shared__ float scratch[33];
+  __shared__ float2 moments[32];
+  __shared__ float counts[32];
   pdl_trigger();
   const int n4 = a.hidden / 4, r = blockIdx.x;
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -55,18 +100,12 @@ __global__ void post_norm_join_vec_kernel(JoinArgs a) {
   if (r >= a.n_rows) return;
   float4* br = reinterpret_cast<float4*>(a.branch + (size_t)r * a.hidden);
   float4* xr = reinterpret_cast<float4*>(a.x + (size_t)r * a.hidden);
-  float4 z[VEC], acc[VEC];
-  float sum = 0.f;
+  float4 z[VEC], acc[VEC], v[VEC];
 #pragma unroll
   for (int i = 0; i < VEC; ++i) {
     const int idx = threadIdx.x + i * blockDim.x;
-    z[i] = zero;
-    if (idx < n4) {
-      const float4 v = br[idx];
-      z[i] = fma4(a.alpha, xr[idx], make_float4(v.x + ob[i].x, v.y + ob[i].y, v.z + ob[i].z, v.w + ob[i].w));
-      br[idx] = zero;
-    }
-    sum += (z[i].x + z[i].y) + (z[i].z + z[i].w);
+    v[i] = idx < n4 ? br[idx] : zero;
+    z[i] = idx < n4 ? xr[idx] : zero;
     acc[i] = zero;
   }
   if (a.stages != nullptr) {
@@ -81,17 +120,13 @@ __global__ void post_norm_join_vec_kernel(JoinArgs a) {
       }
     }
   }
-  const float mean = block_sum(sum, scratch) / (float)a.hidden;
-  float ss = 0.f;
 #pragma unroll
   for (int i = 0; i < VEC; ++i) {
-    if (threadIdx.x + i * blockDim.x < n4) {
-      z[i] = make_float4(z[i].x - mean, z[i].y - mean, z[i].z - mean, z[i].w - mean);
-      ss += (z[i].x * z[i].x + z[i].y * z[i].y) + (z[i].z * z[i].z + z[i].w * z[i].w);
-    }
+    z[i] = fma4(a.alpha, z[i], make_float4(v[i].x + ob[i].x, v[i].y + ob[i].y, v[i].z + ob[i].z, v[i].w + ob[i].w));
   }
-  ss = block_sum(ss, scratch);
-  const float inv = 1.f / sqrtf(ss / (float)a.hidden + a.eps);
+  float mean, m2;
+  row_moments<VEC>(z, n4, moments, counts, mean, m2);
+  const float inv = 1.f / sqrtf(m2 / (float)a.hidden + a.eps);
   const float last = a.stages != nullptr ? a.mix[a.n_stages] : 0.f;
   float4* own = a.stages != nullptr ? reinterpret_cast<float4*>(a.stages + a.n_stages * a.stage_stride + (size_t)r * a.hidden) : nullptr;
 #pragma unroll
@@ -99,18 +134,15 @@ __global__ void post_norm_join_vec_kernel(JoinArgs a) {
     const int idx = threadIdx.x + i * blockDim.x;
     if (idx >= n4) continue;
     const float4 w = __ldg(reinterpret_cast<const float4*>(a.w) + idx), b = __ldg(reinterpret_cast<const float4*>(a.b) + idx);
-    float4 y = make_float4(fmaf(z[i].x * inv, w.x, b.x), fmaf(z[i].y * inv, w.y, b.y), fmaf(z[i].z * inv, w.z, b.z), fmaf(z[i].w * inv, w.w, b.w));
+    float4 y = make_float4(fmaf((z[i].x - mean) * inv, w.x, b.x), fmaf((z[i].y - mean) * inv, w.y, b.y),
+                           fmaf((z[i].z - mean) * inv, w.z, b.z), fmaf((z[i].w - mean) * inv, w.w, b.w));
     if (own != nullptr) {
       if (a.keep) own[idx] = y;
       y = fma4(last, y, acc[i]);
     }
     xr[idx] = y;
-    if (a.copy != nullptr) {
-      uint2 pk;
-      *reinterpret_cast<__nv_bfloat162*>(&pk.x) = __floats2bfloat162_rn(y.x, y.y);
-      *reinterpret_cast<__nv_bfloat162*>(&pk.y) = __floats2bfloat162_rn(y.z, y.w);
-      reinterpret_cast<uint2*>(a.copy + (size_t)r * a.hidden)[idx] = pk;
-    }
+    br[idx] = zero;
+    if (a.copy != nullptr) put4(a.copy + (size_t)r * a.hidden + 4 * idx, y);
   }
 }
 
@@ -150,6 +182,35 @@ __global__ void post_norm_join_kernel(JoinArgs a) {
     }
     xr[i] = y;
     if (a.copy) a.copy[(size_t)r * a.hidden + i] = __float2bfloat16_rn(y);
+  }
+}
+
+template <typename T, int VEC>
+__global__ void layer_norm_vec_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ b,
+                                      T* __restrict__ out, const int* __restrict__ rows, int n_rows, int hidden, float eps) {
+  __shared__ float2 moments[32];
+  __shared__ float counts[32];
+  pdl_trigger();
+  pdl_wait();
+  const int r = blockIdx.x, n4 = hidden / 4;
+  if (r >= n_rows) return;
+  const float4* src = reinterpret_cast<const float4*>(x + (size_t)(rows ? rows[r] : r) * hidden);
+  float4 z[VEC];
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    const int idx = threadIdx.x + i * blockDim.x;
+    z[i] = idx < n4 ? src[idx] : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  float mean, m2;
+  row_moments<VEC>(z, n4, moments, counts, mean, m2);
+  const float inv = 1.f / sqrtf(m2 / (float)hidden + eps);
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    const int idx = threadIdx.x + i * blockDim.x;
+    if (idx >= n4) continue;
+    const float4 wv = __ldg(reinterpret_cast<const float4*>(w) + idx), bv = __ldg(reinterpret_cast<const float4*>(b) + idx);
+    put4(out + (size_t)r * hidden + 4 * idx, make_float4(fmaf((z[i].x - mean) * inv, wv.x, bv.x), fmaf((z[i].y - mean) * inv, wv.y, bv.y),
+                                                          fmaf((z[i].z - mean) * inv, wv.z, bv.z), fmaf((z[i].w - mean) * inv, wv.w, bv.w)));
   }
 }
 
@@ -219,9 +280,7 @@ extern "C" int tllm_post_norm_join(float* branch, float* x, const float* out_bia
   const auto off = [](const void* p, int to) { return ((uintptr_t)p % to) != 0; };
   if (hidden % 4 == 0 && hidden <= 4 * 4 * 512 && !off(branch, 16) && !off(x, 16) && !off(out_bias, 16) && !off(w, 16) && !off(b, 16) &&
       !off(copy_bf16, 8) && !off(stages, 16) && stage_stride % 4 == 0) {
-    // the threads depend on the width alone, so that a row's sums have the same order in every batch
-    const int n4 = hidden / 4;
-    const int threads = n4 <= 128 ? (n4 + 31) / 32 * 32 : (n4 <= 512 ? 256 : 512);
+    const int n4 = hidden / 4, threads = row_threads(n4);
     const int vec = (n4 + threads - 1) / threads;
     if (vec <= 1) TLLM_LAUNCH("post_norm_join", post_norm_join_vec_kernel<1>, n_rows, threads, 0, s, a);
     else if (vec == 2) TLLM_LAUNCH("post_norm_join", post_norm_join_vec_kernel<2>, n_rows, threads, 0, s, a);
@@ -234,15 +293,30 @@ extern "C" int tllm_post_norm_join(float* branch, float* x, const float* out_bia
   return TLLM_OK;
 }
 
+template <typename T>
+static int launch_layer_norm(const float* x, const float* w, const float* b, T* out, const int* rows, int n_rows, int hidden,
+                             float eps, cudaStream_t s) {
+  const auto aligned = [](const void* p) { return ((uintptr_t)p % 16) == 0; };
+  if (hidden % 4 == 0 && hidden <= 4 * 4 * 512 && aligned(x) && aligned(w) && aligned(b) && aligned(out)) {
+    const int n4 = hidden / 4, threads = row_threads(n4), vec = (n4 + threads - 1) / threads;
+    if (vec <= 1) TLLM_LAUNCH("layer_norm", (layer_norm_vec_kernel<T, 1>), n_rows, threads, 0, s, x, w, b, out, rows, n_rows, hidden, eps);
+    else if (vec == 2) TLLM_LAUNCH("layer_norm", (layer_norm_vec_kernel<T, 2>), n_rows, threads, 0, s, x, w, b, out, rows, n_rows, hidden, eps);
+    else TLLM_LAUNCH("layer_norm", (layer_norm_vec_kernel<T, 4>), n_rows, threads, 0, s, x, w, b, out, rows, n_rows, hidden, eps);
+    return TLLM_OK;
+  }
+  TLLM_REQUIRE(hidden <= MAX_WIDTH, "layer_norm: rows of %d values (at most %d)", hidden, MAX_WIDTH);
+  const int threads = hidden >= 2048 ? 512 : (hidden >= 512 ? 256 : 128);
+  TLLM_LAUNCH("layer_norm", layer_norm_kernel<T>, n_rows, threads, hidden * 4, s, x, w, b, out, rows, n_rows, hidden, eps);
+  return TLLM_OK;
+}
+
 extern "C" int tllm_layer_norm(const float* x, const float* w, const float* b, void* out, const int* rows, int n_rows,
                                int hidden, float eps, int out_dtype, void* stream) {
-  TLLM_REQUIRE(n_rows > 0 && hidden > 0 && hidden <= MAX_WIDTH, "layer_norm: %d rows of %d values (at most %d)", n_rows, hidden, MAX_WIDTH);
-  const int threads = hidden >= 2048 ? 512 : (hidden >= 512 ? 256 : 128);
+  TLLM_REQUIRE(n_rows > 0 && hidden > 0, "layer_norm: %d rows of %d values", n_rows, hidden);
   cudaStream_t s = (cudaStream_t)stream;
-  if (out_dtype == TLLM_F32) TLLM_LAUNCH("layer_norm", layer_norm_kernel<float>, n_rows, threads, hidden * 4, s, x, w, b, (float*)out, rows, n_rows, hidden, eps);
-  else if (out_dtype == TLLM_BF16) TLLM_LAUNCH("layer_norm", layer_norm_kernel<__nv_bfloat16>, n_rows, threads, hidden * 4, s, x, w, b, (__nv_bfloat16*)out, rows, n_rows, hidden, eps);
-  else TLLM_FAIL(TLLM_ERR_ARG, "layer_norm: unknown dtype code %d", out_dtype);
-  return TLLM_OK;
+  if (out_dtype == TLLM_F32) return launch_layer_norm<float>(x, w, b, (float*)out, rows, n_rows, hidden, eps, s);
+  if (out_dtype == TLLM_BF16) return launch_layer_norm<__nv_bfloat16>(x, w, b, (__nv_bfloat16*)out, rows, n_rows, hidden, eps, s);
+  TLLM_FAIL(TLLM_ERR_ARG, "layer_norm: unknown dtype code %d", out_dtype);
 }
 
 extern "C" int tllm_depth_average(float* x, float* stages, long long stage_stride, int n_stages, int keep, const float* mix,

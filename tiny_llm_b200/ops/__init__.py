@@ -780,7 +780,7 @@ def conv_norm_kv_write(proj: torch.Tensor, batch, num_heads: int, num_kv_heads: 
                        norm_k: Optional[torch.Tensor] = None, eps: float = 0.0) -> None:
     """Rows of `proj` begin with num_heads query heads and num_kv_heads key heads of key_dim values, then num_kv_heads
     value heads of value_dim values.  With x = row + bias (float32 [channels]) every channel is filtered over time,
-    y_t = sum_j taps[:, j] x_(t - n + 1 + j) (taps float32 [channels, n], zeros before the sequence's start; the last
+    y_t = sum_j taps[j] x_(t - n + 1 + j) (taps float32 [n, channels], zeros before the sequence's start; the last
     n - 1 inputs lie in kept[slot], float32 [slots, n - 1, channels], and are brought up to date); then all query values
     of a token together become y / sqrt(mean(y^2) + eps) * norm_q (float32 [num_heads * key_dim]), and all its key values
     the same with norm_k.  Queries go to q_out [T, num_heads * key_dim], keys and values to their pages; `proj` stays as
@@ -790,7 +790,7 @@ def conv_norm_kv_write(proj: torch.Tensor, batch, num_heads: int, num_kv_heads: 
     t = proj.shape[0]
     nqc, nkc = num_heads * key_dim, num_kv_heads * key_dim
     channels = nqc + nkc + num_kv_heads * value_dim
-    n = 1 if taps is None else taps.shape[1]
+    n = 1 if taps is None else taps.shape[0]
     if proj.stride(1) != 1 or proj.shape[1] < channels or q_out.shape != (t, nqc) or not q_out.is_contiguous() or \
             q_out.dtype != proj.dtype:
         raise KernelError("conv_norm_kv_write: the rows of the projection or of the query buffer do not fit")
@@ -798,7 +798,7 @@ def conv_norm_kv_write(proj: torch.Tensor, batch, num_heads: int, num_kv_heads: 
     _paged("conv_norm_kv_write", v_cache, num_kv_heads, value_dim)
     if k_cache.dtype != proj.dtype or v_cache.dtype != proj.dtype or k_cache.shape[2] != v_cache.shape[2]:
         raise KernelError("conv_norm_kv_write: cache dtype or page size does not fit")
-    for name, b, shape in (("bias", bias, (channels,)), ("filter", taps, (channels, n)), ("query norm", norm_q, (nqc,)),
+    for name, b, shape in (("bias", bias, (channels,)), ("filter", taps, (n, channels)), ("query norm", norm_q, (nqc,)),
                            ("key norm", norm_k, (nkc,))):
         if b is not None and (b.dtype != torch.float32 or tuple(b.shape) != shape or not b.is_contiguous()):
             raise KernelError(f"conv_norm_kv_write: the {name} must be contiguous float32 of shape {shape}")
@@ -1135,6 +1135,7 @@ def attention_talk(q: torch.Tensor, num_heads: int, num_kv_heads: int, key_dim: 
 
 
 EPI_BF16, EPI_F32, EPI_ADD_F32, EPI_SWIGLU, EPI_ATOMIC_F32 = 0, 1, 2, 3, 4
+EPI_GLU_CLAMPED = 11                               # EPI_SWIGLU with the clamped gate
 EPI_CL_ADD_F32, EPI_CL_ROPE_KV, EPI_CL_SWIGLU, EPI_CL_BF16 = 5, 6, 7, 8   # K slices reduced inside a thread-block cluster
 _sm_count = {}
 
@@ -1220,7 +1221,7 @@ def _cluster_slices(n: int, k: int, limit: int = 8) -> int:
 
 
 def _cluster_call(epi, a, w, out, slices, positions=None, cos=None, sin=None, nq=0, nkv=0, hd=0, k_cache=None,
-                  v_cache=None, slot_mapping=None):
+                  v_cache=None, slot_mapping=None, limit=0.0):
     lib = build.load_library("linear_tc")
     m, k = a.shape
     page_size = page_stride = head_stride = 0
@@ -1229,7 +1230,7 @@ def _cluster_call(epi, a, w, out, slices, positions=None, cos=None, sin=None, nq
     _call(lib, lib.tllm_linear_tc_cluster,
         _ptr(a), _ptr(w), _ptr(out), m, w.shape[0], k, a.stride(0), out.stride(0), epi, slices, _ptr(positions),
         _ptr(cos), _ptr(sin), nq, nkv, hd, _ptr(k_cache), _ptr(v_cache), _ptr(slot_mapping), page_size,
-        ctypes.c_longlong(page_stride), ctypes.c_longlong(head_stride), _ptr(status_word(a.device)), _stream())
+        ctypes.c_longlong(page_stride), ctypes.c_longlong(head_stride), ctypes.c_float(limit), _ptr(status_word(a.device)), _stream())
 
 
 def linear_rope_kv(h: torch.Tensor, w_qkv: torch.Tensor, qkv: torch.Tensor, positions: torch.Tensor,
@@ -1327,7 +1328,7 @@ def linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate: bool
             if splits > 1:
                 epi = EPI_ATOMIC_F32
         _call(lib, lib.tllm_linear_tc, _ptr(a), _ptr(w), _ptr(out), m, n, k, a.stride(0), out.stride(0), epi, swap,
-                                       splits, _ptr(status_word(a.device)), _stream())
+                                       splits, ctypes.c_float(0.0), _ptr(status_word(a.device)), _stream())
         return
     lib = build.load_library("linear_generic")
     _call(lib, lib.tllm_linear_generic, _ptr(a), _ptr(w), _ptr(out), m, n, k, a.stride(0), out.stride(0),
@@ -1337,11 +1338,14 @@ def linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate: bool
 def linear_swiglu(a: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, block: int, workspace,
                   act: str = "silu", limit: float = 0.0) -> None:
     """out = act(a Wg^T) * (a Wu^T) with Wg, Wu interleaved in `w_gate_up` in row blocks of `block`; act one of GLU_ACTS.
-    With blocks of 128 and more than 128 rows the product and SiLU*up are one tensor-core kernel (SiLU only: another
-    activation takes the product and the element-wise kernel)."""
+    With blocks of 128 the product and the gate are one tensor-core kernel (SiLU and the clamped form: another activation
+    takes the product and the element-wise kernel)."""
     m = a.shape[0]
     n2 = w_gate_up.shape[0]
-    if act != "silu":
+    if act not in GLU_ACTS or (act == "clamped" and not limit > 0):
+        raise KernelError(f"linear_swiglu: unknown activation {act!r} (known: {', '.join(GLU_ACTS)}; \"clamped\" needs a limit)")
+    limit = float(limit) if act == "clamped" else 0.0
+    if act == "relu":
         if prefers_split(a, w_gate_up):
             acc = workspace.get_zeroed("gate_up_f32", (m, n2))
             linear(a, w_gate_up, acc, accumulate=True)
@@ -1355,22 +1359,23 @@ def linear_swiglu(a: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, b
         _need_cuda(a, w_gate_up, out)
         lib = build.load_library("linear_tc")
         _call(lib, lib.tllm_linear_tc, _ptr(a), _ptr(w_gate_up), _ptr(out), m, n2, a.shape[1], a.stride(0),
-                                       out.stride(0), EPI_SWIGLU, 0, 1, _ptr(status_word(a.device)), _stream())
+                                       out.stride(0), EPI_GLU_CLAMPED if act == "clamped" else EPI_SWIGLU, 0, 1,
+                                       ctypes.c_float(limit), _ptr(status_word(a.device)), _stream())
         return
     if (cluster_mask & 4) and _tc_ok(a, w_gate_up, out) and block == 128 and m <= 128 and n2 % 256 == 0 and \
             out.stride(1) == 1 and w_gate_up.is_contiguous():
         # the gate tile, the up tile beside it and their K slices form one cluster; SiLU * up in its epilogue
         _need_cuda(a, w_gate_up, out)
-        _cluster_call(EPI_CL_SWIGLU, a, w_gate_up, out, _cluster_slices(n2, a.shape[1], limit=4))
+        _cluster_call(EPI_CL_SWIGLU, a, w_gate_up, out, _cluster_slices(n2, a.shape[1], limit=4), limit=limit)
         return
     if prefers_split(a, w_gate_up):
         acc = workspace.get_zeroed("gate_up_f32", (m, n2))
         linear(a, w_gate_up, acc, accumulate=True)
-        silu_mul(acc, out, block, consume=True)
+        silu_mul(acc, out, block, consume=True, act=act, limit=limit)
         return
     gu = workspace.get("gate_up", (m, n2), a.dtype)
     linear(a, w_gate_up, gu)
-    silu_mul(gu, out, block)
+    silu_mul(gu, out, block, act=act, limit=limit)
 
 
 # ----------------------------------------------------------------------------- attention

@@ -194,7 +194,7 @@ class SinkAttention:
         self.w_sink = weights[prefix + "sink"] if self.sink else None
         if self.filtered:
             self.bias_row = torch.cat(self.biases).contiguous() if self.bias else None
-            self.taps = torch.cat([weights[prefix + n + ".conv"] for n in ("q", "k", "v")]).contiguous() if self.conv else None
+            self.taps = torch.cat([weights[prefix + n + ".conv"] for n in ("q", "k", "v")]).T.contiguous() if self.conv else None   # [taps, channels]
         if self.bias_max is not None:   # a row of biases by distance per head; distances past the row take its last value
             table = weights[prefix + "rel"]
             rows = torch.tensor(distance_buckets(table.shape[0], float(self.bias_max)), device=table.device)
