@@ -151,8 +151,8 @@ def test_parts_refuse_what_they_do_not_have():
     base = dict(hidden_size=16, num_heads=2, num_kv_heads=1, key_dim=8, value_dim=8, scale=1.0, eps=1e-5)
     with pytest.raises(ValueError, match="norms per head"):
         SinkAttention(**base, conv=3)
-    with pytest.raises(ValueError, match="rotations"):
-        SinkAttention(**base, qk_norm="whole", rot_dims=4)
+    with pytest.raises(ValueError, match="stretched queries"):
+        SinkAttention(**base, qk_norm="whole", stretch_coef=0.5, stretch_every=4)
     with pytest.raises(ValueError, match="mixed scores"):
         SinkAttention(**base, talk=True, bias_max=10.0)
     with pytest.raises(ValueError, match="query/key norm"):

@@ -8,7 +8,8 @@ from .zozenex import ZozenexConfig
 from .fiponex import FiponexConfig
 from .gevovik import GevovikConfig
 from .vigodra import VigodraConfig
+from .lovapel import LovapelConfig
 
-__all__ = ["ConfigError", "LlamaConfig", "DunelixConfig", "ZozenexConfig", "FiponexConfig", "GevovikConfig", "VigodraConfig", "LayerCall", "LayerSpec", "ModelSpec", "PartSpec",
+__all__ = ["ConfigError", "LlamaConfig", "DunelixConfig", "ZozenexConfig", "FiponexConfig", "GevovikConfig", "VigodraConfig", "LovapelConfig", "LayerCall", "LayerSpec", "ModelSpec", "PartSpec",
            "config_class_for", "config_from_dict", "load_config", "register_architecture",
            "registered_architectures"]

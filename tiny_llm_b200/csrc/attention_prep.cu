@@ -19,8 +19,10 @@
 //   them channels of a short causal filter over time: y_t[c] = sum_j taps[j, c] x_(t - n_taps + 1 + j)[c] with x the
 //   projection plus its bias, zero before the sequence's start; the last n_taps - 1 inputs of every channel are the
 //   request's state.  The filtered queries TOGETHER (all heads of the token) are divided by sqrt(mean(y^2) + eps) and
-//   multiplied by a weight per channel, and so are the keys.  Queries go to a buffer of their own (other tokens' filters
-//   still read the projection), keys and values to their pages.
+//   multiplied by a weight per channel, and so are the keys.  With a frequency table the first rot_dims values of every
+//   query and key head are then turned as in qk_norm_kv_write (a token's cosines and sines are taken once for all its
+//   heads).  Queries go to a buffer of their own (other tokens' filters still read the projection), keys and values to
+//   their pages.
 // sigmoid_gate: out[t, h, :] = x[t, h, :] * sigmoid(gate), the gate one value per element or one per head.
 #include "common.cuh"
 
@@ -237,6 +239,10 @@ struct ConvArgs {
   long long k_page_stride, k_head_stride, v_page_stride, v_head_stride;
   int n_tokens;
   int update;                   // every request brings one token: its kept inputs move up here
+  const int* positions;
+  const float* freq;            // [rot_dims / 2] or null: query and key heads are rotated behind the norm
+  int rot_dims, rot_pairs;      // the first rot_dims values of a head turn; pairs (2i, 2i + 1) or halves (i, i + rot_dims / 2)
+  float rot_mag;                // cos and sin are multiplied by this
 };
 
 template <typename T, int V> struct Piece { T v[V]; };   // V neighbouring channels; 8 of them are 16-byte aligned
@@ -250,7 +256,7 @@ template <> struct __align__(16) Piece<__nv_bfloat16, 8> { __nv_bfloat16 v[8]; }
 constexpr int CONV_THREADS = 384;
 template <typename T, int V, int TOK, int NT>
 __global__ void __launch_bounds__(CONV_THREADS) conv_norm_kv_write_kernel(ConvArgs a) {
-  extern __shared__ __align__(16) float ys[];        // [TOK, (nq + nkv) * kd]
+  extern __shared__ __align__(16) float ys[];        // [TOK, (nq + nkv) * kd], then [TOK, rot_dims / 2] cosines and sines
   __shared__ float part[2 * TOK][33];
   pdl_trigger();
   const int nqc = a.nq * a.kd, nkc = a.nkv * a.kd, nvc = a.nkv * a.vd, channels = nqc + nkc + nvc, nqk = nqc + nkc;
@@ -261,8 +267,19 @@ __global__ void __launch_bounds__(CONV_THREADS) conv_norm_kv_write_kernel(ConvAr
   float ssq[TOK], ssk[TOK];
 #pragma unroll
   for (int i = 0; i < TOK; ++i) ssq[i] = ssk[i] = 0.f;
+  const int half = a.rot_dims / 2;
+  float *turn_c = ys + (size_t)TOK * nqk, *turn_s = turn_c + TOK * half;
+  for (int i = threadIdx.x; i < TOK * half; i += blockDim.x) {
+    const int t = t0 + i / half;
+    if (t >= a.n_tokens) continue;
+    const float ang = __fmul_rn((float)a.positions[t], a.freq[i % half]);
+    turn_c[i] = __fmul_rn(cosf(ang), a.rot_mag);
+    turn_s[i] = __fmul_rn(sinf(ang), a.rot_mag);
+  }
   bool inside = false;
-  if (TOK > 1 && NT > 0 && t0 + TOK <= a.n_tokens) {
+  if (NT == 1) {
+    inside = TOK > 1 && t0 + TOK <= a.n_tokens;    // one tap reads the token itself, whatever its request
+  } else if (TOK > 1 && NT > 0 && t0 + TOK <= a.n_tokens) {
     const int req = a.token_request[t0];
     inside = req == a.token_request[t0 + TOK - 1] && t0 - a.cu_q[req] >= NT - 1;
   }
@@ -276,7 +293,14 @@ __global__ void __launch_bounds__(CONV_THREADS) conv_norm_kv_write_kernel(ConvAr
     Piece<float, V> w[NT ? NT : 1];
     if (NT) {
 #pragma unroll
-      for (int j = 0; j < NT; ++j) w[j] = *reinterpret_cast<const Piece<float, V>*>(a.taps + (size_t)j * channels + c);
+      for (int j = 0; j < NT; ++j) {
+        if (NT == 1 && a.taps == nullptr) {          // no filter
+#pragma unroll
+          for (int e = 0; e < V; ++e) w[j].v[e] = 1.f;
+        } else {
+          w[j] = *reinterpret_cast<const Piece<float, V>*>(a.taps + (size_t)j * channels + c);
+        }
+      }
     }
     Piece<float, V> add;
     if (a.bias) {
@@ -400,7 +424,25 @@ __global__ void __launch_bounds__(CONV_THREADS) conv_norm_kv_write_kernel(ConvAr
       }
       Piece<T, V> p;
 #pragma unroll
-      for (int e = 0; e < V; ++e) p.v[e] = from_f32<T>(__fmul_rn(__fmul_rn(y[e], f), w.v[e]));
+      for (int e = 0; e < V; ++e) y[e] = __fmul_rn(__fmul_rn(y[e], f), w.v[e]);
+      const int d0 = is_q ? c % a.kd : d;             // the piece's place in its head (a head is whole pieces)
+      if (half > 0 && d0 < a.rot_dims) {
+        const float* row = ys + (size_t)i * nqk + (c - d0);
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          const int at = d0 + e;
+          if (at >= a.rot_dims) continue;
+          const bool first = a.rot_pairs ? !(at & 1) : at < half;
+          const int other = a.rot_pairs ? at ^ 1 : (first ? at + half : at - half);
+          const int pair = i * half + (a.rot_pairs ? at >> 1 : (first ? at : at - half));
+          const float cs = turn_c[pair], sn = turn_s[pair];
+          const float wo = wn ? wn[(is_q ? c : c - nqc) - d0 + other] : 1.f;
+          const float yo = __fmul_rn(__fmul_rn(row[other], f), wo);
+          y[e] = first ? fmaf(y[e], cs, -__fmul_rn(yo, sn)) : fmaf(y[e], cs, __fmul_rn(yo, sn));
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < V; ++e) p.v[e] = from_f32<T>(y[e]);
       *reinterpret_cast<Piece<T, V>*>(dst) = p;
     }
   }
@@ -410,7 +452,7 @@ template <typename T, int V, int TOK, int NT>
 static int launch_conv(const ConvArgs& a, cudaStream_t s) {
   const int channels = (a.nq + a.nkv) * a.kd + a.nkv * a.vd, pieces = channels / V;
   const int threads = pieces >= CONV_THREADS ? CONV_THREADS : (pieces + 31) / 32 * 32;
-  const size_t smem = (size_t)TOK * (a.nq + a.nkv) * a.kd * 4;
+  const size_t smem = (size_t)TOK * ((a.nq + a.nkv) * a.kd + a.rot_dims) * 4;
   static size_t configured = 48 * 1024;
   if (smem + 2 * TOK * 33 * 4 > configured) {
     cudaError_t e = cudaFuncSetAttribute(conv_norm_kv_write_kernel<T, V, TOK, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -424,8 +466,9 @@ static int launch_conv(const ConvArgs& a, cudaStream_t s) {
 template <typename T>
 static int launch_conv_sizes(const ConvArgs& a, bool vec, cudaStream_t s) {
   constexpr int TOK = 4;
-  const bool many = !a.update && a.n_tokens >= 148 * TOK && (size_t)TOK * (a.nq + a.nkv) * a.kd * 4 <= 160 * 1024;
+  const bool many = !a.update && a.n_tokens >= 148 * TOK && (size_t)TOK * ((a.nq + a.nkv) * a.kd + a.rot_dims) * 4 <= 160 * 1024;
   if (!vec) return launch_conv<T, 1, 1, 0>(a, s);
+  if (a.n_taps == 1) return many ? launch_conv<T, 8, TOK, 1>(a, s) : launch_conv<T, 8, 1, 1>(a, s);
   if (a.taps && a.n_taps == 4) return many ? launch_conv<T, 8, TOK, 4>(a, s) : launch_conv<T, 8, 1, 4>(a, s);
   return many ? launch_conv<T, 8, TOK, 0>(a, s) : launch_conv<T, 8, 1, 0>(a, s);
 }
@@ -504,14 +547,18 @@ extern "C" int tllm_conv_norm_kv_write(const void* proj, int ld, int nq, int nkv
                                        const int* token_request, const float* wq, const float* wk, float eps, void* q_out,
                                        void* kcache, void* vcache, const int* slot_mapping, int page_size,
                                        long long k_page_stride, long long k_head_stride, long long v_page_stride,
-                                       long long v_head_stride, int n_tokens, int update, int dtype, void* stream) {
-  TLLM_REQUIRE(n_tokens > 0 && nq > 0 && nkv > 0 && kd > 0 && vd > 0 && ((long long)(nq + nkv) * kd) * 4 <= 220 * 1024,
+                                       long long v_head_stride, int n_tokens, int update, const int* positions,
+                                       const float* freq, int rot_dims, int rot_pairs, float rot_mag, int dtype, void* stream) {
+  TLLM_REQUIRE(n_tokens > 0 && nq > 0 && nkv > 0 && kd > 0 && vd > 0 && rot_dims >= 0 && ((long long)(nq + nkv) * kd + rot_dims) * 4 <= 220 * 1024,
                "conv_norm_kv_write: %d tokens, %d / %d heads, key size %d, value size %d (queries and keys of a token: at most %d values)",
                n_tokens, nq, nkv, kd, vd, 220 * 256);
   TLLM_REQUIRE(n_taps >= 1 && (n_taps == 1 || (taps && kept && slots)) && proj && q_out && kcache && vcache && slot_mapping && cu_q &&
                token_request && page_size > 0 && (wq == nullptr) == (wk == nullptr),
                "conv_norm_kv_write: %d taps; a filter needs weights, kept inputs and slots; norm weights for both or neither", n_taps);
+  TLLM_REQUIRE(rot_dims % 2 == 0 && rot_dims <= kd && (rot_dims == 0 || (freq && positions)),
+               "conv_norm_kv_write: %d rotated values of %d (even, at most the head's size, with a frequency table and positions)", rot_dims, kd);
   ConvArgs a;
+  a.positions = positions; a.freq = freq; a.rot_dims = rot_dims; a.rot_pairs = rot_pairs; a.rot_mag = rot_mag;
   a.proj = proj; a.ld = ld; a.nq = nq; a.nkv = nkv; a.kd = kd; a.vd = vd; a.bias = bias; a.taps = taps; a.n_taps = n_taps;
   a.kept = kept; a.slots = slots; a.cu_q = cu_q; a.token_request = token_request; a.wq = wq; a.wk = wk; a.eps = eps;
   a.q_out = q_out; a.kcache = kcache; a.vcache = vcache; a.slot_mapping = slot_mapping; a.page_size = page_size;

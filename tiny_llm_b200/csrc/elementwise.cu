@@ -134,7 +134,8 @@ __global__ void rms_norm_vec_kernel(const float* __restrict__ x, const float* __
 }
 
 // What a gated feed-forward makes of a gate value and an up value: SiLU(g) u (act 0), ReLU(g) u (act 1), or the clamped
-// form (act 2): g <- min(g, limit), u <- clamp(u, -limit, limit), g sigmoid(1.702 g) (u + 1).
+// form (act 2): g <- min(g, limit), u <- clamp(u, -limit, limit), g sigmoid(1.702 g) (u + 1), or the tanh form of GELU
+// (act 3): gelu(g) u with gelu(g) = g / 2 (1 + tanh(y)) = g / (1 + exp(-2 y)), y = sqrt(2 / pi) (g + 0.044715 g^3).
 __device__ __forceinline__ float glu_value(float g, float u, int act, float limit) {
   if (act == 1) return fmaxf(g, 0.f) * u;
   if (act == 2) {
@@ -142,6 +143,7 @@ __device__ __forceinline__ float glu_value(float g, float u, int act, float limi
     u = fminf(fmaxf(u, -limit), limit);
     return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
   }
+  if (act == 3) return g / (1.f + expf(-1.59576912160573081f * g * fmaf(0.044715f * g, g, 1.f))) * u;   // 2 sqrt(2 / pi)
   return g / (1.f + expf(-g)) * u;
 }
 
@@ -668,7 +670,7 @@ extern "C" int tllm_silu_mul(void* gu, void* out, int m, int inter, int blk, int
                              int act, float limit, void* stream) {
   TLLM_REQUIRE(m > 0 && inter > 0 && blk > 0 && inter % blk == 0,
                "silu_mul: %d rows, width %d, block %d (the block must divide the width)", m, inter, blk);
-  TLLM_REQUIRE(act >= 0 && act <= 2 && (act != 2 || limit > 0.f), "silu_mul: activation code %d, limit %g", act, (double)limit);
+  TLLM_REQUIRE(act >= 0 && act <= 3 && (act != 2 || limit > 0.f), "silu_mul: activation code %d, limit %g", act, (double)limit);
   const size_t total = (size_t)m * inter;
   const int threads = 256;
   const int blocks = (int)((total + threads - 1) / threads < 148 * 16 ? (total + threads - 1) / threads : 148 * 16);
@@ -785,6 +787,27 @@ __global__ void bigram_add_kernel(const int* __restrict__ tokens, const int* __r
 }
 
 // ---------------------------------------------------------------- element by element: a copy in another type, or relu(x)^2
+// x <- cap * tanh(scale * x / cap) (cap 0: x <- scale * x), float32, in place
+__global__ void soft_cap_kernel(float* __restrict__ x, long long n, float scale, float cap) {
+  pdl_trigger();
+  pdl_wait();
+  const long long stride = (long long)gridDim.x * blockDim.x, first = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  const bool vec = (n & 3) == 0 && ((uintptr_t)x & 15) == 0;
+  auto one = [&](float v) {
+    v = __fmul_rn(v, scale);
+    return cap > 0.f ? __fmul_rn(cap, tanhf(v / cap)) : v;
+  };
+  if (vec) {
+    for (long long i = first; i < n / 4; i += stride) {
+      float4 v = reinterpret_cast<float4*>(x)[i];
+      v.x = one(v.x); v.y = one(v.y); v.z = one(v.z); v.w = one(v.w);
+      reinterpret_cast<float4*>(x)[i] = v;
+    }
+  } else {
+    for (long long i = first; i < n; i += stride) x[i] = one(x[i]);
+  }
+}
+
 template <typename TI, typename TO>
 __global__ void unary_kernel(const TI* __restrict__ x, TO* __restrict__ out, long long n, int act) {
   pdl_trigger();
@@ -846,5 +869,13 @@ extern "C" int tllm_scaled_add(float* x, float* resid, long long n, float scale,
   const long long want = (n + threads - 1) / threads;
   const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
   TLLM_LAUNCH("scaled_add", scaled_add_kernel, blocks, threads, 0, (cudaStream_t)stream, x, resid, n, scale, clear);
+  return TLLM_OK;
+}
+
+extern "C" int tllm_soft_cap(float* x, long long n, float scale, float cap, void* stream) {
+  TLLM_REQUIRE(n > 0 && cap >= 0.f, "soft_cap: %lld values, cap %g", n, (double)cap);
+  const int threads = 256;
+  const long long want = (n / ((n & 3) ? 1 : 4) + threads - 1) / threads;
+  TLLM_LAUNCH("soft_cap", soft_cap_kernel, (unsigned)(want < 148 * 16 ? want : 148 * 16), threads, 0, (cudaStream_t)stream, x, n, scale, cap);
   return TLLM_OK;
 }

@@ -42,15 +42,20 @@ enum Epilogue { EPI_BF16 = 0, EPI_F32 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU = 3, EPI_
                 // NORMAL orientation: Q/K/V projection with rotation and cache write (head size 64 or 128)
                 EPI_ROPE_KV = 9,
                 EPI_GELU_BF16 = 10,    // bfloat16 store of the exact GELU of the sums (the grouped expert product)
-                EPI_GLU_CLAMPED = 11 };   // like EPI_SWIGLU with the clamped gate (glu_f)
+                EPI_GLU_CLAMPED = 11,     // like EPI_SWIGLU with the clamped gate (glu_f)
+                EPI_GLU_GELU = 12 };      // like EPI_SWIGLU with the tanh form of GELU (glu_f)
 
 constexpr int ERR_PRODUCER = 1, ERR_MMA = 2, ERR_EPILOGUE = 3;
 
 __device__ __forceinline__ float silu_f(float x) { return __fdividef(x, 1.f + __expf(-x)); }
 
 // What the gate/up epilogues store: SiLU(g) u, or, clamped, with g <- min(g, limit) and u <- clamp(u, -limit, limit),
-// g sigmoid(1.702 g) (u + 1).
-constexpr bool is_glu(int epi) { return epi == EPI_SWIGLU || epi == EPI_GLU_CLAMPED; }
+// g sigmoid(1.702 g) (u + 1), or gelu(g) u with gelu(g) = g / 2 (1 + tanh(y)) = g / (1 + exp(-2 y)),
+// y = sqrt(2 / pi) (g + 0.044715 g^3).
+constexpr bool is_glu(int epi) { return epi == EPI_SWIGLU || epi == EPI_GLU_CLAMPED || epi == EPI_GLU_GELU; }
+__device__ __forceinline__ float gelu_tanh_f(float g) {
+  return __fdividef(g, 1.f + __expf(-1.59576912160573081f * g * fmaf(0.044715f * g, g, 1.f)));   // 2 sqrt(2 / pi)
+}
 __device__ __forceinline__ float clamped_glu_f(float g, float u, float limit) {
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
@@ -58,7 +63,7 @@ __device__ __forceinline__ float clamped_glu_f(float g, float u, float limit) {
 }
 template <int EPI>
 __device__ __forceinline__ float glu_f(float g, float u, float limit) {
-  return EPI == EPI_GLU_CLAMPED ? clamped_glu_f(g, u, limit) : silu_f(g) * u;
+  return EPI == EPI_GLU_CLAMPED ? clamped_glu_f(g, u, limit) : (EPI == EPI_GLU_GELU ? gelu_tanh_f(g) : silu_f(g)) * u;
 }
 
 template <int BN, int STAGES>
@@ -92,9 +97,9 @@ struct ClusterArgs {
   // every role), whose weights are rows [expert * expert_rows, +rows_b) of the stacked B matrix (null: one B for all)
   const int* tile_expert;
   int expert_rows;
-  // gate/up epilogues: the clamped gate's limit; the cluster kernel's gate: 0 SiLU, 1 clamped
+  // gate/up epilogues: the clamped gate's limit; the cluster kernel's gate: 0 SiLU, 2 clamped, 3 the tanh form of GELU
   float limit;
-  int clamped;
+  int act;
 };
 
 // Epilogue of one 128 x BN tile of C in the NORMAL orientation: this thread owns row `row` of the
@@ -646,8 +651,9 @@ linear_tc_cluster_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
 #pragma unroll
       for (int e = 0; e < 4; ++e)
         if (2 * col0 + BM + r + e < rows_a)   // the matching up row exists
-          dst[e] = __float2bfloat16_rn(ca.clamped ? clamped_glu_f(gate[e], up[e], ca.limit)
-                                                  : (gate[e] / (1.f + expf(-gate[e]))) * up[e]);
+          dst[e] = __float2bfloat16_rn(ca.act == 2 ? clamped_glu_f(gate[e], up[e], ca.limit)
+                                       : ca.act == 3 ? gelu_tanh_f(gate[e]) * up[e]
+                                                     : (gate[e] / (1.f + expf(-gate[e]))) * up[e]);
     }
   } else if (EPI == EPI_CL_ROPE_KV) {
     // pairs (d, d + hd/2) of whole heads: 64 pairs per tile, dealt to the CZ CTAs, four neighbouring pairs per item
@@ -1125,13 +1131,14 @@ using namespace tllm;
 // out[M, N] (row stride ldo) = / += a[M, K] (row stride lda) . w[N, K]^T, bfloat16 operands.
 //   epi: 0 store bfloat16, 1 store float32, 2 add into float32, 3 SiLU(gate)*up with gate/up rows of w
 //        interleaved in blocks of 128 (out is [M, N/2] bfloat16), 4 atomic add into float32, 11 the same as 3
-//        with the clamped gate and its `limit`.
+//        with the clamped gate and its `limit`, 12 with the tanh form of GELU.
 //   swap: 0 = 128 x 256 tiles of C per CTA (large M); 1 = weights on the 128-row side, M <= 128,
 //        `splits` slices of K per weight tile (epi 4 when splits > 1).
 // `status` is a device int that receives a non-zero code if a bounded wait expired.
 // The grouped product of a mixture of experts: A [rows, k] holds whole tiles of 128 rows, every tile the rows of ONE
 // expert (tile_expert[rows / 128], -1 for a tile that does not exist); w is [experts * n, k], expert e's matrix in rows
-// [e n, (e + 1) n); out [rows, n]: bfloat16 of GELU(sums) (epi 10) or float32 sums (epi 1).
+// [e n, (e + 1) n); out [rows, n]: bfloat16 of GELU(sums) (epi 10) or float32 sums (epi 1), or [rows, n / 2]: bfloat16 of
+// SiLU(gate) * up (epi 3) with every expert's gate and up rows interleaved in blocks of 128.
 extern "C" int tllm_linear_tc_grouped(const void* a, const void* w, void* out, int rows, int n, int k, int lda, int ldo,
                                       int experts, const int* tile_expert, int epi, int* status, void* stream) {
   TLLM_REQUIRE(rows > 0 && rows % BM == 0 && n > 0 && k > 0 && experts > 0, "linear_tc_grouped: %d rows (whole tiles of %d), %d x %d, %d experts", rows, BM, n, k, experts);
@@ -1149,8 +1156,11 @@ extern "C" int tllm_linear_tc_grouped(const void* a, const void* w, void* out, i
   switch (epi) {
     case EPI_GELU_BF16: return launch_persistent<EPI_GELU_BF16>(ma, mb, out, rows, n, k, ldo, status, s, ca);
     case EPI_F32: return launch_persistent<EPI_F32>(ma, mb, out, rows, n, k, ldo, status, s, ca);
+    case EPI_SWIGLU:
+      TLLM_REQUIRE(n % 256 == 0, "linear_tc_grouped: SiLU*up needs gate/up blocks of 128 rows (N = %d)", n);
+      return launch_persistent<EPI_SWIGLU>(ma, mb, out, rows, n, k, ldo, status, s, ca);   // (no strips: no weight pointer)
   }
-  TLLM_FAIL(TLLM_ERR_ARG, "linear_tc_grouped: epilogue %d (GELU to bfloat16 or float32 sums)", epi);
+  TLLM_FAIL(TLLM_ERR_ARG, "linear_tc_grouped: epilogue %d (GELU or SiLU*up to bfloat16, or float32 sums)", epi);
 }
 
 extern "C" int tllm_linear_tc(const void* a, const void* w, void* out, int m, int n, int k, int lda, int ldo, int epi,
@@ -1177,6 +1187,7 @@ extern "C" int tllm_linear_tc(const void* a, const void* w, void* out, int m, in
         ca.limit = limit;
         return launch_persistent<EPI_GLU_CLAMPED>(ma, mb, out, m, n, k, ldo, status, s, ca, w);
       }
+      case EPI_GLU_GELU: return launch_persistent<EPI_GLU_GELU>(ma, mb, out, m, n, k, ldo, status, s, ClusterArgs(), w);
     }
     TLLM_FAIL(TLLM_ERR_ARG, "linear_tc: unknown epilogue %d", epi);
   }
@@ -1214,12 +1225,13 @@ extern "C" int tllm_linear_tc(const void* a, const void* w, void* out, int m, in
 //      hd 16, 32, 64 or 128; cos/sin null: no rotation.  This one also takes more than 128 rows (head size
 //      64 or 128): then it runs as 128 x 256 tiles of C with the same epilogue per tile;
 //   7: SiLU(gate) * up with gate/up rows of w interleaved in blocks of 128, out bfloat16 [M, N/2]
-//      (slices <= 4: the cluster also spans the gate tile and the up tile); with `limit` > 0 the clamped gate instead;
+//      (slices <= 4: the cluster also spans the gate tile and the up tile); `act` 2: the clamped gate with its `limit`
+//      instead, 3: the tanh form of GELU;
 //   8: out (bfloat16 [M, N]) = product.
 extern "C" int tllm_linear_tc_cluster(const void* a, const void* w, void* out, int m, int n, int k, int lda, int ldo,
                                       int epi, int slices, const int* positions, const float* cos, const float* sin,
                                       int nq, int nkv, int hd, void* kcache, void* vcache, const int* slot_mapping,
-                                      int page_size, long long page_stride, long long head_stride, float limit,
+                                      int page_size, long long page_stride, long long head_stride, int act, float limit,
                                       int* status, void* stream) {
   TLLM_REQUIRE(m > 0 && n > 0 && k > 0 && (m <= 128 || epi == EPI_CL_ROPE_KV),
                "linear_tc_cluster: product %d x %d x %d (at most 128 rows, except for the Q/K/V projection)", m, n, k);
@@ -1230,7 +1242,8 @@ extern "C" int tllm_linear_tc_cluster(const void* a, const void* w, void* out, i
   TLLM_REQUIRE(slices <= (k + BK - 1) / BK, "linear_tc_cluster: %d slices of a K of %d", slices, k);
   ClusterArgs ca = {};
   ca.cy = 1; ca.cz = slices;
-  ca.limit = limit; ca.clamped = limit > 0.f;
+  TLLM_REQUIRE((act == 0 || act == 2 || act == 3) && (act != 2 || limit > 0.f), "linear_tc_cluster: gate activation %d, limit %g", act, (double)limit);
+  ca.limit = limit; ca.act = act;
   if (epi == EPI_CL_SWIGLU) {
     TLLM_REQUIRE(n % 256 == 0 && slices <= 4, "linear_tc_cluster: SiLU*up needs gate/up blocks of 128 rows (N = %d) and at most 4 slices", n);
     ca.cy = 2;

@@ -1,17 +1,22 @@
 // Mixture of experts: routing on the device and one grouped product for all experts.
 //
 // moe_route: per token, s_e = sigmoid(z_e), or softmax(z)_e over all experts; the `top` experts with the largest
-//   s_e + correction_e (no correction: s_e) are chosen (ties: the lower index); their weights are s_e * scale.  One
-//   warp per token, 32-bit.
+//   c_e = s_e + correction_e (no correction: s_e) are chosen (ties: the lower index); their weights are s_e * scale, or
+//   with `renorm` s_e / (sum of the chosen s + 1e-20) * scale.  With `groups` > 1 the experts form that many equal groups
+//   of neighbours, a group is worth its largest c (ties: the lower group), and only members of the best `keep` groups
+//   stand for choice.  One warp per token, 32-bit.
 // moe_align: the (token, choice) pairs of the step, numbered token * top + choice, are grouped by expert into tiles
 //   of `tile` rows: sorted_rows[tile * tile_rows + i] is a pair's number or -1 (padding), tile_expert[tile] the
-//   tile's expert or -1 (no such tile).  The host knows only the upper bound of the tile count.
+//   tile's expert or -1 (no such tile).  The host knows only the upper bound of the tile count.  Pairs whose expert is
+//   n_experts or above (experts that hand their input on and have no matrices) are left out; their pair_pos is -1.
 // moe_linear: out[row] = act(W[expert of the row's tile] . in[row / rows_per_input]) for every row named by
 //   sorted_rows.  W: [experts, N, K].  Two kernels: FFMA tiles for float32 (every output element is one chain of
 //   fmaf over ascending k, so a row's result does not depend on the tile it landed in) and mma.sync tiles for
-//   bfloat16 (below).
+//   bfloat16 (below).  The tensor-core kernel also makes SiLU(gate) * up of matrices whose gate and up rows alternate in
+//   blocks: out is then N / 2 wide.
 // moe_combine: resid[t] += sum_c weight[t, c] * y[t * top + c] (+ sigmoid(gate logit) * shared[t]), choices in the
-//   order the router found them; with pair_pos, y is in the grouped order and pair p lies in row pair_pos[p].
+//   order the router found them; with pair_pos, y is in the grouped order and pair p lies in row pair_pos[p]; a choice
+//   of n_experts or above stands for the token's own input row h[t].
 // moe_gather: the grouped order's input rows made contiguous (for a product that fetches A tiles by TMA).
 // gelu: the exact (erf) GELU, element by element.
 #include "common.cuh"
@@ -24,9 +29,31 @@ __device__ __forceinline__ float gelu_erf(float x) { return 0.5f * x * (1.f + er
 
 constexpr int ROUTE_PER_LANE = 16;   // experts per lane: at most 512 experts
 
-__global__ void moe_route_kernel(const float* __restrict__ logits, int ld, int n_experts, const float* __restrict__ correction,
-                                 float scale, int top, int* __restrict__ ids, float* __restrict__ weights, int n_tokens,
-                                 int softmax) {
+constexpr int ROUTE_WARPS = 4;
+
+struct RouteArgs {
+  const float* logits;
+  int ld, n_experts;
+  const float* correction;      // [n_experts] or null
+  float scale;
+  int top;
+  int* ids;                     // [n_tokens, top]
+  float* weights;
+  int n_tokens, softmax, renorm, groups, keep;
+};
+
+// A float's bits in an order that unsigned comparison understands.
+__device__ __forceinline__ unsigned ordered_bits(float v) {
+  const unsigned u = __float_as_uint(v);
+  return (u & 0x80000000u) ? ~u : (u | 0x80000000u);
+}
+
+__global__ void moe_route_kernel(RouteArgs a) {
+  __shared__ unsigned worth[ROUTE_WARPS][32 * ROUTE_PER_LANE];     // per group: its largest choice score
+  __shared__ unsigned char open[ROUTE_WARPS][32 * ROUTE_PER_LANE]; // per group: whether its members stand for choice
+  const float* __restrict__ logits = a.logits;
+  const float* __restrict__ correction = a.correction;
+  const int ld = a.ld, n_experts = a.n_experts, top = a.top, n_tokens = a.n_tokens, softmax = a.softmax;
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -60,6 +87,33 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int ld, int n
       c[i] = -INFINITY;
     }
   }
+  if (a.groups > 1) {
+    const int warp = threadIdx.x >> 5, size = n_experts / a.groups;
+    for (int g = lane; g < a.groups; g += 32) worth[warp][g] = 0u;    // below every score's bits
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < ROUTE_PER_LANE; ++i) {
+      const int e = lane + 32 * i;
+      if (e < n_experts) atomicMax(&worth[warp][e / size], ordered_bits(c[i]));
+    }
+    __syncwarp();
+    for (int g = lane; g < a.groups; g += 32) {
+      const unsigned mine = worth[warp][g];
+      int better = 0;
+      for (int o = 0; o < a.groups; ++o) {
+        const unsigned w = worth[warp][o];
+        better += w > mine || (w == mine && o < g);
+      }
+      open[warp][g] = better < a.keep;
+    }
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < ROUTE_PER_LANE; ++i) {
+      const int e = lane + 32 * i;
+      if (e < n_experts && !open[warp][e / size]) c[i] = -INFINITY;
+    }
+  }
+  float chosen_sum = 0.f;
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
     int bi = 0x7fffffff;
@@ -76,13 +130,21 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int ld, int n
       const float os = __shfl_xor_sync(0xffffffffu, bs, o);
       if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; bs = os; }
     }
-    if (lane == 0) {
-      ids[(size_t)t * top + k] = bi;
-      weights[(size_t)t * top + k] = bs * scale;
+    if (bi == 0x7fffffff) bi = k;   // scores that are not numbers: any valid index, the token's output is lost anyway
+    if (lane == (k & 31)) {
+      a.ids[(size_t)t * top + k] = bi;
+      a.weights[(size_t)t * top + k] = bs * (a.renorm ? 1.f : a.scale);
     }
+    chosen_sum += bs;
 #pragma unroll
     for (int i = 0; i < ROUTE_PER_LANE; ++i)
       if (lane + 32 * i == bi) c[i] = -INFINITY;
+  }
+  if (a.renorm) {   // every lane comes back to the weights it wrote itself
+    for (int k = lane; k < top; k += 32) {
+      float* w = a.weights + (size_t)t * top + k;
+      *w = __fmul_rn(__fdiv_rn(*w, chosen_sum + 1e-20f), a.scale);
+    }
   }
 }
 
@@ -96,7 +158,8 @@ __global__ void moe_align_kernel(const int* __restrict__ ids, int n_pairs, int n
   for (int e = threadIdx.x; e < n_experts; e += blockDim.x) counts[e] = 0;
   pdl_wait();
   __syncthreads();
-  for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) atomicAdd(&counts[ids[i]], 1);
+  for (int i = threadIdx.x; i < n_pairs; i += blockDim.x)
+    if (ids[i] < n_experts) atomicAdd(&counts[ids[i]], 1);
   for (int i = threadIdx.x; i < max_tiles * tile; i += blockDim.x) sorted_rows[i] = -1;
   __syncthreads();
   if (threadIdx.x == 0) {
@@ -115,6 +178,10 @@ __global__ void moe_align_kernel(const int* __restrict__ ids, int n_pairs, int n
   // does not depend on where in its expert's tiles it lies.
   for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) {
     const int e = ids[i];
+    if (e >= n_experts) {
+      if (pair_pos) pair_pos[i] = -1;
+      continue;
+    }
     const int at = start[e] + atomicAdd(&counts[e], 1);
     sorted_rows[at] = i;
     if (pair_pos) pair_pos[i] = at;     // where the pair's row lies in the grouped order
@@ -218,12 +285,18 @@ __device__ __forceinline__ void mma_bf16(float* c, const unsigned* a, unsigned b
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-template <typename TO, int BM, bool GELU>
+//
+// ACT_SILU_UP: the n rows of an expert's matrix are gate and up rows in alternating blocks of `glu_block`; the CTA's 128
+// rows of W are then 64 gate rows and their up rows, laid into shared memory in blocks of 8, so that a thread's
+// neighbouring accumulators are a gate value and its up value; out is n / 2 wide.
+enum MoeAct { ACT_NONE = 0, ACT_GELU = 1, ACT_SILU_UP = 2 };
+
+template <typename TO, int BM, int ACT>
 __global__ void __launch_bounds__(256) moe_linear_mma_kernel(const __nv_bfloat16* __restrict__ in, int ld_in,
                                                              const __nv_bfloat16* __restrict__ w,
                                                              const int* __restrict__ sorted_rows,
                                                              const int* __restrict__ tile_expert, TO* __restrict__ out,
-                                                             int n, int k, int rows_per_input) {
+                                                             int n, int k, int rows_per_input, int glu_block) {
   constexpr int BN = 128, BK = 32, LDS = 40, STAGES = BM == 16 ? 4 : 3;
   constexpr int WM = BM >= 64 ? 2 : 1, WN = 8 / WM;           // warps along rows and columns
   constexpr int WTM = BM / WM, WTN = BN / WN;                 // a warp's outputs: 64 x 32, 32 x 32 or 16 x 16
@@ -240,6 +313,7 @@ __global__ void __launch_bounds__(256) moe_linear_mma_kernel(const __nv_bfloat16
   const int e = tile_expert[blockIdx.x];
   if (e < 0) return;
   const int n0 = blockIdx.y * BN;
+  const int n_out = ACT == ACT_SILU_UP ? n / 2 : n;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   if (tid < BM) srow[tid] = sorted_rows[(size_t)blockIdx.x * BM + tid];
   __syncthreads();
@@ -253,6 +327,20 @@ __global__ void __launch_bounds__(256) moe_linear_mma_kernel(const __nv_bfloat16
     const int src = idx < BM * 4 ? srow[idx >> 2] : -1;
     a_ok[x] = src >= 0;
     a_ptr[x] = in + (size_t)(src < 0 ? 0 : src / rows_per_input) * ld_in + (idx & 3) * 8;
+  }
+  // ... and where its two rows of B begin (null: past the matrix)
+  const __nv_bfloat16* b_ptr[2];
+#pragma unroll
+  for (int x = 0; x < 2; ++x) {
+    const int r = (tid + x * 256) >> 2;
+    int row = n0 + r;
+    bool ok = row < n;
+    if (ACT == ACT_SILU_UP) {
+      const int o = n0 / 2 + (r >> 4) * 8 + (r & 7);     // the output column whose gate (r & 8 == 0) or up row this is
+      ok = o < n_out;
+      row = (o / glu_block) * 2 * glu_block + o % glu_block + ((r & 8) ? glu_block : 0);
+    }
+    b_ptr[x] = ok ? we + (size_t)row * k : nullptr;
   }
   const int nk = (k + BK - 1) / BK;
   auto load = [&](int stage, int kb) {
@@ -268,8 +356,8 @@ __global__ void __launch_bounds__(256) moe_linear_mma_kernel(const __nv_bfloat16
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
       const int idx = tid + x * 256, r = idx >> 2, c = (idx & 3) * 8;
-      const bool ok = n0 + r < n && k0 + c < k;
-      cp_async16(&sb[stage][r][c], we + (size_t)(ok ? n0 + r : 0) * k + (ok ? k0 + c : 0), ok);
+      const bool ok = b_ptr[x] != nullptr && k0 + c < k;
+      cp_async16(&sb[stage][r][c], ok ? b_ptr[x] + k0 + c : we, ok);
     }
   };
   float acc[MI][NI][4];
@@ -315,32 +403,54 @@ __global__ void __launch_bounds__(256) moe_linear_mma_kernel(const __nv_bfloat16
       const int row = srow[wm * WTM + i * 16 + (lane >> 2) + half * 8];
       if (row < 0) continue;
 #pragma unroll
-      for (int j = 0; j < NI; ++j) {
-        const int c = n0 + wn * WTN + j * 8 + (lane & 3) * 2;
+      for (int j = 0; j < NI; j += ACT == ACT_SILU_UP ? 2 : 1) {
+        int c = n0 + wn * WTN + j * 8 + (lane & 3) * 2;
         float v0 = acc[i][j][half * 2], v1 = acc[i][j][half * 2 + 1];
-        if (GELU) { v0 = gelu_erf(v0); v1 = gelu_erf(v1); }
-        if (c < n) out[(size_t)row * n + c] = from_f32<TO>(v0);
-        if (c + 1 < n) out[(size_t)row * n + c + 1] = from_f32<TO>(v1);
+        if (ACT == ACT_GELU) { v0 = gelu_erf(v0); v1 = gelu_erf(v1); }
+        if (ACT == ACT_SILU_UP) {
+          c = (n0 + wn * WTN + j * 8) / 2 + (lane & 3) * 2;
+          v0 = v0 / (1.f + expf(-v0)) * acc[i][j + (ACT == ACT_SILU_UP)][half * 2];
+          v1 = v1 / (1.f + expf(-v1)) * acc[i][j + (ACT == ACT_SILU_UP)][half * 2 + 1];
+        }
+        if (c < n_out) out[(size_t)row * n_out + c] = from_f32<TO>(v0);
+        if (c + 1 < n_out) out[(size_t)row * n_out + c + 1] = from_f32<TO>(v1);
       }
     }
 }
 
-__global__ void moe_combine_kernel(const float* __restrict__ y, const float* __restrict__ weights, int top,
-                                   const float* __restrict__ shared, const float* __restrict__ logits, int ld_logits,
-                                   int gate_col, float* __restrict__ resid, int width, const int* __restrict__ pair_pos) {
+struct CombineArgs {
+  const float *y, *weights;
+  int top;
+  const float* shared;          // [n_tokens, width] or null
+  const float* logits;
+  int ld_logits, gate_col;
+  float* resid;
+  int width;
+  const int* pair_pos;          // or null
+  const int* ids;               // with identity experts, else null
+  int n_experts;
+  const void* h;                // [n_tokens, width], rows of ld_h values
+  int ld_h;
+};
+
+template <typename T>
+__global__ void moe_combine_kernel(CombineArgs a) {
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
   float g = 0.f;
-  if (shared) g = 1.f / (1.f + expf(-logits[(size_t)t * ld_logits + gate_col]));
-  for (int c = threadIdx.x; c < width; c += blockDim.x) {
+  if (a.shared) g = 1.f / (1.f + expf(-a.logits[(size_t)t * a.ld_logits + a.gate_col]));
+  for (int c = threadIdx.x; c < a.width; c += blockDim.x) {
     float acc = 0.f;
-    for (int x = 0; x < top; ++x) {
-      const size_t pair = (size_t)t * top + x;
-      acc = fmaf(weights[pair], y[(pair_pos ? (size_t)pair_pos[pair] : pair) * width + c], acc);
+    for (int x = 0; x < a.top; ++x) {
+      const size_t pair = (size_t)t * a.top + x;
+      const float v = a.ids && a.ids[pair] >= a.n_experts
+                          ? to_f32(((const T*)a.h)[(size_t)t * a.ld_h + c])
+                          : a.y[(a.pair_pos ? (size_t)a.pair_pos[pair] : pair) * a.width + c];
+      acc = fmaf(a.weights[pair], v, acc);
     }
-    if (shared) acc = fmaf(g, shared[(size_t)t * width + c], acc);
-    resid[(size_t)t * width + c] += acc;
+    if (a.shared) acc = fmaf(g, a.shared[(size_t)t * a.width + c], acc);
+    a.resid[(size_t)t * a.width + c] += acc;
   }
 }
 
@@ -356,13 +466,19 @@ __global__ void gelu_kernel(const T* __restrict__ x, T* __restrict__ y, long lon
 
 using namespace tllm;
 
+// groups > 1: equal groups of neighbours of which `keep` stand for choice; renorm: the chosen scores over their sum.
 extern "C" int tllm_moe_route(const float* logits, int ld, int n_experts, const float* correction, float scale, int top,
-                              int* ids, float* weights, int n_tokens, int softmax, void* stream) {
+                              int* ids, float* weights, int n_tokens, int softmax, int renorm, int groups, int keep,
+                              void* stream) {
   TLLM_REQUIRE(n_tokens > 0 && n_experts > 0 && top > 0 && top <= n_experts, "moe_route: %d of %d experts for %d tokens", top, n_experts, n_tokens);
   TLLM_REQUIRE(n_experts <= 32 * ROUTE_PER_LANE, "moe_route: %d experts (at most %d)", n_experts, 32 * ROUTE_PER_LANE);
-  const int warps = 4;
-  TLLM_LAUNCH("moe_route", moe_route_kernel, (unsigned)((n_tokens + warps - 1) / warps), warps * 32, 0, (cudaStream_t)stream,
-              logits, ld, n_experts, correction, scale, top, ids, weights, n_tokens, softmax);
+  TLLM_REQUIRE(groups >= 1 && n_experts % groups == 0 && keep >= 1 && keep <= groups && top <= keep * (n_experts / groups),
+               "moe_route: %d of %d experts in the best %d of %d groups", top, n_experts, keep, groups);
+  RouteArgs a;
+  a.logits = logits; a.ld = ld; a.n_experts = n_experts; a.correction = correction; a.scale = scale; a.top = top; a.ids = ids;
+  a.weights = weights; a.n_tokens = n_tokens; a.softmax = softmax; a.renorm = renorm; a.groups = groups; a.keep = keep;
+  TLLM_LAUNCH("moe_route", moe_route_kernel, (unsigned)((n_tokens + ROUTE_WARPS - 1) / ROUTE_WARPS), ROUTE_WARPS * 32, 0,
+              (cudaStream_t)stream, a);
   return TLLM_OK;
 }
 
@@ -400,16 +516,22 @@ static int moe_linear_launch(const void* in, int ld_in, const void* w, const int
 }
 
 // in: [rows, k] rows of ld_in values; w: [experts, n, k]; out: [pairs, n] of out_dtype.  use_mma != 0: bfloat16 products
-// whose K and row stride are multiples of 8 run on the tensor cores; everything else on the FFMA kernel.
+// whose K and row stride are multiples of 8 run on the tensor cores; everything else on the FFMA kernel.  act: 0 the sums,
+// 1 GELU, 2 SiLU(gate) * up of rows in alternating blocks of glu_block (tensor cores and bfloat16 out only; out is n / 2
+// wide).
 extern "C" int tllm_moe_linear(const void* in, int ld_in, const void* w, const int* sorted_rows, const int* tile_expert,
-                               void* out, int n, int k, int rows_per_input, int tile, int max_tiles, int gelu, int dtype,
-                               int out_dtype, int use_mma, void* stream) {
+                               void* out, int n, int k, int rows_per_input, int tile, int max_tiles, int act, int glu_block,
+                               int dtype, int out_dtype, int use_mma, void* stream) {
+  const int gelu = act == ACT_GELU;
   TLLM_REQUIRE(n > 0 && k > 0 && rows_per_input > 0 && max_tiles > 0 && (tile == 16 || tile == 64 || tile == 128), "moe_linear: sizes do not fit (tile %d)", tile);
   TLLM_REQUIRE(tile != 128 || (dtype == TLLM_BF16 && use_mma && k % 8 == 0 && ld_in % 8 == 0 && ((uintptr_t)in & 15) == 0 && ((uintptr_t)w & 15) == 0),
                "moe_linear: tiles of 128 rows are the tensor-core kernel's");
   TLLM_REQUIRE(max_tiles <= 2147483647 && (n + 63) / 64 <= 65535, "moe_linear: the grid is too large");
   cudaStream_t s = (cudaStream_t)stream;
-  if (dtype == TLLM_BF16 && use_mma && k % 8 == 0 && ld_in % 8 == 0 && ((uintptr_t)in & 15) == 0 && ((uintptr_t)w & 15) == 0) {
+  const bool mma = dtype == TLLM_BF16 && use_mma && k % 8 == 0 && ld_in % 8 == 0 && ((uintptr_t)in & 15) == 0 && ((uintptr_t)w & 15) == 0;
+  TLLM_REQUIRE(act >= 0 && act <= 2 && (act != ACT_SILU_UP || (mma && out_dtype == TLLM_BF16 && glu_block > 0 && n % (2 * glu_block) == 0)),
+               "moe_linear: activation %d (SiLU*up: bfloat16 on the tensor cores, whole blocks of %d rows)", act, glu_block);
+  if (mma) {
     const dim3 grid((unsigned)max_tiles, (unsigned)((n + 127) / 128));
     TLLM_REQUIRE((n + 127) / 128 <= 65535, "moe_linear: the grid is too large");
 #define TLLM_MOE_MMA(TO, BM, G)                                                                                           \
@@ -422,17 +544,20 @@ extern "C" int tllm_moe_linear(const void* in, int ld_in, const void* w, const i
       configured = true;                                                                                                  \
     }                                                                                                                     \
     TLLM_LAUNCH("moe_linear", (moe_linear_mma_kernel<TO, BM, G>), grid, 256, smem, s, (const __nv_bfloat16*)in, ld_in,     \
-                (const __nv_bfloat16*)w, sorted_rows, tile_expert, (TO*)out, n, k, rows_per_input);                        \
+                (const __nv_bfloat16*)w, sorted_rows, tile_expert, (TO*)out, n, k, rows_per_input, glu_block);             \
   } while (0)
-#define TLLM_MOE_MMA_TILES(TO)                                                                      \
-  do {                                                                                              \
-    if (tile == 16) { if (gelu) TLLM_MOE_MMA(TO, 16, true); else TLLM_MOE_MMA(TO, 16, false); }      \
-    else if (tile == 64) { if (gelu) TLLM_MOE_MMA(TO, 64, true); else TLLM_MOE_MMA(TO, 64, false); } \
-    else { if (gelu) TLLM_MOE_MMA(TO, 128, true); else TLLM_MOE_MMA(TO, 128, false); }               \
-    return TLLM_OK;                                                                                 \
+#define TLLM_MOE_MMA_TILES(TO, G)                   \
+  do {                                              \
+    if (tile == 16) TLLM_MOE_MMA(TO, 16, G);        \
+    else if (tile == 64) TLLM_MOE_MMA(TO, 64, G);   \
+    else TLLM_MOE_MMA(TO, 128, G);                  \
+    return TLLM_OK;                                 \
   } while (0)
-    if (out_dtype == TLLM_BF16) TLLM_MOE_MMA_TILES(__nv_bfloat16);
-    if (out_dtype == TLLM_F32) TLLM_MOE_MMA_TILES(float);
+    if (act == ACT_SILU_UP) TLLM_MOE_MMA_TILES(__nv_bfloat16, ACT_SILU_UP);
+    if (out_dtype == TLLM_BF16 && gelu) TLLM_MOE_MMA_TILES(__nv_bfloat16, ACT_GELU);
+    if (out_dtype == TLLM_BF16) TLLM_MOE_MMA_TILES(__nv_bfloat16, ACT_NONE);
+    if (out_dtype == TLLM_F32 && gelu) TLLM_MOE_MMA_TILES(float, ACT_GELU);
+    if (out_dtype == TLLM_F32) TLLM_MOE_MMA_TILES(float, ACT_NONE);
 #undef TLLM_MOE_MMA_TILES
 #undef TLLM_MOE_MMA
   }
@@ -445,13 +570,21 @@ extern "C" int tllm_moe_linear(const void* in, int ld_in, const void* w, const i
   TLLM_FAIL(TLLM_ERR_ARG, "moe_linear: dtype codes %d -> %d", dtype, out_dtype);
 }
 
+// ids (with h, rows of ld_h values of h_dtype): choices of n_experts or above stand for the token's own row of h.
 extern "C" int tllm_moe_combine(const float* y, const float* weights, int top, const float* shared, const float* logits,
                                 int ld_logits, int gate_col, float* resid, int n_tokens, int width, const int* pair_pos,
-                                void* stream) {
+                                const int* ids, int n_experts, const void* h, int ld_h, int h_dtype, void* stream) {
   TLLM_REQUIRE(n_tokens > 0 && width > 0 && top > 0, "moe_combine: empty input");
   TLLM_REQUIRE(!shared || logits, "moe_combine: a shared expert needs its gate's logits");
-  TLLM_LAUNCH("moe_combine", moe_combine_kernel, (unsigned)n_tokens, width >= 1024 ? 256 : 128, 0, (cudaStream_t)stream, y, weights, top,
-              shared, logits, ld_logits, gate_col, resid, width, pair_pos);
+  TLLM_REQUIRE(!ids || h, "moe_combine: experts that hand their input on need it");
+  CombineArgs a;
+  a.y = y; a.weights = weights; a.top = top; a.shared = shared; a.logits = logits; a.ld_logits = ld_logits; a.gate_col = gate_col;
+  a.resid = resid; a.width = width; a.pair_pos = pair_pos; a.ids = ids; a.n_experts = n_experts; a.h = h; a.ld_h = ld_h;
+  const int threads = width >= 1024 ? 256 : 128;
+  cudaStream_t s = (cudaStream_t)stream;
+  if (h_dtype == TLLM_F32) TLLM_LAUNCH("moe_combine", moe_combine_kernel<float>, (unsigned)n_tokens, threads, 0, s, a);
+  else if (h_dtype == TLLM_BF16) TLLM_LAUNCH("moe_combine", moe_combine_kernel<__nv_bfloat16>, (unsigned)n_tokens, threads, 0, s, a);
+  else TLLM_FAIL(TLLM_ERR_ARG, "moe_combine: unknown dtype code %d", h_dtype);
   return TLLM_OK;
 }
 

@@ -2,8 +2,13 @@
 // a weighted sum of everything that came before them.  All float32; means and variances in two passes over values held
 // in registers or shared memory.
 //
-// layer_norm: out[r] = (x - mean) / sqrt(var + eps) * w + b with x = row rows[r] (or r), var the mean of the squared
+// layer_norm: out[r] = (x - mean) / sqrt(var + eps) * w (+ b) with x = row rows[r] (or r), var the mean of the squared
 //   deviations, rounded once to the output's type.
+// layer_norm_add: what a block does that norms a branch before it joins the stream, one kernel per branch:
+//     x <- x + n(branch),   next = n'(x)
+//   `branch` is a zeroed buffer that products added into and is handed back zeroed; `copy` receives the new stream in
+//   bfloat16, and `next`, where asked for, what the norm ahead of the following branch makes of it (the same sums in the
+//   same order as layer_norm's, so that it does not matter which kernel made them).
 // post_norm_join: what a block does that norms the SUM of the stream and a branch (post-norm), one kernel per branch:
 //     y = n(alpha * x + branch + out_bias),   x <- y
 //   `branch` is a zeroed buffer that products added into and is handed back zeroed; `copy` receives the new stream in
@@ -77,6 +82,15 @@ __device__ __forceinline__ void put4(__nv_bfloat16* p, float4 v) {
   *reinterpret_cast<__nv_bfloat162*>(&pk.x) = __floats2bfloat162_rn(v.x, v.y);
   *reinterpret_cast<__nv_bfloat162*>(&pk.y) = __floats2bfloat162_rn(v.z, v.w);
   *reinterpret_cast<uint2*>(p) = pk;
+}
+
+// (z - mean) * inv * w + b
+__device__ __forceinline__ float4 norm4(float4 z, float mean, float inv, float4 w, float4 b) {
+  return make_float4(fmaf((z.x - mean) * inv, w.x, b.x), fmaf((z.y - mean) * inv, w.y, b.y),
+                     fmaf((z.z - mean) * inv, w.z, b.z), fmaf((z.w - mean) * inv, w.w, b.w));
+}
+__device__ __forceinline__ float4 ldg4_or(const float* p, int idx, float4 other) {
+  return p != nullptr ? __ldg(reinterpret_cast<const float4*>(p) + idx) : other;
 }
 
 // The threads of a row depend on the width alone, so that a row's sums have the same order in every batch.
@@ -208,9 +222,8 @@ __global__ void layer_norm_vec_kernel(const float* __restrict__ x, const float* 
   for (int i = 0; i < VEC; ++i) {
     const int idx = threadIdx.x + i * blockDim.x;
     if (idx >= n4) continue;
-    const float4 wv = __ldg(reinterpret_cast<const float4*>(w) + idx), bv = __ldg(reinterpret_cast<const float4*>(b) + idx);
-    put4(out + (size_t)r * hidden + 4 * idx, make_float4(fmaf((z[i].x - mean) * inv, wv.x, bv.x), fmaf((z[i].y - mean) * inv, wv.y, bv.y),
-                                                          fmaf((z[i].z - mean) * inv, wv.z, bv.z), fmaf((z[i].w - mean) * inv, wv.w, bv.w)));
+    const float4 wv = __ldg(reinterpret_cast<const float4*>(w) + idx), bv = ldg4_or(b, idx, make_float4(0.f, 0.f, 0.f, 0.f));
+    put4(out + (size_t)r * hidden + 4 * idx, norm4(z[i], mean, inv, wv, bv));
   }
 }
 
@@ -238,7 +251,109 @@ __global__ void layer_norm_kernel(const float* __restrict__ x, const float* __re
   }
   ss = block_sum(ss, scratch);
   const float inv = 1.f / sqrtf(ss / (float)hidden + eps);
-  for (int i = threadIdx.x; i < hidden; i += blockDim.x) out[(size_t)r * hidden + i] = from_f32<T>(fmaf(row[i] * inv, w[i], b[i]));
+  for (int i = threadIdx.x; i < hidden; i += blockDim.x) out[(size_t)r * hidden + i] = from_f32<T>(fmaf(row[i] * inv, w[i], b ? b[i] : 0.f));
+}
+
+struct AddArgs {
+  float* branch;            // [rows, hidden]
+  float* x;                 // [rows, hidden]: the stream, in place
+  const float *w, *b;       // [hidden]; b may be null
+  float eps;
+  __nv_bfloat16* copy;      // [rows, hidden] or null
+  void* next;               // [rows, hidden] or null: the following norm's output
+  const float *next_w, *next_b;
+  float next_eps;
+  int n_rows, hidden;
+};
+
+template <typename T, int VEC>
+__global__ void layer_norm_add_vec_kernel(AddArgs a) {
+  __shared__ float2 moments[2][32];
+  __shared__ float counts[2][32];
+  pdl_trigger();
+  const int n4 = a.hidden / 4, r = blockIdx.x;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 w[VEC];   // constants of the model are read ahead of the wait
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    const int idx = threadIdx.x + i * blockDim.x;
+    w[i] = idx < n4 ? __ldg(reinterpret_cast<const float4*>(a.w) + idx) : zero;
+  }
+  pdl_wait();
+  if (r >= a.n_rows) return;
+  float4* br = reinterpret_cast<float4*>(a.branch + (size_t)r * a.hidden);
+  float4* xr = reinterpret_cast<float4*>(a.x + (size_t)r * a.hidden);
+  float4 z[VEC], x[VEC];
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    const int idx = threadIdx.x + i * blockDim.x;
+    z[i] = idx < n4 ? br[idx] : zero;
+    x[i] = idx < n4 ? xr[idx] : zero;
+  }
+  float mean, m2;
+  row_moments<VEC>(z, n4, moments[0], counts[0], mean, m2);
+  float inv = 1.f / sqrtf(m2 / (float)a.hidden + a.eps);
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    const int idx = threadIdx.x + i * blockDim.x;
+    if (idx >= n4) continue;
+    const float4 y = norm4(z[i], mean, inv, w[i], ldg4_or(a.b, idx, zero));
+    x[i] = make_float4(x[i].x + y.x, x[i].y + y.y, x[i].z + y.z, x[i].w + y.w);
+    xr[idx] = x[i];
+    br[idx] = zero;
+    if (a.copy != nullptr) put4(a.copy + (size_t)r * a.hidden + 4 * idx, x[i]);
+  }
+  if (a.next == nullptr) return;
+  row_moments<VEC>(x, n4, moments[1], counts[1], mean, m2);
+  inv = 1.f / sqrtf(m2 / (float)a.hidden + a.next_eps);
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    const int idx = threadIdx.x + i * blockDim.x;
+    if (idx >= n4) continue;
+    put4((T*)a.next + (size_t)r * a.hidden + 4 * idx,
+         norm4(x[i], mean, inv, __ldg(reinterpret_cast<const float4*>(a.next_w) + idx), ldg4_or(a.next_b, idx, zero)));
+  }
+}
+
+// Mean of a row in shared memory, which becomes the row of deviations (a thread meets the same elements in every pass);
+// returns 1 / sqrt(var + eps).
+__device__ __forceinline__ float center_row(float* row, int hidden, float eps, float* scratch) {
+  float sum = 0.f;
+  for (int i = threadIdx.x; i < hidden; i += blockDim.x) sum += row[i];
+  const float mean = block_sum(sum, scratch) / (float)hidden;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+    const float d = row[i] - mean;
+    row[i] = d;
+    ss += d * d;
+  }
+  ss = block_sum(ss, scratch);
+  return 1.f / sqrtf(ss / (float)hidden + eps);
+}
+
+// Any width: the row waits in shared memory.
+template <typename T>
+__global__ void layer_norm_add_kernel(AddArgs a) {
+  extern __shared__ float row[];
+  __shared__ float scratch[33];
+  pdl_trigger();
+  pdl_wait();
+  const int r = blockIdx.x;
+  if (r >= a.n_rows) return;
+  float* br = a.branch + (size_t)r * a.hidden;
+  float* xr = a.x + (size_t)r * a.hidden;
+  for (int i = threadIdx.x; i < a.hidden; i += blockDim.x) { row[i] = br[i]; br[i] = 0.f; }
+  float inv = center_row(row, a.hidden, a.eps, scratch);
+  for (int i = threadIdx.x; i < a.hidden; i += blockDim.x) {
+    const float x = xr[i] + fmaf(row[i] * inv, a.w[i], a.b ? a.b[i] : 0.f);
+    xr[i] = x;
+    row[i] = x;
+    if (a.copy) a.copy[(size_t)r * a.hidden + i] = __float2bfloat16_rn(x);
+  }
+  if (a.next == nullptr) return;
+  inv = center_row(row, a.hidden, a.next_eps, scratch);
+  for (int i = threadIdx.x; i < a.hidden; i += blockDim.x)
+    ((T*)a.next)[(size_t)r * a.hidden + i] = from_f32<T>(fmaf(row[i] * inv, a.next_w[i], a.next_b ? a.next_b[i] : 0.f));
 }
 
 __global__ void depth_average_kernel(float* __restrict__ x, float* __restrict__ stages, long long stage_stride, int n_stages,
@@ -296,7 +411,7 @@ extern "C" int tllm_post_norm_join(float* branch, float* x, const float* out_bia
 template <typename T>
 static int launch_layer_norm(const float* x, const float* w, const float* b, T* out, const int* rows, int n_rows, int hidden,
                              float eps, cudaStream_t s) {
-  const auto aligned = [](const void* p) { return ((uintptr_t)p % 16) == 0; };
+  const auto aligned = [](const void* p) { return ((uintptr_t)p % 16) == 0; };   // (null is)
   if (hidden % 4 == 0 && hidden <= 4 * 4 * 512 && aligned(x) && aligned(w) && aligned(b) && aligned(out)) {
     const int n4 = hidden / 4, threads = row_threads(n4), vec = (n4 + threads - 1) / threads;
     if (vec <= 1) TLLM_LAUNCH("layer_norm", (layer_norm_vec_kernel<T, 1>), n_rows, threads, 0, s, x, w, b, out, rows, n_rows, hidden, eps);
@@ -317,6 +432,38 @@ extern "C" int tllm_layer_norm(const float* x, const float* w, const float* b, v
   if (out_dtype == TLLM_F32) return launch_layer_norm<float>(x, w, b, (float*)out, rows, n_rows, hidden, eps, s);
   if (out_dtype == TLLM_BF16) return launch_layer_norm<__nv_bfloat16>(x, w, b, (__nv_bfloat16*)out, rows, n_rows, hidden, eps, s);
   TLLM_FAIL(TLLM_ERR_ARG, "layer_norm: unknown dtype code %d", out_dtype);
+}
+
+template <typename T>
+static int launch_layer_norm_add(const AddArgs& a, cudaStream_t s) {
+  const auto off = [](const void* p, int to) { return ((uintptr_t)p % to) != 0; };
+  if (a.hidden % 4 == 0 && a.hidden <= 4 * 4 * 512 && !off(a.branch, 16) && !off(a.x, 16) && !off(a.w, 16) && !off(a.b, 16) &&
+      !off(a.copy, 8) && !off(a.next, 16) && !off(a.next_w, 16) && !off(a.next_b, 16)) {
+    const int n4 = a.hidden / 4, threads = row_threads(n4), vec = (n4 + threads - 1) / threads;
+    if (vec <= 1) TLLM_LAUNCH("layer_norm_add", (layer_norm_add_vec_kernel<T, 1>), a.n_rows, threads, 0, s, a);
+    else if (vec == 2) TLLM_LAUNCH("layer_norm_add", (layer_norm_add_vec_kernel<T, 2>), a.n_rows, threads, 0, s, a);
+    else TLLM_LAUNCH("layer_norm_add", (layer_norm_add_vec_kernel<T, 4>), a.n_rows, threads, 0, s, a);
+    return TLLM_OK;
+  }
+  TLLM_REQUIRE(a.hidden <= MAX_WIDTH, "layer_norm_add: rows of %d values (at most %d)", a.hidden, MAX_WIDTH);
+  const int threads = a.hidden >= 2048 ? 512 : (a.hidden >= 512 ? 256 : 128);
+  TLLM_LAUNCH("layer_norm_add", layer_norm_add_kernel<T>, a.n_rows, threads, a.hidden * 4, s, a);
+  return TLLM_OK;
+}
+
+// next (of next_dtype), next_w, next_b, next_eps: the norm ahead of the following branch; next null: none.
+extern "C" int tllm_layer_norm_add(float* branch, float* x, const float* w, const float* b, float eps, void* copy_bf16,
+                                   void* next, const float* next_w, const float* next_b, float next_eps, int next_dtype,
+                                   int n_rows, int hidden, void* stream) {
+  TLLM_REQUIRE(n_rows > 0 && hidden > 0 && branch && x && w, "layer_norm_add: %d rows of %d values", n_rows, hidden);
+  TLLM_REQUIRE(next == nullptr || next_w != nullptr, "layer_norm_add: the following norm needs a weight");
+  AddArgs a;
+  a.branch = branch; a.x = x; a.w = w; a.b = b; a.eps = eps; a.copy = (__nv_bfloat16*)copy_bf16; a.next = next;
+  a.next_w = next_w; a.next_b = next_b; a.next_eps = next_eps; a.n_rows = n_rows; a.hidden = hidden;
+  cudaStream_t s = (cudaStream_t)stream;
+  if (next_dtype == TLLM_F32) return launch_layer_norm_add<float>(a, s);
+  if (next_dtype == TLLM_BF16) return launch_layer_norm_add<__nv_bfloat16>(a, s);
+  TLLM_FAIL(TLLM_ERR_ARG, "layer_norm_add: unknown dtype code %d", next_dtype);
 }
 
 extern "C" int tllm_depth_average(float* x, float* stages, long long stage_stride, int n_stages, int keep, const float* mix,

@@ -262,9 +262,9 @@ def min_gru_scan(zug: torch.Tensor, bias_z: torch.Tensor, bias_u: torch.Tensor, 
           _ptr(summary), _code(zug.dtype), _stream())
 
 
-# what a gated feed-forward makes of gate and up: silu(g) u, relu(g) u, or the clamped form
-# min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u, -limit, limit) + 1)
-GLU_ACTS = {"silu": 0, "relu": 1, "clamped": 2}
+# what a gated feed-forward makes of gate and up: silu(g) u, relu(g) u, the clamped form
+# min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u, -limit, limit) + 1), or gelu(g) u with the tanh form of GELU
+GLU_ACTS = {"silu": 0, "relu": 1, "clamped": 2, "gelu_tanh": 3}
 
 
 def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, block: int, consume: bool = False, act: str = "silu",
@@ -554,9 +554,11 @@ def gelu(x: torch.Tensor, out: torch.Tensor) -> None:
 
 
 def moe_route(logits: torch.Tensor, num_experts: int, correction: Optional[torch.Tensor], scale: float, ids: torch.Tensor,
-              weights: torch.Tensor, softmax: bool = False) -> None:
+              weights: torch.Tensor, softmax: bool = False, renorm: bool = False, groups: int = 1, keep: int = 1) -> None:
     """Per token: s = sigmoid(logits[t, :num_experts]), or softmax over the experts with softmax=True; ids[t] = the `top`
-    experts with the largest s + correction (None: s; ties: the lower index), weights[t] = their s * scale.  logits
+    experts with the largest s + correction (None: s; ties: the lower index), weights[t] = their s * scale, or with
+    renorm=True s / (sum of the chosen s + 1e-20) * scale.  groups > 1: that many equal groups of neighbours, each worth
+    its largest s + correction; only members of the best `keep` groups stand for choice.  logits
     float32 (further columns are ignored), ids int32 [T, top], weights float32 [T, top]."""
     _need_cuda(logits, correction, ids, weights)
     t, top = ids.shape
@@ -567,7 +569,7 @@ def moe_route(logits: torch.Tensor, num_experts: int, correction: Optional[torch
         raise KernelError("moe_route: shapes or dtypes do not fit")
     lib = build.load_library("moe")
     _call(lib, lib.tllm_moe_route, _ptr(logits), logits.stride(0), num_experts, _ptr(correction), ctypes.c_float(scale), top,
-          _ptr(ids), _ptr(weights), t, 1 if softmax else 0, _stream())
+          _ptr(ids), _ptr(weights), t, 1 if softmax else 0, 1 if renorm else 0, groups, keep, _stream())
 
 
 def moe_tile_rows(pairs: int, num_experts: int, tensor_cores: bool = False) -> int:
@@ -587,7 +589,8 @@ def moe_align(ids: torch.Tensor, num_experts: int, tile: int, sorted_rows: torch
               pair_pos: Optional[torch.Tensor] = None) -> None:
     """Groups the pairs (token, choice), numbered in the order of `ids`, by expert into tiles of `tile` rows:
     sorted_rows[tiles * tile] (pair numbers, -1 = padding) and tile_expert[tiles] (-1 = no such tile); with `pair_pos`
-    (int32 [pairs]) also where every pair's row lies in that order."""
+    (int32 [pairs]) also where every pair's row lies in that order.  Pairs with an id of num_experts or above are left
+    out (pair_pos -1)."""
     _need_cuda(ids, sorted_rows, tile_expert, pair_pos)
     _i32(pair_pos, "pair_pos")
     if pair_pos is not None and pair_pos.numel() != ids.numel():
@@ -629,20 +632,23 @@ def moe_gather(a: torch.Tensor, sorted_rows: torch.Tensor, tile_expert: torch.Te
           rows_per_input, _ptr(out), k, _stream())
 
 
-def moe_linear_tc(a: torch.Tensor, w: torch.Tensor, tile_expert: torch.Tensor, out: torch.Tensor, gelu: bool = False) -> None:
+def moe_linear_tc(a: torch.Tensor, w: torch.Tensor, tile_expert: torch.Tensor, out: torch.Tensor, gelu: bool = False,
+                  silu_up: bool = False) -> None:
     """The grouped product on tcgen05: a [tiles * 128, K] bfloat16 in the grouped order (every tile of 128 rows one
-    expert's), w [experts, N, K]; out [tiles * 128, N]: bfloat16 of GELU(sums) with gelu=True, else float32 sums."""
+    expert's), w [experts, N, K]; out [tiles * 128, N]: bfloat16 of GELU(sums) with gelu=True, else float32 sums; with
+    silu_up=True [tiles * 128, N / 2]: bfloat16 of SiLU(gate) * up, every expert's gate and up rows interleaved in blocks
+    of 128."""
     _need_cuda(a, w, tile_expert, out)
     _i32(tile_expert, "tile_expert")
     experts, n, k = w.shape
     rows = tile_expert.numel() * MOE_TC_TILE
     if a.shape != (rows, k) or a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or not w.is_contiguous() or \
-            a.stride(1) != 1 or out.shape != (rows, n) or out.stride(1) != 1 or \
-            out.dtype != (torch.bfloat16 if gelu else torch.float32):
+            a.stride(1) != 1 or out.shape != (rows, n // 2 if silu_up else n) or out.stride(1) != 1 or (gelu and silu_up) or \
+            (silu_up and n % 256) or out.dtype != (torch.bfloat16 if gelu or silu_up else torch.float32):
         raise KernelError("moe_linear_tc: shapes or dtypes do not fit")
     lib = build.load_library("linear_tc")
     _call(lib, lib.tllm_linear_tc_grouped, _ptr(a), _ptr(w), _ptr(out), rows, n, k, a.stride(0), out.stride(0), experts,
-          _ptr(tile_expert), 10 if gelu else EPI_F32, _ptr(status_word(a.device)), _stream())
+          _ptr(tile_expert), 10 if gelu else EPI_SWIGLU if silu_up else EPI_F32, _ptr(status_word(a.device)), _stream())
 
 
 # bfloat16 grouped products on the tensor cores (0: the FFMA kernel, for comparisons)
@@ -652,37 +658,51 @@ moe_mma = os.environ.get("TLLM_MOE_MMA", "1") != "0"
 moe_wide_tiles = os.environ.get("TLLM_MOE_TILE_128", "0") == "1"
 
 
+def moe_silu_up_fused(a: torch.Tensor, w: torch.Tensor) -> bool:
+    """Whether `moe_linear` takes SiLU(gate) * up inside the product: bfloat16 on the tensor cores."""
+    return (a.dtype == torch.bfloat16 and moe_mma and not force_generic and w.shape[2] % 8 == 0 and a.stride(0) % 8 == 0 and
+            a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
+
+
 def moe_linear(a: torch.Tensor, w: torch.Tensor, sorted_rows: torch.Tensor, tile_expert: torch.Tensor, tile: int,
-               out: torch.Tensor, rows_per_input: int = 1, gelu: bool = False) -> None:
+               out: torch.Tensor, rows_per_input: int = 1, gelu: bool = False, silu_up_block: int = 0) -> None:
     """out[p] = act(w[expert of p] . a[p // rows_per_input]) for every pair p named in sorted_rows; w [experts, N, K],
-    out [pairs, N] in a's dtype or float32; act is the exact GELU or nothing."""
+    out [pairs, N] in a's dtype or float32; act is the exact GELU or nothing.  silu_up_block > 0: gate and up rows of w
+    alternate in blocks of that many and out [pairs, N / 2] is SiLU(gate) * up (only where `moe_silu_up_fused` says so)."""
     _need_cuda(a, w, sorted_rows, tile_expert, out)
     n, k = w.shape[1], w.shape[2]
-    if a.shape[1] != k or a.stride(1) != 1 or a.dtype != w.dtype or not w.is_contiguous() or out.shape[1] != n or \
+    if a.shape[1] != k or a.stride(1) != 1 or a.dtype != w.dtype or not w.is_contiguous() or \
+            out.shape[1] != (n // 2 if silu_up_block else n) or \
             not out.is_contiguous() or out.dtype not in (a.dtype, torch.float32):
         raise KernelError("moe_linear: shapes or dtypes do not fit")
     lib = build.load_library("moe")
     _call(lib, lib.tllm_moe_linear, _ptr(a), a.stride(0), _ptr(w), _ptr(sorted_rows), _ptr(tile_expert), _ptr(out), n, k,
-          rows_per_input, tile, tile_expert.numel(), 1 if gelu else 0, _code(a.dtype), _code(out.dtype),
+          rows_per_input, tile, tile_expert.numel(), 2 if silu_up_block else 1 if gelu else 0, silu_up_block, _code(a.dtype), _code(out.dtype),
           1 if (moe_mma and not force_generic) else 0, _stream())
 
 
 def moe_combine(y: torch.Tensor, weights: torch.Tensor, shared: Optional[torch.Tensor], logits: Optional[torch.Tensor],
-                gate_col: int, resid: torch.Tensor, pair_pos: Optional[torch.Tensor] = None) -> None:
+                gate_col: int, resid: torch.Tensor, pair_pos: Optional[torch.Tensor] = None,
+                ids: Optional[torch.Tensor] = None, num_experts: int = 0, h: Optional[torch.Tensor] = None) -> None:
     """resid[t] += sum_c weights[t, c] * y[t * top + c] + sigmoid(logits[t, gate_col]) * shared[t] (the last term only
-    with `shared`); all float32.  With `pair_pos` (int32 [T * top]) y is in the grouped order: pair p lies in row pair_pos[p]."""
-    _need_cuda(y, weights, shared, logits, resid, pair_pos)
+    with `shared`); all float32.  With `pair_pos` (int32 [T * top]) y is in the grouped order: pair p lies in row pair_pos[p].
+    With `ids` (int32 [T, top]) a choice of num_experts or above stands for the token's own input row h[t]."""
+    _need_cuda(y, weights, shared, logits, resid, pair_pos, ids, h)
     _i32(pair_pos, "pair_pos")
+    _i32(ids, "ids")
     t, width = resid.shape
     top = weights.shape[1]
     if (pair_pos is None and y.shape != (t * top, width)) or y.shape[1] != width or \
             (pair_pos is not None and pair_pos.numel() != t * top) or any(x.dtype != torch.float32 or not x.is_contiguous() for x in (y, weights, resid)) or \
+            (ids is not None and (ids.shape != weights.shape or h is None or h.shape != resid.shape or h.stride(1) != 1)) or \
             (shared is not None and (shared.shape != resid.shape or shared.dtype != torch.float32 or not shared.is_contiguous()
                                      or logits is None or logits.dtype != torch.float32 or logits.shape[1] <= gate_col)):
         raise KernelError("moe_combine: shapes or dtypes do not fit")
     lib = build.load_library("moe")
     _call(lib, lib.tllm_moe_combine, _ptr(y), _ptr(weights), top, _ptr(shared), _ptr(logits),
-          0 if logits is None else logits.stride(0), gate_col, _ptr(resid), t, width, _ptr(pair_pos), _stream())
+          0 if logits is None else logits.stride(0), gate_col, _ptr(resid), t, width, _ptr(pair_pos), _ptr(ids), num_experts,
+          _ptr(h if ids is not None else None), h.stride(0) if ids is not None else 0,
+          _code(h.dtype) if ids is not None else F32, _stream())
 
 
 # ----------------------------------------------------------------------------- attention without rotate-half, delta rule
@@ -777,14 +797,17 @@ def conv_norm_kv_write(proj: torch.Tensor, batch, num_heads: int, num_kv_heads: 
                        k_cache: torch.Tensor, v_cache: torch.Tensor, slot_mapping: torch.Tensor, q_out: torch.Tensor,
                        bias: Optional[torch.Tensor] = None, taps: Optional[torch.Tensor] = None,
                        kept: Optional[torch.Tensor] = None, norm_q: Optional[torch.Tensor] = None,
-                       norm_k: Optional[torch.Tensor] = None, eps: float = 0.0) -> None:
+                       norm_k: Optional[torch.Tensor] = None, eps: float = 0.0, freq: Optional[torch.Tensor] = None,
+                       rot_pairs: bool = False, rot_mag: float = 1.0) -> None:
     """Rows of `proj` begin with num_heads query heads and num_kv_heads key heads of key_dim values, then num_kv_heads
     value heads of value_dim values.  With x = row + bias (float32 [channels]) every channel is filtered over time,
     y_t = sum_j taps[j] x_(t - n + 1 + j) (taps float32 [n, channels], zeros before the sequence's start; the last
     n - 1 inputs lie in kept[slot], float32 [slots, n - 1, channels], and are brought up to date); then all query values
     of a token together become y / sqrt(mean(y^2) + eps) * norm_q (float32 [num_heads * key_dim]), and all its key values
     the same with norm_k.  Queries go to q_out [T, num_heads * key_dim], keys and values to their pages; `proj` stays as
-    it is.  Without taps there is no filter, without norm weights no norm."""
+    it is.  Without taps there is no filter, without norm weights no norm.  With `freq` (float32 [r / 2]) the first r
+    values of every query and key head are then rotated by positions[t] * freq[i] (value i with i + r / 2, or with
+    rot_pairs 2i with 2i + 1; cos and sin times rot_mag), in 32-bit."""
     _need_cuda(proj, k_cache, v_cache, slot_mapping, q_out, bias, taps, kept, norm_q, norm_k)
     _i32(slot_mapping, "slot_mapping")
     t = proj.shape[0]
@@ -804,6 +827,10 @@ def conv_norm_kv_write(proj: torch.Tensor, batch, num_heads: int, num_kv_heads: 
             raise KernelError(f"conv_norm_kv_write: the {name} must be contiguous float32 of shape {shape}")
     if n > 1 and (kept is None or kept.dtype != torch.float32 or not kept.is_contiguous() or tuple(kept.shape[1:]) != (n - 1, channels)):
         raise KernelError(f"conv_norm_kv_write: the kept inputs must be contiguous float32 [slots, {n - 1}, {channels}]")
+    _need_cuda(freq)
+    rot_dims = 0 if freq is None else 2 * freq.numel()
+    if freq is not None and (freq.dtype != torch.float32 or not freq.is_contiguous() or rot_dims > key_dim):
+        raise KernelError("conv_norm_kv_write: the frequency table does not fit")
     single = batch.max_q_len == 1     # then the one token of a request also moves its kept inputs up
     ll = ctypes.c_longlong
     lib = build.load_library("attention_prep")
@@ -811,7 +838,8 @@ def conv_norm_kv_write(proj: torch.Tensor, batch, num_heads: int, num_kv_heads: 
           _ptr(bias), _ptr(taps), n, _ptr(kept if n > 1 else None), _ptr(batch.slots), _ptr(batch.cu_q), _ptr(batch.token_request),
           _ptr(norm_q), _ptr(norm_k), ctypes.c_float(eps), _ptr(q_out), _ptr(k_cache), _ptr(v_cache), _ptr(slot_mapping),
           k_cache.shape[2], ll(k_cache.stride(0)), ll(k_cache.stride(1)), ll(v_cache.stride(0)), ll(v_cache.stride(1)), t,
-          1 if single else 0, _code(proj.dtype), _stream())
+          1 if single else 0, _ptr(batch.positions if rot_dims else None), _ptr(freq), rot_dims, 1 if rot_pairs else 0,
+          ctypes.c_float(rot_mag), _code(proj.dtype), _stream())
     if n > 1 and not single:
         conv_state_update(proj, kept, batch, n, channels, bias=bias)
 
@@ -956,20 +984,39 @@ def bigram_add(tokens: torch.Tensor, table: torch.Tensor, last: torch.Tensor, ba
           _code(table.dtype), _stream())
 
 
-def layer_norm(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, eps: float, out: torch.Tensor,
+def layer_norm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float, out: torch.Tensor,
                rows: Optional[torch.Tensor] = None) -> None:
-    """out[r, :] = (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps) * weight + bias with v = x[rows[r], :]; x, weight
-    and bias are float32."""
+    """out[r, :] = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight + bias with x = x[rows[r], :]; x, weight and bias
+    (None: no bias) are float32."""
     _need_cuda(x, weight, bias, out, rows)
     _i32(rows, "rows")
     h, n = x.shape[1], out.shape[0]
-    if any(v.dtype != torch.float32 or not v.is_contiguous() for v in (x, weight, bias)) or not out.is_contiguous() or \
-            out.shape[1] != h or weight.numel() != h or bias.numel() != h or \
+    if any(v.dtype != torch.float32 or not v.is_contiguous() for v in (x, weight)) or not out.is_contiguous() or \
+            out.shape[1] != h or weight.numel() != h or \
+            (bias is not None and (bias.dtype != torch.float32 or not bias.is_contiguous() or bias.numel() != h)) or \
             (rows is None and n != x.shape[0]) or (rows is not None and rows.numel() != n):
         raise KernelError("layer_norm: shapes or dtypes do not fit")
     lib = build.load_library("post_norm")
     _call(lib, lib.tllm_layer_norm, _ptr(x), _ptr(weight), _ptr(bias), _ptr(out), _ptr(rows), n, h, ctypes.c_float(eps),
           _code(out.dtype), _stream())
+
+
+def layer_norm_add(branch: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float,
+                   copy: Optional[torch.Tensor] = None, then=None, out: Optional[torch.Tensor] = None) -> None:
+    """x += layer_norm(branch), row by row, all float32; `branch` is handed back zeroed (products add into it) and `copy`
+    (bfloat16) receives the new stream rounded.  With `then` = (weight, bias, eps) `out` [T, H] receives what that layer
+    norm makes of the new stream (the bits `layer_norm` would give)."""
+    w2, b2, eps2 = then if then is not None else (None, None, 0.0)
+    _need_cuda(branch, x, weight, bias, copy, w2, b2, out)
+    h = x.shape[1]
+    if any(v.dtype != torch.float32 or not v.is_contiguous() for v in (branch, x)) or branch.shape != x.shape or \
+            any(v is not None and (v.dtype != torch.float32 or v.numel() != h or not v.is_contiguous()) for v in (weight, bias, w2, b2)) or \
+            (copy is not None and (copy.dtype != torch.bfloat16 or copy.shape != x.shape or not copy.is_contiguous())) or \
+            (then is None) != (out is None) or (out is not None and (out.shape != x.shape or not out.is_contiguous())):
+        raise KernelError("layer_norm_add: shapes or dtypes do not fit")
+    lib = build.load_library("post_norm")
+    _call(lib, lib.tllm_layer_norm_add, _ptr(branch), _ptr(x), _ptr(weight), _ptr(bias), ctypes.c_float(eps), _ptr(copy),
+          _ptr(out), _ptr(w2), _ptr(b2), ctypes.c_float(eps2), F32 if out is None else _code(out.dtype), x.shape[0], h, _stream())
 
 
 def _check_stages(name: str, x: torch.Tensor, stages: torch.Tensor, done: int, mix: torch.Tensor, keep: bool) -> None:
@@ -1036,6 +1083,15 @@ def unary(x: torch.Tensor, out: torch.Tensor, act: str = "copy") -> None:
     lib = build.load_library("elementwise")
     _call(lib, lib.tllm_unary, _ptr(x), _ptr(out), ctypes.c_longlong(x.numel()), _code(x.dtype), _code(out.dtype),
           UNARY_ACTS[act], _stream())
+
+
+def soft_cap(x: torch.Tensor, scale: float = 1.0, cap: Optional[float] = None) -> None:
+    """x <- cap * tanh(scale * x / cap) in place (no cap: scale * x), float32."""
+    _need_cuda(x)
+    if x.dtype != torch.float32 or not x.is_contiguous() or (cap is not None and not cap > 0):
+        raise KernelError("soft_cap: a contiguous float32 tensor and a positive cap (or none)")
+    lib = build.load_library("elementwise")
+    _call(lib, lib.tllm_soft_cap, _ptr(x), ctypes.c_longlong(x.numel()), ctypes.c_float(scale), ctypes.c_float(cap or 0.0), _stream())
 
 
 def scaled_add(x: torch.Tensor, scale: float, resid: torch.Tensor, clear: bool = True) -> None:
@@ -1135,7 +1191,7 @@ def attention_talk(q: torch.Tensor, num_heads: int, num_kv_heads: int, key_dim: 
 
 
 EPI_BF16, EPI_F32, EPI_ADD_F32, EPI_SWIGLU, EPI_ATOMIC_F32 = 0, 1, 2, 3, 4
-EPI_GLU_CLAMPED = 11                               # EPI_SWIGLU with the clamped gate
+EPI_GLU_CLAMPED, EPI_GLU_GELU = 11, 12             # EPI_SWIGLU with the clamped gate, with the tanh form of GELU
 EPI_CL_ADD_F32, EPI_CL_ROPE_KV, EPI_CL_SWIGLU, EPI_CL_BF16 = 5, 6, 7, 8   # K slices reduced inside a thread-block cluster
 _sm_count = {}
 
@@ -1221,7 +1277,7 @@ def _cluster_slices(n: int, k: int, limit: int = 8) -> int:
 
 
 def _cluster_call(epi, a, w, out, slices, positions=None, cos=None, sin=None, nq=0, nkv=0, hd=0, k_cache=None,
-                  v_cache=None, slot_mapping=None, limit=0.0):
+                  v_cache=None, slot_mapping=None, act=0, limit=0.0):
     lib = build.load_library("linear_tc")
     m, k = a.shape
     page_size = page_stride = head_stride = 0
@@ -1230,7 +1286,7 @@ def _cluster_call(epi, a, w, out, slices, positions=None, cos=None, sin=None, nq
     _call(lib, lib.tllm_linear_tc_cluster,
         _ptr(a), _ptr(w), _ptr(out), m, w.shape[0], k, a.stride(0), out.stride(0), epi, slices, _ptr(positions),
         _ptr(cos), _ptr(sin), nq, nkv, hd, _ptr(k_cache), _ptr(v_cache), _ptr(slot_mapping), page_size,
-        ctypes.c_longlong(page_stride), ctypes.c_longlong(head_stride), ctypes.c_float(limit), _ptr(status_word(a.device)), _stream())
+        ctypes.c_longlong(page_stride), ctypes.c_longlong(head_stride), act, ctypes.c_float(limit), _ptr(status_word(a.device)), _stream())
 
 
 def linear_rope_kv(h: torch.Tensor, w_qkv: torch.Tensor, qkv: torch.Tensor, positions: torch.Tensor,
@@ -1338,8 +1394,8 @@ def linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate: bool
 def linear_swiglu(a: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, block: int, workspace,
                   act: str = "silu", limit: float = 0.0) -> None:
     """out = act(a Wg^T) * (a Wu^T) with Wg, Wu interleaved in `w_gate_up` in row blocks of `block`; act one of GLU_ACTS.
-    With blocks of 128 the product and the gate are one tensor-core kernel (SiLU and the clamped form: another activation
-    takes the product and the element-wise kernel)."""
+    With blocks of 128 the product and the gate are one tensor-core kernel (ReLU takes the product and the element-wise
+    kernel)."""
     m = a.shape[0]
     n2 = w_gate_up.shape[0]
     if act not in GLU_ACTS or (act == "clamped" and not limit > 0):
@@ -1359,14 +1415,14 @@ def linear_swiglu(a: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, b
         _need_cuda(a, w_gate_up, out)
         lib = build.load_library("linear_tc")
         _call(lib, lib.tllm_linear_tc, _ptr(a), _ptr(w_gate_up), _ptr(out), m, n2, a.shape[1], a.stride(0),
-                                       out.stride(0), EPI_GLU_CLAMPED if act == "clamped" else EPI_SWIGLU, 0, 1,
+                                       out.stride(0), {"silu": EPI_SWIGLU, "clamped": EPI_GLU_CLAMPED, "gelu_tanh": EPI_GLU_GELU}[act], 0, 1,
                                        ctypes.c_float(limit), _ptr(status_word(a.device)), _stream())
         return
     if (cluster_mask & 4) and _tc_ok(a, w_gate_up, out) and block == 128 and m <= 128 and n2 % 256 == 0 and \
             out.stride(1) == 1 and w_gate_up.is_contiguous():
         # the gate tile, the up tile beside it and their K slices form one cluster; SiLU * up in its epilogue
         _need_cuda(a, w_gate_up, out)
-        _cluster_call(EPI_CL_SWIGLU, a, w_gate_up, out, _cluster_slices(n2, a.shape[1], limit=4), limit=limit)
+        _cluster_call(EPI_CL_SWIGLU, a, w_gate_up, out, _cluster_slices(n2, a.shape[1], limit=4), act=GLU_ACTS[act], limit=limit)
         return
     if prefers_split(a, w_gate_up):
         acc = workspace.get_zeroed("gate_up_f32", (m, n2))

@@ -13,8 +13,13 @@ of the stacked weights); smaller steps gather their rows inside an `mma.sync` (b
 
 Variants, chosen by parameters.  `router="softmax"`: s = softmax(z) over all experts (the weights are still the chosen
 experts' s * route_scale, not renormalised).  `correction=False`: the choice reads s alone and no correction tensor is
-stored.  `glu="silu"` (or "relu"): an expert is W_down (act(W_gate h) * (W_up h)); its gate and up matrices are stacked
-into one grouped product whose halves an element-wise kernel joins."""
+stored.  `renorm=True`: the weights are s / (sum of the chosen s + 1e-20) * route_scale.  `groups` > 1: the experts form
+that many equal groups of neighbours, a group is worth its largest s + correction, and only members of the best `keep`
+groups stand for choice.  `identity` > 0: that many further experts behind the others take part in the router, the
+correction and the groups, have no matrices, and give back the input h itself (times their weight).  `glu="silu"` (or
+"relu"): an expert is W_down (act(W_gate h) * (W_up h)); its gate and up rows are interleaved in blocks of one grouped
+product, which takes SiLU * up in its epilogue (bfloat16; otherwise an element-wise kernel joins the halves); a shared
+expert is then of the same form and, with `shared_gate=False`, added as it is."""
 from __future__ import annotations
 
 from typing import Optional
@@ -23,7 +28,7 @@ import torch
 
 from .. import ops
 from ..weights import COMPUTE, FLOAT32, WeightSpec
-from .feed_forward import scaled_matrix
+from .feed_forward import SwiGLU, gate_up_block, interleave_gate_up, scaled_matrix
 from .registry import register_part
 
 
@@ -32,15 +37,23 @@ class RoutedExperts:
 
     def __init__(self, hidden_size: int, num_experts: int, top: int, expert_size: int, route_scale: float = 1.0,
                  shared_size: Optional[int] = None, out_scale: float = 1.0, router: str = "sigmoid",
-                 correction: bool = True, glu: Optional[str] = None):
-        if not 0 < top <= num_experts:
-            raise ValueError(f"{top} of {num_experts} experts cannot be chosen")
+                 correction: bool = True, glu: Optional[str] = None, renorm: bool = False, groups: int = 1, keep: int = 1,
+                 identity: int = 0, shared_gate: bool = True):
+        routed = num_experts + identity     # what the router chooses from
+        if identity < 0 or not 0 < top <= routed:
+            raise ValueError(f"{top} of {routed} experts cannot be chosen")
+        if groups < 1 or routed % groups or not 1 <= keep <= groups or top > keep * (routed // groups):
+            raise ValueError(f"{top} of {routed} experts cannot be chosen in {keep} of {groups} equal groups")
         if router not in ("sigmoid", "softmax"):
             raise ValueError(f"unknown router {router!r}; known: sigmoid, softmax")
         if glu is not None and glu not in ops.GLU_ACTS:
             raise ValueError(f"unknown gate activation {glu!r}; known: {', '.join(ops.GLU_ACTS)}")
-        if glu is not None and shared_size is not None:
-            raise ValueError("a shared expert beside gated experts is not built")
+        if shared_size is not None and shared_gate != (glu is None):
+            raise ValueError("a shared expert has a gate per token beside experts without gates, none beside gated ones")
+        self.renorm, self.groups, self.keep, self.identity, self.routed = renorm, groups, keep, identity, routed
+        self.block = gate_up_block(expert_size)
+        self.shared = None if glu is None or shared_size is None else \
+            SwiGLU(hidden_size, shared_size, names=("gate", "up", "down"), out_scale=out_scale, act=glu)
         self.router, self.has_correction, self.glu = router, correction, glu
         self.hidden_size, self.num_experts, self.top = hidden_size, num_experts, top
         self.expert_size, self.shared_size = expert_size, shared_size
@@ -50,14 +63,17 @@ class RoutedExperts:
 
     def weight_specs(self, prefix: str):
         h, f = self.hidden_size, self.expert_size
-        specs = [WeightSpec(prefix + "router", (self.num_experts, h), COMPUTE)]
-        if self.has_correction:
-            specs.append(WeightSpec(prefix + "correction", (self.num_experts,), FLOAT32, init=("normal", 0.3)))
+        specs = [WeightSpec(prefix + "router", (self.routed, h), COMPUTE)]
+        if self.has_correction:   # (a softmax's scores lie around 1 / routed: corrections of their size)
+            specs.append(WeightSpec(prefix + "correction", (self.routed,), FLOAT32,
+                                    init=("normal", 0.3 if self.router == "sigmoid" else 0.3 / self.routed)))
         for e in range(self.num_experts):
             if self.glu is not None:
                 specs.append(WeightSpec(prefix + f"e{e}.gate", (f, h), COMPUTE))
             specs += [WeightSpec(prefix + f"e{e}.up", (f, h), COMPUTE), WeightSpec(prefix + f"e{e}.down", (h, f), COMPUTE)]
-        if self.shared_size is not None:
+        if self.shared is not None:
+            specs += self.shared.weight_specs(prefix + "shared.")
+        elif self.shared_size is not None:
             specs += [WeightSpec(prefix + "shared.up", (self.shared_size, h), COMPUTE),
                       WeightSpec(prefix + "shared.down", (h, self.shared_size), COMPUTE),
                       WeightSpec(prefix + "shared.sg", (1, h), COMPUTE)]
@@ -65,16 +81,18 @@ class RoutedExperts:
 
     def load(self, prefix: str, weights) -> None:
         n = self.num_experts
-        rows = [weights[prefix + "router"]] + ([weights[prefix + "shared.sg"]] if self.shared_size is not None else [])
+        rows = [weights[prefix + "router"]] + ([weights[prefix + "shared.sg"]] if self.shared_size is not None and self.shared is None else [])
         self.w_route = torch.cat(rows, dim=0).contiguous()
         self.correction = weights[prefix + "correction"] if self.has_correction else None
-        if self.glu is not None:   # per expert [gate rows | up rows]: one grouped product gives both halves
-            self.w_up = torch.stack([torch.cat([weights[prefix + f"e{e}.gate"], weights[prefix + f"e{e}.up"]], dim=0)
+        if self.glu is not None:   # per expert blocks of gate rows and their up rows: one grouped product gives both halves
+            self.w_up = torch.stack([interleave_gate_up(weights[prefix + f"e{e}.gate"], weights[prefix + f"e{e}.up"], self.block)
                                      for e in range(n)]).contiguous()
         else:
             self.w_up = torch.stack([weights[prefix + f"e{e}.up"] for e in range(n)]).contiguous()
         self.w_down = torch.stack([scaled_matrix(weights[prefix + f"e{e}.down"], self.out_scale) for e in range(n)]).contiguous()
-        if self.shared_size is not None:
+        if self.shared is not None:
+            self.shared.load(prefix + "shared.", weights)
+        elif self.shared_size is not None:
             self.w_shared_up = weights[prefix + "shared.up"]
             self.w_shared_down = scaled_matrix(weights[prefix + "shared.down"], self.out_scale)
 
@@ -85,7 +103,10 @@ class RoutedExperts:
         ops.linear(h, self.w_route, logits)
         ids = ws.get("moe_ids", (t, top), torch.int32)
         weights = ws.get("moe_weights", (t, top), torch.float32)
-        ops.moe_route(logits, n, self.correction, self.route_scale, ids, weights, softmax=self.router == "softmax")
+        ops.moe_route(logits, self.routed, self.correction, self.route_scale, ids, weights, softmax=self.router == "softmax",
+                      renorm=self.renorm, groups=self.groups, keep=self.keep)
+        if self.shared is not None:
+            self.shared.forward(ctx, h, resid)
         pairs = t * top
         glu, f = self.glu, self.expert_size
         up_rows = 2 * f if glu is not None else f
@@ -100,10 +121,12 @@ class RoutedExperts:
             grouped_in = ws.get("moe_in", (tiles * tile, self.hidden_size), ctx.dtype)
             ops.moe_gather(h, sorted_rows, tile_expert, tile, grouped_in, rows_per_input=top)
             act = ws.get("moe_act", (tiles * tile, f), ctx.dtype)
-            if glu is not None:
+            if glu == "silu" and self.block == 128:
+                ops.moe_linear_tc(grouped_in, self.w_up, tile_expert, act, silu_up=True)
+            elif glu is not None:
                 both = ws.get("moe_gate_up", (tiles * tile, up_rows), torch.float32)
                 ops.moe_linear_tc(grouped_in, self.w_up, tile_expert, both)
-                ops.silu_mul(both, act, f, act=glu)     # the product stores its sums: nothing to hand back zeroed
+                ops.silu_mul(both, act, self.block, act=glu)     # the product stores its sums: nothing to hand back zeroed
             else:
                 ops.moe_linear_tc(grouped_in, self.w_up, tile_expert, act, gelu=True)
             y = ws.get("moe_y", (tiles * tile, self.hidden_size), torch.float32)
@@ -117,22 +140,24 @@ class RoutedExperts:
             tile_expert = ws.get("moe_tile_expert", (tiles,), torch.int32)
             ops.moe_align(ids, n, tile, sorted_rows, tile_expert)
             act = ws.get("moe_act", (pairs, f), ctx.dtype)
-            if glu is not None:
+            if glu == "silu" and ops.moe_silu_up_fused(h, self.w_up):
+                ops.moe_linear(h, self.w_up, sorted_rows, tile_expert, tile, act, rows_per_input=top, silu_up_block=self.block)
+            elif glu is not None:
                 both = ws.get("moe_gate_up", (pairs, up_rows), ctx.dtype)
                 ops.moe_linear(h, self.w_up, sorted_rows, tile_expert, tile, both, rows_per_input=top, gelu=False)
-                ops.silu_mul(both, act, f, act=glu)
+                ops.silu_mul(both, act, self.block, act=glu)
             else:
                 ops.moe_linear(h, self.w_up, sorted_rows, tile_expert, tile, act, rows_per_input=top, gelu=False if glu else True)
             y = ws.get("moe_y", (pairs, self.hidden_size), torch.float32)
             ops.moe_linear(act, self.w_down, sorted_rows, tile_expert, tile, y, rows_per_input=1, gelu=False)
         shared = None
-        if self.shared_size is not None:
+        if self.shared_size is not None and self.shared is None:
             sact = ws.get("ffn_act", (t, self.shared_size), ctx.dtype)
             ops.linear(h, self.w_shared_up, sact)
             ops.gelu(sact, sact)
             shared = ws.get("moe_shared", (t, self.hidden_size), torch.float32)
             ops.linear(sact, self.w_shared_down, shared)
-        ops.moe_combine(y, weights, shared, logits, n, resid, pair_pos)
+        ops.moe_combine(y, weights, shared, logits, n, resid, pair_pos, ids=ids if self.identity else None, num_experts=n, h=h)
 
 
 register_part("ffn", "routed_experts", RoutedExperts)

@@ -45,7 +45,8 @@ class SwiGLU:
                  act: str = "silu", limit: float = 0.0):
         """`names`: what the gate, up and down matrices are called behind the part's prefix.  `out_scale`: a
         constant the part's output is multiplied by; it is folded into the down matrix when that is loaded.
-        `act`: the gate's activation, "silu" or "relu" (m = (act(y Wg^T) * (y Wu^T)) Wd^T), or "clamped", which bounds
+        `act`: the gate's activation, "silu", "relu" or "gelu_tanh" (m = (act(y Wg^T) * (y Wu^T)) Wd^T; the last is
+        z / 2 (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))), or "clamped", which bounds
         both sides by `limit`: with g = min(y Wg^T, limit) and u = clamp(y Wu^T, -limit, limit),
         m = (g sigmoid(1.702 g) (u + 1)) Wd^T."""
         if act == "clamped" and not limit > 0:

@@ -2,6 +2,8 @@
 per request offers `cache_need()` like a mixer and takes the view as a third argument of `forward`."""
 from __future__ import annotations
 
+from typing import Optional
+
 import torch
 
 from .. import ops
@@ -55,5 +57,25 @@ class BigramEmbedding:
         ops.bigram_add(ctx.batch.tokens, self.table, cache.state, ctx.batch, x, self.mul_prev, self.mul_cur)
 
 
+class SoftCap:
+    """What a model does to its logits last: z <- cap * tanh(scale * z / cap), or scale * z without a cap.  In 32-bit."""
+    graph_safe = True
+
+    def __init__(self, scale: float = 1.0, cap: Optional[float] = None):
+        if cap is not None and not cap > 0:
+            raise ValueError("a soft cap is positive")
+        self.scale, self.cap = float(scale), None if cap is None else float(cap)
+
+    def weight_specs(self, prefix: str):
+        return []
+
+    def load(self, prefix: str, weights) -> None:
+        pass
+
+    def forward(self, ctx, x) -> None:
+        ops.soft_cap(x, self.scale, self.cap)
+
+
+register_part("hook", "soft_cap", SoftCap)
 register_part("hook", "learned_positions", LearnedPositions)
 register_part("hook", "bigram_embedding", BigramEmbedding)

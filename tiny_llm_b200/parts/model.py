@@ -71,7 +71,12 @@ class SandwichBlock:
     """Norms on both sides of each branch: x += norm1_out(mixer(norm1(x))); x += norm2_out(ffn(norm2(x))).  The two
     norms behind the branches are named in `LayerSpec.more` under the roles "norm1_out" and "norm2_out" (the second
     only when the layer has a feed-forward).  A branch adds its output into a zeroed float32 buffer, whose norm is
-    then added into the stream by one kernel that also hands the buffer back zeroed."""
+    then added into the stream by one kernel that also hands the buffer back zeroed.  Where the norms allow it (layer
+    norms) that kernel also takes the norm ahead of the next branch, the next layer's included: the model names that
+    norm in `ctx.next_norm`, and `ctx.norm_ahead` = (the stream's address, the norm, its output) hands the rows on
+    (whoever else changes the stream drops it)."""
+
+    takes_norm_ahead = True
 
     def __init__(self, spec: LayerSpec, shares_cache: bool = False):
         more = {role: (family, part, name) for role, family, part, name in spec.more}
@@ -94,7 +99,7 @@ class SandwichBlock:
             self.ffn = build_part("ffn", spec.ffn)
             self.norm2_out = build_part("norm", more["norm2_out"][1])
         self._out_names = {role: more[role][2] for role in ("norm1_out", "norm2_out") if role in more}
-        self.hidden_size = None
+        self.first_norm = self.norm1     # what the layer does to the stream first
 
     def parts(self):
         return [p for p in (self.norm1, self.mixer, self.norm1_out, self.norm2, self.ffn, self.norm2_out) if p is not None]
@@ -114,14 +119,21 @@ class SandwichBlock:
             part.load(name, weights)
 
     def forward(self, ctx, resid, cache) -> None:
-        h = self.norm1.forward(ctx, resid)
+        ahead = getattr(ctx, "norm_ahead", None)
+        held = ahead is not None and ahead[0] == resid.data_ptr() and ahead[1] is self.norm1 and ahead[2].shape[0] == resid.shape[0]
+        h = ahead[2] if held else self.norm1.forward(ctx, resid)
+        ctx.norm_ahead = None
         branch = ctx.workspace.get_zeroed("branch_out", tuple(resid.shape))
         self.mixer.forward(ctx, h, branch, cache)
-        self.norm1_out.add_into(ctx, branch, resid)
+        after = getattr(ctx, "next_norm", None)
+        h = self.norm1_out.add_into(ctx, branch, resid, then=after if self.ffn is None else self.norm2)
         if self.ffn is not None:
-            h = self.norm2.forward(ctx, resid)
+            if h is None:
+                h = self.norm2.forward(ctx, resid)
             self.ffn.forward(ctx, h, branch)
-            self.norm2_out.add_into(ctx, branch, resid)
+            h = self.norm2_out.add_into(ctx, branch, resid, then=after)
+        if h is not None:
+            ctx.norm_ahead = (resid.data_ptr(), after, h)
 
 
 register_block("sandwich_norm", SandwichBlock)
@@ -354,6 +366,7 @@ class DecoderModel:
                       twin=None if stages is None or self.after_embedding is not None else stages[0])
         # a rounded copy of the stream that a block may leave for the next one
         ctx.stream_copy = None if copy is None else (resid.data_ptr(), copy)
+        ctx.norm_ahead = None
         if self._hook_keeps:
             self.after_embedding.forward(ctx, resid, ctx.cache_view(len(s.order)))
         elif self.after_embedding is not None:
@@ -366,6 +379,12 @@ class DecoderModel:
                 ops.embedding(b.tokens, self.embed, resid, accumulate=True)
                 ctx.stream_copy = None
             block = self.blocks[call.layer]
+            # the norm that reads the stream right behind this layer, for a block that can take it along
+            following = s.order[pos + 1] if pos + 1 < len(s.order) else None
+            ctx.next_norm = None if following is None or following.add_embedding or stages is not None else \
+                getattr(self.blocks[following.layer], "first_norm", None)
+            if not getattr(block, "takes_norm_ahead", False):
+                ctx.norm_ahead = None
             if stages is None:
                 block.forward(ctx, resid, ctx.cache_view(owner))
             else:

@@ -1,6 +1,6 @@
 """Norms.  RMSNorm: y_j = (w_j x_j) / sqrt(mean_j(x_j^2) + eps), statistics in 32-bit
 (tiny_llm/ops/cuda/norm.cu:16-49).  Any width; the reference stops at 2048.  With `one_plus` the stored weight lies
-around zero and the norm multiplies by 1 + w_j.  LayerNorm: y_j = (x_j - mean) / sqrt(var + eps) w_j + b_j."""
+around zero and the norm multiplies by 1 + w_j.  LayerNorm: y_j = (x_j - mean) / sqrt(var + eps) w_j (+ b_j)."""
 from __future__ import annotations
 
 from .. import ops
@@ -34,10 +34,11 @@ class RMSNorm:
             w = w.reshape(1).expand(self.size).contiguous()
         self.weight = (w + 1.0).contiguous() if self.one_plus else w
 
-    def add_into(self, ctx, branch, resid, copy=None) -> None:
+    def add_into(self, ctx, branch, resid, copy=None, then=None):
         """resid += norm(branch): for a block that norms a branch's output before it joins the stream.  `branch` is a
         zeroed float32 buffer that products added into; it is handed back zeroed.  `copy` (bfloat16) also receives the
-        new stream, rounded."""
+        new stream, rounded.  `then`: the norm that reads the new stream next; a norm that can take it along returns what
+        `then.forward(ctx, resid)` would (this one returns None)."""
         ops.rms_norm_add(branch, self.weight, self.eps, 1.0, resid, copy=copy)
 
     def forward(self, ctx, x, rows=None):
@@ -76,19 +77,32 @@ class DynamicTanh:
 
 class LayerNorm:
     """y_j = (x_j - mean) / sqrt(mean((x - mean)^2) + eps) * w_j + b_j, all in 32-bit.  The weight is stored under the
-    part's own name, the bias beside it as `<name>.b`."""
+    part's own name, the bias beside it as `<name>.b` (`has_bias=False`: there is none)."""
     graph_safe = True
 
-    def __init__(self, size: int, eps: float):
-        self.size, self.eps = size, float(eps)
+    def __init__(self, size: int, eps: float, has_bias: bool = True):
+        self.size, self.eps, self.has_bias = size, float(eps), has_bias
         self.weight = self.bias = None
 
     def weight_specs(self, prefix: str):
-        return [WeightSpec(prefix, (self.size,), FLOAT32, init=("uniform", 0.5, 1.5)),
-                WeightSpec(prefix + ".b", (self.size,), FLOAT32, init=("normal", 0.2))]
+        specs = [WeightSpec(prefix, (self.size,), FLOAT32, init=("uniform", 0.5, 1.5))]
+        if self.has_bias:
+            specs.append(WeightSpec(prefix + ".b", (self.size,), FLOAT32, init=("normal", 0.2)))
+        return specs
 
     def load(self, prefix: str, weights) -> None:
-        self.weight, self.bias = weights[prefix], weights[prefix + ".b"]
+        self.weight, self.bias = weights[prefix], weights[prefix + ".b"] if self.has_bias else None
+
+    def add_into(self, ctx, branch, resid, copy=None, then=None):
+        """resid += norm(branch), as RMSNorm.add_into; a following layer norm `then` of the new stream is taken in the same
+        kernel and its output returned."""
+        if not isinstance(then, LayerNorm) or then.size != self.size:
+            ops.layer_norm_add(branch, resid, self.weight, self.bias, self.eps, copy=copy)
+            return None
+        out = ctx.workspace.get("norm_out", (resid.shape[0], self.size), ctx.dtype)
+        ops.layer_norm_add(branch, resid, self.weight, self.bias, self.eps, copy=copy,
+                           then=(then.weight, then.bias, then.eps), out=out)
+        return out
 
     def join(self, ctx, branch, resid, stream_scale, out_bias=None, copy=None, depth=None) -> None:
         """resid <- norm(stream_scale * resid + branch + out_bias): for a block that norms the sum.  `branch` is a zeroed

@@ -17,7 +17,7 @@ meet in one kernel (`ops.attention_talk`), which takes scale, temperatures and m
 M[h, g] = talk[h, g] * temp[g] * scale (made in 32-bit at load).  `conv` > 0 passes every channel of q, k and v (projection
 plus bias) through a causal filter of that many taps before the norms; the last conv - 1 inputs of a request are state
 beside its keys and values.  `qk_norm="whole"` norms all query rows of a token at once, and all its key rows, with a
-weight per channel.  `bias_max` adds a learned bias `rel`[bucket(distance), head] to the scaled scores (`distance_buckets`;
+weight per channel (a rotation comes behind either).  `bias_max` adds a learned bias `rel`[bucket(distance), head] to the scaled scores (`distance_buckets`;
 the number of buckets is the stored table's).  `keep_first` leaves the first positions visible to every token whatever
 the window.  `out_bias` adds `o.b` behind the output projection (a block that joins the branch itself takes it over:
 `defer_out_bias`).
@@ -114,10 +114,10 @@ class SinkAttention:
             raise ValueError(f"unknown gate kind {gate!r} (True: one per value, \"head\": one per head, False: none)")
         if qk_norm not in (True, False, "whole"):
             raise ValueError(f"unknown query/key norm {qk_norm!r} (True: per head, \"whole\": all heads at once, False: none)")
-        # filters and whole-row norms leave q, k, v through one kernel that knows neither rotations nor stretched queries
+        # filters and whole-row norms leave q, k, v through one kernel that knows no stretched queries
         self.filtered = conv > 0 or qk_norm == "whole"
-        if self.filtered and (qk_norm is True or rot_dims or stretch_every):
-            raise ValueError("short filters and norms over all heads go without norms per head, rotations and stretched queries")
+        if self.filtered and (qk_norm is True or stretch_every):
+            raise ValueError("short filters and norms over all heads go without norms per head and stretched queries")
         if (head_temp or talk) and (bias_max is not None or keep_first or self.filtered):
             raise ValueError("mixed scores go without filters, distance biases and kept first positions")
         self.conv, self.bias_max, self.out_bias = int(conv), bias_max, out_bias
@@ -220,7 +220,8 @@ class SinkAttention:
             q = ctx.workspace.get("filtered_q", (t, self.q_dim), ctx.dtype)
             ops.conv_norm_kv_write(proj, ctx.batch, nh, nkv, kd, vd, cache.k, cache.v, cache.slot_mapping, q,
                                    bias=self.bias_row, taps=self.taps, kept=None if kept is None else kept.state,
-                                   norm_q=self.norms[0], norm_k=self.norms[1], eps=self.eps)
+                                   norm_q=self.norms[0], norm_k=self.norms[1], eps=self.eps, freq=self.freq,
+                                   rot_pairs=self.rot_layout == "pairs", rot_mag=self.rot_mag)
         else:
             ops.qk_norm_kv_write(proj, ctx.batch.positions, nh, nkv, kd, vd, cache.k, cache.v, cache.slot_mapping,
                                  *self.biases, *self.norms, eps=self.eps, stretch_coef=self.stretch_coef,
