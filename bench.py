@@ -18,7 +18,8 @@ like kernels, each against its roofline (`--only decode` with it: the decode poi
 the same for a Zozenex model (retention and gated linear attention, window attention with pooled blocks, routed
 experts) beside the Dunelix model at equal width, layers and vocabulary, `--design gevovik` for a Gevovik model beside
 the Fiponex model, `--design vigodra` for a Vigodra model (attention behind short filters with a distance bias, latent
-attention with a gate per value, post-norm blocks with a depth average) beside the Gevovik model, `--design fiponex` for a Fiponex model (gated
+attention with a gate per value, post-norm blocks with a depth average) beside the Gevovik model, `--design lovapel` for a
+Lovapel model (window attention with a sink, sandwich layer norms, grouped experts with identity experts) beside the Fiponex model, `--design fiponex` for a Fiponex model (gated
 delta rule, latent attention, attention with a sink, dense and routed gated feed-forwards) beside the Zozenex model."""
 import argparse
 import json
@@ -746,8 +747,10 @@ def fiponex_decode_bytes(model, runner, batch, mean_ctx, itemsize):
         if f is None or not hasattr(f, "num_experts"):
             continue
         expert = (3 if f.glu is not None else 2) * f.expert_size * f.hidden_size * itemsize
-        chosen = f.num_experts * (1.0 - (1.0 - f.top / f.num_experts) ** batch)
+        chosen = f.num_experts * (1.0 - (1.0 - f.top / f.routed) ** batch)
         total += (chosen - f.num_experts) * expert     # spec_weight_bytes counts every expert
+    if model.spec.tie_word_embeddings:                 # the table is the output matrix too
+        total += model.spec.vocab_size * model.spec.hidden_size * itemsize
     for g in runner.cache.groups:
         seen = mean_ctx if g.need.window is None else min(mean_ctx, g.need.window + g.need.keep_first)
         total += batch * seen * g.bytes_per_token(itemsize)
@@ -1249,6 +1252,159 @@ def vigodra_kernels(dtype, device, pk, tokens=2048):
     return out
 
 
+# `--design lovapel`: a Lovapel model (layer norms on both sides of every branch, attention over a window with a sink, norms
+# over the whole projection and a rotation, dense feed-forwards gated by the tanh form of GELU and gated experts chosen in
+# groups with identity experts among them and a shared one beside them, soft-capped logits from the embedding table) at the
+# same width, layers and vocabulary, beside the Fiponex model above (the closest design the engine has: sandwich norms,
+# attention with a sink, softmax-routed gated experts).  No span of layers is repeated, so that both run as many.
+def lovapel_shape(layers=DESIGN_LAYERS, width=2048, vocab=32000, ff=5632, window=1024):
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": 1408}, "shared": {"ff": 1408},
+           "router": {"experts": 30, "identity": 2, "top": 4, "groups": {"count": 4, "keep": 2}}}
+    att = {"heads": 16, "kv_heads": 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": window},
+           "rot": {"dims": 64, "base": 10000.0}}
+    return {"architecture": "Lovapel", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "initializer_range": 0.02,
+            "logit_scale": 0.5, "logit_softcap": 30.0,
+            "layers": [{"type": "attention", "mixer": att, "mlp": dense if i % 2 == 0 else moe} for i in range(layers)]}
+
+
+def lovapel_kernels(dtype, device, pk, tokens=2048):
+    """The design's kernels alone at the sizes of one layer of the --design shape and `tokens` tokens of one prompt, and
+    their like kernels of the Fiponex, Vigodra and Zozenex paths: microseconds, achieved GB/s or TFLOP/s, share of the peak."""
+    import types
+    import torch
+    from tiny_llm_b200 import ops
+    from tiny_llm_b200.engine import Workspace
+    t, width, page, window = tokens, 2048, PAGE, 1024
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=device)
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=device)
+    rnd = lambda *shape: torch.randn(*shape, device=device).to(dtype)
+    out = {}
+    isz = 2 if dtype == torch.bfloat16 else 4
+
+    def mem(name, us, nbytes):
+        out[name] = {"us": round(us, 2), "gbs": round(nbytes / us / 1e3, 1), "frac": round(nbytes / us / 1e3 / pk["hbm_gbs"], 3)}
+
+    def flop(name, us, flops):
+        out[name] = {"us": round(us, 2), "tflops": round(flops / us / 1e6, 1), "frac": round(flops / us / 1e6 / pk["bf16_tflops"], 3)}
+
+    ws = Workspace(torch.device(device))
+    pages = -(-t // page)
+    table = i32([list(range(pages))])
+    slots, pos = i32(list(range(t))), i32(list(range(t)))
+    meta = types.SimpleNamespace(token_request=i32([0] * t), positions=pos, cu_q=i32([0, t]), q_start=i32([0]), slots=i32([1]),
+                                 num_requests=1, num_tokens=t, max_q_len=t, max_kv_len=t, num_leading_decodes=0)
+
+    # attention: norms over all heads + rotation + cache write; the scores over a window with a sink
+    h, kvh, kd, vd = 16, 4, 128, 128
+    nqc, nkc, nvc = h * kd, kvh * kd, kvh * vd
+    ch = nqc + nkc + nvc
+    proj = rnd(t, ch)
+    kc = torch.zeros(pages, kvh, page, kd, dtype=dtype, device=device)
+    vc = torch.zeros(pages, kvh, page, vd, dtype=dtype, device=device)
+    q = torch.empty(t, nqc, dtype=dtype, device=device)
+    wq, wk = torch.ones(nqc, device=device), torch.ones(nkc, device=device)
+    freq = torch.pow(torch.tensor(10000.0), -torch.arange(32, dtype=torch.float32) * 2 / 64).to(device)
+    mem("conv_norm_kv_write (norms over all heads, rotation, no filter)", time_kernel(lambda: ops.conv_norm_kv_write(
+        proj, meta, h, kvh, kd, vd, kc, vc, slots, q, norm_q=wq, norm_k=wk, eps=1e-6, freq=freq), flush), t * ch * isz * 2)
+    mem("conv_norm_kv_write (norms over all heads, no rotation; like)", time_kernel(lambda: ops.conv_norm_kv_write(
+        proj, meta, h, kvh, kd, vd, kc, vc, slots, q, norm_q=wq, norm_k=wk, eps=1e-6), flush), t * ch * isz * 2)
+    qn, kn = torch.ones(kd, device=device), torch.ones(kd, device=device)
+    mem("qk_norm_kv_write (like: norms per head, rotation)", time_kernel(lambda: ops.qk_norm_kv_write(
+        proj, pos, h, kvh, kd, vd, kc, vc, slots, None, None, None, qn, kn, eps=1e-6, freq=freq), flush), t * ch * isz * 2)
+    att16 = torch.empty(t, h * vd, dtype=dtype, device=device)
+    att32 = torch.empty(t, h * vd, dtype=torch.float32, device=device)
+    sink = torch.zeros(h, device=device)
+    wpairs, pairs = sum(min(p + 1, window) for p in range(t)), t * (t + 1) // 2
+    kq = rnd(t, nqc)
+    flop("attention, window 1024, sink (16 heads of 128)", time_kernel(lambda: ops.paged_attention_maps(
+        kq, h, kvh, 1, kd, vd, kc, vc, table, meta, att16, kd ** -0.5, window, None, sink=sink, workspace=ws), flush, repeats=5),
+        2.0 * wpairs * h * (kd + vd))
+    flop("attention with a sink, causal (like)", time_kernel(lambda: ops.paged_attention_maps(
+        kq, h, kvh, 1, kd, vd, kc, vc, table, meta, att32, kd ** -0.5, None, None, sink=sink, workspace=ws), flush, repeats=5),
+        2.0 * pairs * h * (kd + vd))
+
+    # the stream: the norm behind a branch with the next branch's norm; the gate of the dense feed-forward
+    x, branch = torch.randn(t, width, device=device), torch.randn(t, width, device=device)
+    w1 = torch.ones(width, device=device)
+    yy = torch.empty(t, width, dtype=dtype, device=device)
+    mem("layer_norm_add with the next norm", time_kernel(lambda: ops.layer_norm_add(
+        branch, x, w1, None, 1e-6, then=(w1, None, 1e-6), out=yy), flush), t * width * (16 + isz))
+    mem("layer_norm_add", time_kernel(lambda: ops.layer_norm_add(branch, x, w1, None, 1e-6), flush), t * width * 16)
+    mem("rms_norm_add (like)", time_kernel(lambda: ops.rms_norm_add(branch, w1, 1e-6, 1.0, x), flush), t * width * 16)
+    mem("layer_norm", time_kernel(lambda: ops.layer_norm(x, w1, None, 1e-6, yy), flush), t * width * (4 + isz))
+    mem("rms_norm (like)", time_kernel(lambda: ops.rms_norm(x, w1, 1e-6, yy), flush), t * width * (4 + isz))
+    ff = 5632
+    h_in, w_gu = rnd(t, width), rnd(2 * ff, width)
+    act = torch.empty(t, ff, dtype=dtype, device=device)
+    for name, a in (("gate and up product with the tanh form of GELU", "gelu_tanh"), ("gate and up product with SiLU (like)", "silu")):
+        flop(name, time_kernel(lambda: ops.linear_swiglu(h_in, w_gu, act, 128, ws, act=a), flush), 2.0 * t * 2 * ff * width)
+    sact = torch.empty(8, ff, dtype=dtype, device=device)
+    for name, a in (("gate and up product, 8 tokens, tanh form of GELU", "gelu_tanh"), ("gate and up product, 8 tokens, SiLU (like)", "silu")):
+        mem(name, time_kernel(lambda: ops.linear_swiglu(h_in[:8], w_gu, sact, 128, ws, act=a), flush), 2 * ff * width * isz)
+
+    # the experts: groups, renormalised weights, identity experts; the gate inside the grouped product; the combine
+    experts, identity, top, ff = 30, 2, 4, 1408
+    routed = experts + identity
+    logits = torch.randn(t, routed, device=device)
+    corr = torch.randn(routed, device=device) * 0.01
+    ids = torch.empty(t, top, dtype=torch.int32, device=device)
+    wts = torch.empty(t, top, device=device)
+    mem("moe_route (groups, renormalised)", time_kernel(lambda: ops.moe_route(
+        logits, routed, corr, 1.0, ids, wts, softmax=True, renorm=True, groups=4, keep=2), flush), t * (routed * 4 + top * 8))
+    ids2, wts2 = torch.empty_like(ids), torch.empty_like(wts)
+    mem("moe_route (softmax; like)", time_kernel(lambda: ops.moe_route(logits, routed, None, 1.0, ids2, wts2, softmax=True), flush),
+        t * (routed * 4 + top * 8))
+    t128 = ops.moe_max_tiles(t * top, experts, ops.MOE_TC_TILE)
+    rows128 = torch.empty(t128 * 128, dtype=torch.int32, device=device)
+    texp128 = torch.empty(t128, dtype=torch.int32, device=device)
+    pos128 = torch.empty(t * top, dtype=torch.int32, device=device)
+    mem("moe_align (shared with the like)", time_kernel(lambda: ops.moe_align(ids, experts, 128, rows128, texp128, pos128), flush), t * top * 12)
+    resid = torch.zeros(t, width, device=device)
+    if dtype == torch.bfloat16:
+        chosen = int((ids < experts).sum())
+        w_up = (torch.randn(experts, 2 * ff, width, device=device) * 0.02).to(dtype)
+        w_down = (torch.randn(experts, width, ff, device=device) * 0.02).to(dtype)
+        gin = torch.zeros(t128 * 128, width, dtype=dtype, device=device)
+        both = torch.zeros(t128 * 128, 2 * ff, device=device)
+        gact = torch.zeros(t128 * 128, ff, dtype=dtype, device=device)
+        gy = torch.zeros(t128 * 128, width, device=device)
+        mem("moe_gather (shared with the like)", time_kernel(lambda: ops.moe_gather(h_in, rows128, texp128, 128, gin, rows_per_input=top), flush),
+            chosen * width * 2 * isz)
+        flop("moe_linear_tc gate and up with SiLU * up inside", time_kernel(lambda: ops.moe_linear_tc(gin, w_up, texp128, gact, silu_up=True), flush),
+             2.0 * chosen * 2 * ff * width)
+        flop("moe_linear_tc gate and up, 32-bit sums out, and silu_mul (like)", time_kernel(lambda: (
+            ops.moe_linear_tc(gin, w_up, texp128, both), ops.silu_mul(both, gact, 128, act="silu")), flush), 2.0 * chosen * 2 * ff * width)
+        flop("moe_linear_tc down (shared with the like)", time_kernel(lambda: ops.moe_linear_tc(gact, w_down, texp128, gy), flush),
+             2.0 * chosen * ff * width)
+        mem("moe_combine with identity experts", time_kernel(lambda: ops.moe_combine(
+            gy, wts, None, None, 0, resid, pos128, ids=ids, num_experts=experts, h=h_in), flush), chosen * width * 4 + t * width * (8 + isz))
+        ops.moe_align(ids2, routed, 128, torch.empty((t128 + 2) * 128, dtype=torch.int32, device=device),
+                      torch.empty(t128 + 2, dtype=torch.int32, device=device), pos128)
+        gy2 = torch.zeros((t128 + 2) * 128, width, device=device)
+        mem("moe_combine (like)", time_kernel(lambda: ops.moe_combine(gy2, wts2, None, None, 0, resid, pos128), flush),
+            t * top * width * 4 + t * width * 8)
+        # a decode step of 8 tokens: 32 pairs, every one an expert of its own at worst
+        d_ids = (torch.arange(8 * top, device=device, dtype=torch.int32).view(8, top) * 7) % experts
+        tiles = ops.moe_max_tiles(8 * top, experts, 16)
+        rows16, texp16 = torch.empty(tiles * 16, dtype=torch.int32, device=device), torch.empty(tiles, dtype=torch.int32, device=device)
+        ops.moe_align(d_ids, experts, 16, rows16, texp16)
+        dact, dboth = torch.empty(8 * top, ff, dtype=dtype, device=device), torch.empty(8 * top, 2 * ff, dtype=dtype, device=device)
+        used = int(d_ids.unique().numel())
+        mem("moe_linear gate and up, 8 tokens, SiLU * up inside", time_kernel(lambda: ops.moe_linear(
+            h_in[:8], w_up, rows16, texp16, 16, dact, rows_per_input=top, silu_up_block=128), flush), used * 2 * ff * width * isz)
+        mem("moe_linear gate and up, 8 tokens, and silu_mul (like)", time_kernel(lambda: (ops.moe_linear(
+            h_in[:8], w_up, rows16, texp16, 16, dboth, rows_per_input=top), ops.silu_mul(dboth, dact, 128)), flush), used * 2 * ff * width * isz)
+        dy = torch.empty(8 * top, width, device=device)
+        mem("moe_linear down, 8 tokens (shared with the like)", time_kernel(lambda: ops.moe_linear(dact, w_down, rows16, texp16, 16, dy), flush),
+            used * ff * width * isz)
+    lg = torch.randn(64, 32000, device=device)
+    mem("soft_cap (64 rows of logits)", time_kernel(lambda: ops.soft_cap(lg, 0.5, 30.0), flush), 64 * 32000 * 8)
+    lg2 = torch.empty_like(lg)
+    mem("unary copy of 64 rows of logits (like)", time_kernel(lambda: ops.unary(lg, lg2), flush), 64 * 32000 * 8)
+    return out
+
+
 def design_run(args, dtype, device, pk):
     import gc
     import torch
@@ -1281,13 +1437,18 @@ def design_run(args, dtype, device, pk):
                         "plain + 64 rotated, values of 128, latent 192, window 1024, gate per value); attention; latent attention "
                         "reading the cache of the one before; post-norm blocks averaged over the depth; every layer with a clamped "
                         "gated feed-forward of 5632; beside: the Gevovik model of --design gevovik at equal width, layers and "
-                        "vocabulary"}
+                        "vocabulary",
+             "lovapel": "width 2048, vocabulary 32000; attention (16 heads, 4 key/value heads, keys and values of 128, window 1024, "
+                        "64 rotated values, norms over all heads, sink); layers in turn: a dense feed-forward of 5632 gated by the "
+                        "tanh form of GELU; 30 gated experts of 1408 and 2 identity experts, 4 chosen in 2 of 4 groups, a shared "
+                        "expert of 1408; beside: the Fiponex model of --design fiponex at equal width, layers and vocabulary"}
     result = {"design": args.design, "dtype": args.dtype, "layers": DESIGN_LAYERS, "peaks": pk["source"],
               "sizes": sizes[args.design],
               "l2": "whole steps: weights larger than L2; kernels alone: L2 flushed before every timed call"}
     sampler = ClockSampler().start()
     labels = {"dunelix": ("dunelix", "llama"), "zozenex": ("zozenex", "dunelix"), "fiponex": ("fiponex", "zozenex"),
-              "gevovik": ("gevovik", "fiponex"), "vigodra": ("vigodra", "gevovik")}[args.design]
+              "gevovik": ("gevovik", "fiponex"), "vigodra": ("vigodra", "gevovik"),
+              "lovapel": ("lovapel", "fiponex")}[args.design]
     for label in labels[:1 if args.only == "decode" else 2]:
         if label == "dunelix":
             cfg, model = build_design(dunelix_shape(), dtype, device)
@@ -1299,6 +1460,8 @@ def design_run(args, dtype, device, pk):
             cfg, model = build_design(gevovik_shape(), dtype, device)
         elif label == "vigodra":
             cfg, model = build_design(vigodra_shape(), dtype, device)
+        elif label == "lovapel":
+            cfg, model = build_design(lovapel_shape(), dtype, device)
         else:
             cfg, model = build_model(DESIGN_LAYERS, dtype, device)
         runner = make_runner(model, dtype, device, max_tokens=64 * CONTEXT, page_size=PAGE, max_requests=64,
@@ -1311,7 +1474,7 @@ def design_run(args, dtype, device, pk):
             ms, launched, ctx = timed_decode(runner, bsz, CONTEXT - (REPEATS * steps + warmup), steps, warmup, out, repeats=REPEATS)
             moved = design_decode_bytes(model, runner, bsz, ctx, itemsize) if label == "dunelix" else \
                 zozenex_decode_bytes(model, runner, bsz, ctx, itemsize) if label == "zozenex" else \
-                fiponex_decode_bytes(model, runner, bsz, ctx, itemsize) if label in ("fiponex", "gevovik", "vigodra") else \
+                fiponex_decode_bytes(model, runner, bsz, ctx, itemsize) if label in ("fiponex", "gevovik", "vigodra", "lovapel") else \
                 decode_bytes(model, runner, bsz, ctx, itemsize)
             rec[f"decode_b{bsz}"] = {"ms_per_step": round(ms, 4), "tokens_per_s": round(bsz * 1e3 / ms, 1),
                                      "hbm_frac": round(moved / (ms * 1e-3) / 1e9 / pk["hbm_gbs"], 4), "gpu_launches": launched}
@@ -1322,7 +1485,7 @@ def design_run(args, dtype, device, pk):
     result["clocks"] = sampler.stop()
     if dtype == torch.bfloat16 and args.only == "all":
         result["kernels"] = {"dunelix": design_kernels, "zozenex": zozenex_kernels, "fiponex": fiponex_kernels,
-                             "gevovik": gevovik_kernels, "vigodra": vigodra_kernels}[args.design](dtype, device, pk)
+                             "gevovik": gevovik_kernels, "vigodra": vigodra_kernels, "lovapel": lovapel_kernels}[args.design](dtype, device, pk)
     ops.check_status()
     print(json.dumps(result))
     return 0
@@ -1347,7 +1510,7 @@ def main():
     ap.add_argument("--page-size", type=int, default=PAGE, help="tokens per page of the cache")
     ap.add_argument("--shape", default="tinyllama", choices=["tinyllama"] + list(OTHER_SHAPES),
                     help="layer sizes for --only runs (profiler captures of the other models' kernels)")
-    ap.add_argument("--design", default=None, choices=["dunelix", "zozenex", "fiponex", "gevovik", "vigodra"],
+    ap.add_argument("--design", default=None, choices=["dunelix", "zozenex", "fiponex", "gevovik", "vigodra", "lovapel"],
                     help="instead of the flagship run: this design's prefill and decode at real layer sizes beside the Llama "
                          "decoder at equal sizes, and its kernels beside their like kernels (one plain line, no record)")
     ap.add_argument("--quick", action="store_true",

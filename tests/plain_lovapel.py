@@ -84,13 +84,15 @@ def gelu_tanh(x):
 
 
 def rotate_halves(x, pos, dims, base):
-    """x [T, heads, D]: value i with value i + dims / 2, i < dims / 2, by pos * base^(-2i / dims)."""
+    """x [T, heads, D]: value i with value i + dims / 2, i < dims / 2, by pos * base^(-2i / dims); the angle is taken in
+    x's own precision (in 32-bit, at position 300, it is off by some hundred-thousandths of a radian)."""
     if not dims:
         return x
     half = dims // 2
     i = torch.arange(half, dtype=torch.float64)
-    a = pos.to(torch.float64)[:, None, None] * torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / dims)
-    c, s = torch.cos(a).to(x.dtype), torch.sin(a).to(x.dtype)
+    f = torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / dims)
+    a = pos.to(x.dtype)[:, None, None] * f.to(x.dtype)
+    c, s = torch.cos(a), torch.sin(a)
     u, v = x[..., :half], x[..., half:dims]
     return torch.cat([u * c - v * s, v * c + u * s, x[..., dims:]], dim=-1)
 

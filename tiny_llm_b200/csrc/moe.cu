@@ -433,24 +433,53 @@ struct CombineArgs {
   int ld_h;
 };
 
-template <typename T>
+// V neighbouring columns per thread (1 or 4; 4: rows on 16-byte boundaries, h on 4 values').
+template <typename T, int V>
 __global__ void moe_combine_kernel(CombineArgs a) {
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
   float g = 0.f;
   if (a.shared) g = 1.f / (1.f + expf(-a.logits[(size_t)t * a.ld_logits + a.gate_col]));
-  for (int c = threadIdx.x; c < a.width; c += blockDim.x) {
-    float acc = 0.f;
+  auto fetch = [](const float* p, float* v) {
+    if (V == 4) {
+      const float4 x = *reinterpret_cast<const float4*>(p);
+      v[0] = x.x; v[1 % V] = x.y; v[2 % V] = x.z; v[3 % V] = x.w;
+    } else {
+      v[0] = p[0];
+    }
+  };
+  for (int c = threadIdx.x * V; c < a.width; c += blockDim.x * V) {
+    float acc[V], v[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) acc[e] = 0.f;
+#pragma unroll 4
     for (int x = 0; x < a.top; ++x) {
       const size_t pair = (size_t)t * a.top + x;
-      const float v = a.ids && a.ids[pair] >= a.n_experts
-                          ? to_f32(((const T*)a.h)[(size_t)t * a.ld_h + c])
-                          : a.y[(a.pair_pos ? (size_t)a.pair_pos[pair] : pair) * a.width + c];
-      acc = fmaf(a.weights[pair], v, acc);
+      if (a.ids && a.ids[pair] >= a.n_experts) {
+        struct __align__(sizeof(T) * V) Row { T v[V]; };
+        const Row row = *reinterpret_cast<const Row*>((const T*)a.h + (size_t)t * a.ld_h + c);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] = to_f32(row.v[e]);
+      } else {
+        fetch(a.y + (a.pair_pos ? (size_t)a.pair_pos[pair] : pair) * a.width + c, v);
+      }
+      const float w = a.weights[pair];
+#pragma unroll
+      for (int e = 0; e < V; ++e) acc[e] = fmaf(w, v[e], acc[e]);
     }
-    if (a.shared) acc = fmaf(g, a.shared[(size_t)t * a.width + c], acc);
-    a.resid[(size_t)t * a.width + c] += acc;
+    if (a.shared) {
+      fetch(a.shared + (size_t)t * a.width + c, v);
+#pragma unroll
+      for (int e = 0; e < V; ++e) acc[e] = fmaf(g, v[e], acc[e]);
+    }
+    float* dst = a.resid + (size_t)t * a.width + c;
+    fetch(dst, v);
+    if (V == 4) {
+      *reinterpret_cast<float4*>(dst) = make_float4(v[0] + acc[0], v[1 % V] + acc[1 % V], v[2 % V] + acc[2 % V], v[3 % V] + acc[3 % V]);
+    } else {
+      dst[0] = v[0] + acc[0];
+    }
   }
 }
 
@@ -580,11 +609,16 @@ extern "C" int tllm_moe_combine(const float* y, const float* weights, int top, c
   CombineArgs a;
   a.y = y; a.weights = weights; a.top = top; a.shared = shared; a.logits = logits; a.ld_logits = ld_logits; a.gate_col = gate_col;
   a.resid = resid; a.width = width; a.pair_pos = pair_pos; a.ids = ids; a.n_experts = n_experts; a.h = h; a.ld_h = ld_h;
+  const auto off = [](const void* p, int to) { return ((uintptr_t)p % to) != 0; };
+  const int h_size = h_dtype == TLLM_F32 ? 4 : 2;
+  const bool vec = width % 4 == 0 && !off(y, 16) && !off(shared, 16) && !off(resid, 16) && (!ids || (ld_h % 4 == 0 && !off(h, 4 * h_size)));
   const int threads = width >= 1024 ? 256 : 128;
   cudaStream_t s = (cudaStream_t)stream;
-  if (h_dtype == TLLM_F32) TLLM_LAUNCH("moe_combine", moe_combine_kernel<float>, (unsigned)n_tokens, threads, 0, s, a);
-  else if (h_dtype == TLLM_BF16) TLLM_LAUNCH("moe_combine", moe_combine_kernel<__nv_bfloat16>, (unsigned)n_tokens, threads, 0, s, a);
-  else TLLM_FAIL(TLLM_ERR_ARG, "moe_combine: unknown dtype code %d", h_dtype);
+  TLLM_REQUIRE(h_dtype == TLLM_F32 || h_dtype == TLLM_BF16, "moe_combine: unknown dtype code %d", h_dtype);
+  if (h_dtype == TLLM_F32 && vec) TLLM_LAUNCH("moe_combine", (moe_combine_kernel<float, 4>), (unsigned)n_tokens, threads, 0, s, a);
+  else if (h_dtype == TLLM_F32) TLLM_LAUNCH("moe_combine", (moe_combine_kernel<float, 1>), (unsigned)n_tokens, threads, 0, s, a);
+  else if (vec) TLLM_LAUNCH("moe_combine", (moe_combine_kernel<__nv_bfloat16, 4>), (unsigned)n_tokens, threads, 0, s, a);
+  else TLLM_LAUNCH("moe_combine", (moe_combine_kernel<__nv_bfloat16, 1>), (unsigned)n_tokens, threads, 0, s, a);
   return TLLM_OK;
 }
 
