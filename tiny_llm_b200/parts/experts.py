@@ -66,7 +66,7 @@ class RoutedExperts:
         specs = [WeightSpec(prefix + "router", (self.routed, h), COMPUTE)]
         if self.has_correction:   # (a softmax's scores lie around 1 / routed: corrections of their size)
             specs.append(WeightSpec(prefix + "correction", (self.routed,), FLOAT32,
-                                    init=("normal", 0.3 if self.router == "sigmoid" else 0.3 / self.routed)))
+                                    init=("normal", 0.3 if self.router == "sigmoid" else 1.0 / self.routed)))
         for e in range(self.num_experts):
             if self.glu is not None:
                 specs.append(WeightSpec(prefix + f"e{e}.gate", (f, h), COMPUTE))
